@@ -33,7 +33,8 @@ extern "C" {
 
 typedef void* lri_stream_t; /* a cudaStream_t */
 
-enum lri_dtype { LRI_BF16 = 0, LRI_FP16 = 1 };
+/* LRI_FP32 is taken by the entry points that say so (every product and sum a true 32-bit operation). */
+enum lri_dtype { LRI_BF16 = 0, LRI_FP16 = 1, LRI_FP32 = 2 };
 
 enum lri_status {
   LRI_OK = 0,
@@ -63,7 +64,8 @@ int lri_set_gemm_backend(int backend);
  * (LRI_DECODE_SPLITS: 0 choose, 1..64), attn_prefill_tc (LRI_ATTN_PREFILL_TC: 0 mma.sync kernel, 1 tcgen05
  * kernel), gemm_reserve_sms (LRI_GEMM_RESERVE_SMS: SMs
  * the persistent prefill GEMM leaves free for a collective running beside it, 0..64), attn_head_tile
- * (LRI_ATTN_HEAD_TILE: query heads of a KV group per CTA of the cluster decode attention, 0 choose, 1, 2, 4).  Unknown
+ * (LRI_ATTN_HEAD_TILE: query heads of a KV group per CTA of the cluster decode attention, 0 choose, 1, 2, 4),
+ * moe_stream_pairs (LRI_MOE_STREAM_PAIRS: (token, expert) pairs up to which experts run as streaming projections).  Unknown
  * names and values an option does not take return LRI_ERR_ARG.  No counterpart in the reference
  * (its only switches are benchmark.py's command-line flags). */
 int lri_set_option(const char* name, int value);
@@ -113,6 +115,12 @@ int lri_streamk_plan(int64_t M, int N, int K, int* tiles, int* k_tiles, int* max
                      int* token_tile);
 int lri_linear(int dtype, const void* x, const void* w, const void* addend, void* y, int64_t M,
                int N, int K, void* workspace, size_t workspace_bytes, lri_stream_t stream);
+/* y = x W^T with y in fp32, no rounding: projections that feed fp32 arithmetic (norms, gates, recurrences,
+ * routers).  Kernels and workspace as lri_linear.  Both entry points also take LRI_FP32 (then y is fp32 in
+ * either) and any K; those run a plain SIMT kernel.  No counterpart in the reference. */
+size_t lri_linear_f32_workspace_bytes(int64_t M, int N);
+int lri_linear_f32(int dtype, const void* x, const void* w, float* y, int64_t M, int N, int K,
+                   void* workspace, size_t workspace_bytes, lri_stream_t stream);
 
 /* ---- F2: QKV projection + RoPE + KV-cache write ----------------------------------------
  * x [B*S, K]; wqkv [(n_head + 2 n_kv) * head_dim, K] with rows [q heads | k heads | v heads];
@@ -273,6 +281,89 @@ int lri_lm_head_argmax(lri_comm* comm, int dtype, const void* x, const void* w, 
                        int64_t index_offset, int32_t* token_out, void* scratch, size_t scratch_bytes,
                        void* logits_ws, size_t logits_ws_bytes, void* workspace, size_t workspace_bytes,
                        int timeout_ms, lri_stream_t stream);
+/* ==== Layers of designs outside the reference: fp32 residual stream, latent attention, gated recurrence, experts.
+ * All of these take LRI_BF16, LRI_FP16 and LRI_FP32; every size is a parameter. ==== */
+
+/* ---- residual stream in fp32 ----------------------------------------------------------------
+ * y_r   = sum over the row's slots of y[slot]        (slots NULL: rows r * n_slots ...; y has y_rows rows)
+ * t     = sigmoid(gate + gate_bias) * y_r            (gate NULL: t = y_r; gate fp32, row pitch gate_ld)
+ * resid_out = resid + RMSNorm(t) * post_weight       (post_weight NULL: resid + t; resid NULL: 0; may alias)
+ * normed_out = RMSNorm(resid_out) * next_weight      (weight NULL: resid_out; both NULL: none), rounded to `dtype`
+ * RMSNorm(x) = x / sqrt(mean(x^2) + eps), fp32 throughout. */
+int lri_gated_norm_add(int dtype, const float* resid, const void* y, const int32_t* slots, int n_slots,
+                       int64_t y_rows, const float* gate, int64_t gate_ld, const void* gate_bias,
+                       const void* post_weight, float eps, float* resid_out, const void* next_weight,
+                       void* normed_out, int64_t rows, int dim, lri_stream_t stream);
+/* resid_out = table[idx] in fp32, normed_out = RMSNorm(resid_out) * weight. */
+int lri_embed_norm(int dtype, const void* table, const void* idx, int idx_is_i64, int64_t vocab,
+                   float* resid_out, const void* weight, float eps, void* normed_out, int64_t rows, int dim,
+                   lri_stream_t stream);
+
+/* ---- latent attention --------------------------------------------------------------------------
+ * proj [B*S, ld] fp32 holds q (heads of [dim | rot_dim]) at q_off and [latent (rank) | key part (rot_dim)] at
+ * kv_off.  Rotates the rot_dim parts by halves (pair i, i + rot_dim/2) with rope_table [table_rows, rot_dim/2, 2]
+ * (cos, sin; fp32) at the token's position, normalises the latent, and stores q's two parts (pitches in elements)
+ * and the cache row [latent | key part] of cache [B, smax, rank + rot_dim]. */
+int lri_latent_prepare(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t kv_off,
+                       const void* norm_weight, float eps, const float* rope_table, int64_t table_rows,
+                       const void* input_pos, int pos_is_i64, void* qn, int64_t qn_row, int64_t qn_head,
+                       void* qr, int64_t qr_row, int64_t qr_head, void* cache, int64_t smax, int B, int S,
+                       int heads, int dim, int rot_dim, int rank, lri_stream_t stream);
+/* Cache rows of positions input_pos[0] - history .. + rows - 1 of every sequence, split into contiguous
+ * latents [B, rows, rank] and rotated keys [B, rows, rot_dim]; positions below 0 give zeros. */
+int lri_latent_window(int dtype, const void* cache, int64_t smax, int rank, int rot_dim, const void* input_pos,
+                      int pos_is_i64, int B, int history, int rows, void* latent_out, void* k_rot_out,
+                      lri_stream_t stream);
+/* y[row, head] = W[head] x[row, head], W [heads, out, in], or [heads, in, out] when transposed. */
+int lri_head_linear(int dtype, const void* x, int64_t x_row, int64_t x_head, const void* w, int transposed,
+                    void* y, int64_t y_row, int64_t y_head, int64_t rows, int heads, int in, int out,
+                    lri_stream_t stream);
+/* Softmax attention of query (row, head) = [d1 | d2] over the key rows j = [k (d1) | k2 (d2, shared by the heads)]
+ * at positions input_pos[0] - history + j (history < 0: position j) with 0 <= position of the query - position of the key < window_size.
+ * Row j of v has dv elements.  Pitches in elements; a head pitch of 0 shares a row among the heads. */
+int lri_window_attention(int dtype, const void* q, int64_t q_row, int64_t q_head, const void* k, int64_t k_batch,
+                         int64_t k_row, int64_t k_head, const void* k2, int64_t k2_batch, int64_t k2_row,
+                         const void* v, int64_t v_batch, int64_t v_row, int64_t v_head, void* out,
+                         const void* input_pos, int pos_is_i64, int history, int64_t k_rows,
+                         int64_t window_size, float scale, int B, int S, int heads, int d1, int d2, int dv,
+                         lri_stream_t stream);
+
+/* ---- HGRN2 recurrence -----------------------------------------------------------------------------
+ * proj [B*S, ld] fp32 holds q, f, v at the given offsets.  f = lower + (1 - lower) sigmoid(f + f_bias), q = silu(q);
+ * state[c, e] <- f[c] state[c, e] + (1 - f[c]) v[e], o[e] = sum_c q[c] state[c, e] per head, out = RMSNorm over e.
+ * state [B, heads, dim, vdim] fp32 is read and written; a call that starts at position 0 starts from zero. */
+size_t lri_hgrn2_workspace_bytes(int dtype, int B, int S, int heads, int dim, int vdim);
+int lri_hgrn2(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t f_off, int64_t v_off,
+              const void* f_bias, const void* lower, const void* norm_weight, float eps, float* state,
+              const void* input_pos, int pos_is_i64, void* out, int B, int S, int heads, int dim, int vdim,
+              void* workspace, size_t workspace_bytes, lri_stream_t stream);
+
+/* ---- mixture of experts ------------------------------------------------------------------------------
+ * lri_moe_packs: whether a call of this size runs on rows packed by expert (1) or pair by pair (0);
+ * lri_moe_max_tiles: most 128-row tiles the packed form can need. */
+int lri_moe_packs(int dtype, int64_t rows, int top, int dim, int ff);
+int64_t lri_moe_max_tiles(int64_t rows, int top, int experts);
+/* ids, scores [rows, top]: the `top` largest logistic scores of logits [rows, ld] (lowest index on ties).  For the
+ * packed form counts [experts] (zero before the call) and rank [rows * top] are filled too. */
+int lri_moe_route(const float* logits, int64_t ld, int experts, int top, int64_t rows, int32_t* ids,
+                  float* scores, int32_t* counts, int32_t* rank, lri_stream_t stream);
+/* Packs the rows of x by expert into tiles of 128: tiles = {count, expert of each}, packed rows and their scores,
+ * slots [rows * top] = packed row of each pair.  Leaves counts at zero. */
+int lri_moe_pack(int dtype, const void* x, int64_t rows, int dim, int top, int experts, const int32_t* ids,
+                 const float* scores, const int32_t* rank, int32_t* counts, int32_t* first_row, int32_t* tiles,
+                 void* packed, float* row_scale, int32_t* slots, lri_stream_t stream);
+/* hidden = g sigmoid(alpha g) (u + offset), g = min(s gate, limit), u = clamp(s up, -limit, limit) with the score s
+ * of the pair and gate, up the two products with w1 [experts, 2 ff, dim] = [up | gate].  tiles == NULL: x [rows, dim],
+ * hidden [pairs, ff]; else x and hidden are packed rows. */
+int lri_moe_gateup(int dtype, const void* x, const void* w1, void* hidden, const int32_t* ids,
+                   const float* scores, int64_t pairs, int top, const int32_t* tiles, const float* row_scale,
+                   int64_t max_tiles, int experts, int ff, int dim, float alpha, float limit, float offset,
+                   lri_stream_t stream);
+/* y = w2 hidden per pair (or packed row), w2 [experts, dim, ff]; the sum over a token's choices is taken by
+ * lri_gated_norm_add. */
+int lri_moe_down(int dtype, const void* hidden, const void* w2, void* y, const int32_t* ids, int64_t pairs,
+                 const int32_t* tiles, int64_t max_tiles, int experts, int dim, int ff, lri_stream_t stream);
+
 /* Reads (and clears) the device status word: LRI_OK or LRI_ERR_TIMEOUT.  Synchronises `stream`. */
 int lri_comm_status(lri_comm* comm, lri_stream_t stream);
 int lri_comm_destroy(lri_comm* comm);

@@ -63,6 +63,7 @@ enum Option {
   OPT_ATTN_PREFILL_TC,  // LRI_ATTN_PREFILL_TC  0: prefill attention on the mma.sync kernel; 1: tcgen05 / TMEM kernel (default)
   OPT_GEMM_RESERVE_SMS, // LRI_GEMM_RESERVE_SMS  SMs the persistent prefill GEMM leaves free (for a collective running beside it)
   OPT_ATTN_HEAD_TILE,   // LRI_ATTN_HEAD_TILE  query heads per CTA of the cluster decode-attention kernel: 1, 2, 4 (0 = choose)
+  OPT_MOE_STREAM_PAIRS, // LRI_MOE_STREAM_PAIRS  (token, expert) pairs up to which experts run as streaming projections
   OPT_COUNT
 };
 int option(int which);
@@ -142,6 +143,12 @@ struct Num<__half> {
   }
 };
 
+template <>
+struct Num<float> {
+  static __device__ __forceinline__ float to_f(float v) { return v; }
+  static __device__ __forceinline__ float from_f(float f) { return f; }
+};
+
 template <typename T>
 __device__ __forceinline__ void unpack8(const uint4& v, float (&f)[8]) {
   Num<T>::unpack2(v.x, f[0], f[1]);
@@ -215,6 +222,58 @@ __device__ __forceinline__ float exp2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// logistic function in fp32
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+
+// Eight consecutive elements of T as floats / back, 16-byte (fp32: 32-byte) aligned.
+template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&f)[8]) {
+  unpack8<T>(*reinterpret_cast<const uint4*>(p), f);
+}
+template <>
+__device__ __forceinline__ void load8<float>(const float* p, float (&f)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x, f[1] = a.y, f[2] = a.z, f[3] = a.w, f[4] = b.x, f[5] = b.y, f[6] = b.z, f[7] = b.w;
+}
+template <typename T>
+__device__ __forceinline__ void store8(T* p, const float (&f)[8]) {
+  *reinterpret_cast<uint4*>(p) = pack8<T>(f);
+}
+template <>
+__device__ __forceinline__ void store8<float>(float* p, const float (&f)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
+}
+
+// Sum over the CTA, the result in every thread.  `part` is shared memory for one float per warp plus one;
+// consecutive calls may use the same array.
+__device__ __forceinline__ float block_sum(float v, float* part) {
+  const int warps = (blockDim.x + 31) >> 5;
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
+  __syncthreads();
+  if (threadIdx.x < 32) {
+    float t = static_cast<int>(threadIdx.x) < warps ? part[threadIdx.x] : 0.f;
+    t = warp_sum(t);
+    if (threadIdx.x == 0) part[32] = t;
+  }
+  __syncthreads();
+  const float s = part[32];
+  __syncthreads();
+  return s;
+}
+
+// Gated linear unit with clamped inputs: g = min(gate, limit), u = clamp(up, -limit, limit),
+// g * sigmoid(alpha g) * (u + offset), in fp32.
+struct GluParams {
+  float alpha, limit, offset;
+};
+__device__ __forceinline__ float clamped_glu(float gate, float up, const GluParams& p) {
+  const float g = fminf(gate, p.limit);
+  const float u = fminf(fmaxf(up, -p.limit), p.limit);
+  return g * sigmoid_f(p.alpha * g) * (u + p.offset);
 }
 
 // SiLU as torch evaluates it in fp32: x / (1 + exp(-x))

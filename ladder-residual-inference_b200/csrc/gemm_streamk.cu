@@ -223,7 +223,12 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
       const int64_t n = static_cast<int64_t>(tile) * kBM + i;
       if (n >= p.lin.n) continue;
       T* y = static_cast<T*>(p.lin.y) + n;
-      if (EPI == EPI_PLAIN) {
+      if (EPI == EPI_F32) {
+        float* yf = static_cast<float*>(p.lin.y) + n;
+#pragma unroll
+        for (int e = 0; e < BN; ++e)
+          if (e < m) yf[static_cast<int64_t>(e) * p.lin.n] = __uint_as_float(acc[0][e]);
+      } else if (EPI == EPI_PLAIN) {
         const T* add = p.lin.addend ? static_cast<const T*>(p.lin.addend) + n : nullptr;
 #pragma unroll
         for (int e = 0; e < BN; ++e) {
@@ -298,6 +303,10 @@ __global__ void __launch_bounds__(256) streamk_finish_kernel(const StreamKParams
     s0 += v.x;
     s1 += v.y;
   }
+  if (EPI == EPI_F32) {
+    *reinterpret_cast<float2*>(static_cast<float*>(p.lin.y) + static_cast<int64_t>(tok) * p.lin.n + n) = make_float2(s0, s1);
+    return;
+  }
   const float v0 = rnd<T>(s0), v1 = rnd<T>(s1);
   if (EPI == EPI_PLAIN) {
     float o0 = v0, o1 = v1;
@@ -371,6 +380,7 @@ template <typename T, int BN>
 int launch_epi(int dtype, int epi, const LinearParams& lin, float* partial, cudaStream_t st) {
   if (epi == EPI_PLAIN) return launch<T, BN, EPI_PLAIN>(dtype, lin, partial, st);
   if (epi == EPI_SWIGLU) return launch<T, BN, EPI_SWIGLU>(dtype, lin, partial, st);
+  if (epi == EPI_F32) return launch<T, BN, EPI_F32>(dtype, lin, partial, st);
   return launch<T, BN, EPI_QKV>(dtype, lin, partial, st);
 }
 

@@ -38,6 +38,9 @@ struct WorkItem {
 struct GemmGrid {
   int tiles_p, tiles_q;
   int group;  // P tiles per panel
+  // expert tiles: the number of P tiles in use and the weight matrix of each are read from the device
+  const int* tiles;
+  int matrix_rows;
 };
 // Order of the output tiles.  The P tiles are taken in panels of `group`; inside a panel the
 // Q tile is the slow index.  The CTAs that run at the same time then share one panel of P
@@ -68,12 +71,15 @@ __device__ __forceinline__ WorkItem work_item(int item, const GemmGrid& g) {
 //   EPI_SWIGLU  the Q tile is BN/2 up rows followed by the BN/2 matching gate rows of w1, so that a
 //               thread finds up_j and gate_j of its token in the same accumulator row; it stores
 //               silu(gate) * up to h [m, I] (lin.y, lin.n = I)
+//   EPI_GLU     as SWIGLU with the clamped unit, on fp32 accumulators scaled per row (experts)
+//   EPI_F32     stores the fp32 accumulators
 //   EPI_QKV     a thread rotates the 16 adjacent pairs of each 32-column chunk of its token with the
 //               table row of the token's position and stores them to q_out / k-cache / v-cache
 template <typename T, int BN, bool SWAP, int EPI>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_constant__ CUtensorMap tmap_q,
                     T* __restrict__ c, GemmShape shape, GemmGrid grid, int stages, const LinearParams lin) {
+  constexpr bool kGlu = EPI == EPI_SWIGLU || EPI == EPI_GLU;
   extern __shared__ uint8_t smem_raw[];
   constexpr uint32_t kTileP = kBM * kBK * 2;
   constexpr uint32_t kTileQ = BN * kBK * 2;
@@ -89,7 +95,6 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
   const int num_kt = (shape.k + kBK - 1) / kBK;
-  const int items = grid.tiles_p * grid.tiles_q;
 
   const uint32_t full0 = smem_u32(&bars[0]);
   const uint32_t empty0 = smem_u32(&bars[8]);
@@ -122,6 +127,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
   // everything above overlaps the tail of the preceding kernel when launched as its programmatic dependent
   pdl_wait();
   pdl_launch_dependents();
+  if (grid.tiles) {
+    const int used = grid.tiles[0];
+    grid.tiles_p = used < grid.tiles_p ? used : grid.tiles_p;
+  }
+  const int items = grid.tiles_p * grid.tiles_q;
 
   if (warp == 0) {
     if (lane == 0) {
@@ -129,6 +139,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
       bool ok = true;
       for (int item = blockIdx.x; item < items && ok; item += gridDim.x) {
         const WorkItem w = work_item(item, grid);
+        const int row0 = grid.tiles ? grid.tiles[1 + w.tile_p] * grid.matrix_rows : 0;  // first weight row of the tile's matrix
         for (int kt = 0; kt < num_kt; ++kt, ++g) {
           const uint32_t s = g % static_cast<uint32_t>(stages);
           const uint32_t round = g / static_cast<uint32_t>(stages);
@@ -139,11 +150,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
           const uint32_t dst = base + s * kStageBytes;
           const int kx = kt * kBK;
           tma_load_2d(dst, &tmap_p, full0 + 8 * s, kx, w.tile_p * kBM);
-          if (EPI == EPI_SWIGLU) {
-            tma_load_2d(dst + kTileP, &tmap_q, full0 + 8 * s, kx, w.tile_q * (BN / 2));
-            tma_load_2d(dst + kTileP + kTileQ / 2, &tmap_q, full0 + 8 * s, kx, lin.n + w.tile_q * (BN / 2));
+          if (kGlu) {
+            tma_load_2d(dst + kTileP, &tmap_q, full0 + 8 * s, kx, row0 + w.tile_q * (BN / 2));
+            tma_load_2d(dst + kTileP + kTileQ / 2, &tmap_q, full0 + 8 * s, kx, row0 + lin.n + w.tile_q * (BN / 2));
           } else {
-            tma_load_2d(dst + kTileP, &tmap_q, full0 + 8 * s, kx, w.tile_q * BN);
+            tma_load_2d(dst + kTileP, &tmap_q, full0 + 8 * s, kx, row0 + w.tile_q * BN);
           }
         }
       }
@@ -198,8 +209,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
       if (!__all_sync(0xffffffffu, ready)) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t tacc = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + a * kAccCols;
-      if (!SWAP && EPI == EPI_SWIGLU) {
+      if (!SWAP && kGlu) {
         const int64_t row = static_cast<int64_t>(w.tile_p) * kBM + i;
+        const float sc = EPI == EPI_GLU && row < shape.m ? lin.ex.row_scale[row] : 0.f;
 #pragma unroll 1
         for (int cc = 0; cc < BN / 2; cc += 32) {
           uint32_t up[32], gate[32];
@@ -211,7 +223,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
           __align__(16) T out[32];
 #pragma unroll
           for (int e = 0; e < 32; ++e)
-            out[e] = swiglu_rounded<T>(rnd<T>(__uint_as_float(up[e])), rnd<T>(__uint_as_float(gate[e])));
+            out[e] = EPI == EPI_GLU
+                         ? Num<T>::from_f(clamped_glu(sc * __uint_as_float(gate[e]), sc * __uint_as_float(up[e]), lin.ex.glu))
+                         : swiglu_rounded<T>(rnd<T>(__uint_as_float(up[e])), rnd<T>(__uint_as_float(gate[e])));
           if (j0 + 32 <= lin.n && (lin.n & 7) == 0) {
 #pragma unroll
             for (int v = 0; v < 4; ++v) reinterpret_cast<uint4*>(dst)[v] = reinterpret_cast<const uint4*>(out)[v];
@@ -284,7 +298,20 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
         if (!SWAP) {
           const int64_t row = static_cast<int64_t>(w.tile_p) * kBM + i;
           const int64_t col0 = static_cast<int64_t>(w.tile_q) * BN + cc;
-          if (row < shape.m) {
+          if (EPI == EPI_F32) {
+            float* dst = static_cast<float*>(lin.y) + row * shape.n + col0;
+            if (row < shape.m) {
+              if (col0 + kValid <= shape.n) {
+#pragma unroll
+                for (int v = 0; v < kValid / 4; ++v)
+                  reinterpret_cast<uint4*>(dst)[v] = make_uint4(r[v * 4], r[v * 4 + 1], r[v * 4 + 2], r[v * 4 + 3]);
+              } else {
+#pragma unroll
+                for (int e = 0; e < kValid; ++e)
+                  if (col0 + e < shape.n) dst[e] = __uint_as_float(r[e]);
+              }
+            }
+          } else if (row < shape.m) {
             T* dst = c + row * shape.n + col0;
             if (col0 + kValid <= shape.n) {
 #pragma unroll
@@ -305,8 +332,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
           const int64_t tok0 = static_cast<int64_t>(w.tile_q) * BN + cc;
           if (n < shape.n) {
 #pragma unroll
-            for (int e = 0; e < kValid; ++e)
-              if (tok0 + e < shape.m) c[(tok0 + e) * shape.n + n] = Num<T>::from_f(__uint_as_float(r[e]));
+            for (int e = 0; e < kValid; ++e) {
+              if (tok0 + e >= shape.m) continue;
+              if (EPI == EPI_F32)
+                static_cast<float*>(lin.y)[(tok0 + e) * shape.n + n] = __uint_as_float(r[e]);
+              else
+                c[(tok0 + e) * shape.n + n] = Num<T>::from_f(__uint_as_float(r[e]));
+            }
           }
         }
       }
@@ -368,7 +400,9 @@ namespace {
 
 template <typename T, int BN, bool SWAP, int EPI = EPI_PLAIN>
 int launch_tile(int dtype, const void* a, const void* w, void* c, int64_t m, int n, int k, cudaStream_t st,
-                const LinearParams* lin = nullptr) {
+                 const LinearParams* lin = nullptr, int expert_tiles = 0) {
+  // expert_tiles > 0: at most that many tiles of rows, each with its own weight matrix (lin->ex); n = rows of one matrix
+  constexpr bool kGlu = EPI == EPI_SWIGLU || EPI == EPI_GLU;
   CUtensorMap tp, tq;
   const void* p_ptr = SWAP ? w : a;
   const void* q_ptr = SWAP ? a : w;
@@ -376,7 +410,7 @@ int launch_tile(int dtype, const void* a, const void* w, void* c, int64_t m, int
   const int64_t q_rows = SWAP ? m : n;
   int rc = make_tmap(&tp, dtype, p_ptr, p_rows, k, kBM);
   if (rc != LRI_OK) return rc;
-  rc = make_tmap(&tq, dtype, q_ptr, q_rows, k, EPI == EPI_SWIGLU ? BN / 2 : BN);
+  rc = make_tmap(&tq, dtype, q_ptr, expert_tiles > 0 ? lin->ex.pairs * lin->ex.matrix_rows : q_rows, k, kGlu ? BN / 2 : BN);
   if (rc != LRI_OK) return rc;
   constexpr int kStageBytes = (kBM + BN) * kBK * 2;
   int stages = kSmemBudget / kStageBytes;
@@ -385,9 +419,9 @@ int launch_tile(int dtype, const void* a, const void* w, void* c, int64_t m, int
   auto kern = gemm_tcgen05_kernel<T, BN, SWAP, EPI>;
   static std::atomic<unsigned long long> attr_set{0};  // per template instantiation, one bit per device
   LRI_ONCE_PER_DEVICE(attr_set, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBudget + 1024));
-  const int64_t tiles_p = (p_rows + kBM - 1) / kBM;
+  const int64_t tiles_p = expert_tiles > 0 ? expert_tiles : (p_rows + kBM - 1) / kBM;
   // SWIGLU: a Q tile is BN/2 outputs (their up rows and their gate rows)
-  const int64_t tiles_q = EPI == EPI_SWIGLU ? (lin->n + BN / 2 - 1) / (BN / 2) : (q_rows + BN - 1) / BN;
+  const int64_t tiles_q = kGlu ? (lin->n + BN / 2 - 1) / (BN / 2) : (q_rows + BN - 1) / BN;
   const int64_t items = tiles_p * tiles_q;
   if (items >= (1ll << 31)) return fail(LRI_ERR_UNSUPPORTED, "gemm: %lld output tiles", (long long)items);
   // panel of P tiles: about 16 MB of the P operand, between 4 and 16 tiles (LRI_GEMM_GROUP overrides)
@@ -396,7 +430,8 @@ int launch_tile(int dtype, const void* a, const void* w, void* c, int64_t m, int
   group = group < 4 ? 4 : (group > 16 ? 16 : group);
   if (forced_group > 0) group = forced_group;
   group = group > tiles_p ? tiles_p : group;
-  GemmGrid grid{static_cast<int>(tiles_p), static_cast<int>(tiles_q), static_cast<int>(group)};
+  GemmGrid grid{static_cast<int>(tiles_p), static_cast<int>(tiles_q), static_cast<int>(group),
+                expert_tiles > 0 ? lin->ex.tiles : nullptr, expert_tiles > 0 ? static_cast<int>(lin->ex.matrix_rows) : 0};
   GemmShape shape{static_cast<int>(m), n, k};
   // one persistent CTA per SM, minus the SMs left to a collective that runs beside the GEMM (the all-reduce
   // of the previous sublayer in the ladder schedule: a kernel that owns every SM would keep it waiting)
@@ -422,6 +457,34 @@ int launch_typed(int dtype, const void* a, const void* w, void* c, int64_t m, in
   const int64_t cost256 = ((t256 + sms - 1) / sms) * 110, cost128 = ((t128 + sms - 1) / sms) * 100;
   if (cost256 <= cost128) return launch_tile<T, 256, false>(dtype, a, w, c, m, n, k, st);
   return launch_tile<T, 128, false>(dtype, a, w, c, m, n, k, st);
+}
+
+template <typename T>
+int launch_f32(int dtype, const void* a, const void* w, float* c, int64_t m, int n, int k, cudaStream_t st) {
+  LinearParams p{};
+  p.y = c;
+  if (m <= 16) return launch_tile<T, 16, true, EPI_F32>(dtype, a, w, nullptr, m, n, k, st, &p);
+  if (m <= 32) return launch_tile<T, 32, true, EPI_F32>(dtype, a, w, nullptr, m, n, k, st, &p);
+  if (m <= 64) return launch_tile<T, 64, true, EPI_F32>(dtype, a, w, nullptr, m, n, k, st, &p);
+  const int sms = sm_count();
+  const int64_t mt = (m + kBM - 1) / kBM;
+  const int64_t t256 = mt * ((n + 255) / 256), t128 = mt * ((n + 127) / 128);
+  const int64_t cost256 = ((t256 + sms - 1) / sms) * 110, cost128 = ((t128 + sms - 1) / sms) * 100;
+  if (cost256 <= cost128) return launch_tile<T, 256, false, EPI_F32>(dtype, a, w, nullptr, m, n, k, st, &p);
+  return launch_tile<T, 128, false, EPI_F32>(dtype, a, w, nullptr, m, n, k, st, &p);
+}
+
+// expert tiles: p.ex.pairs = number of experts
+template <typename T, int EPI>
+int launch_experts(int dtype, const LinearParams& p, int max_tiles, cudaStream_t st) {
+  const int per256 = EPI == EPI_GLU ? 128 : 256, per128 = EPI == EPI_GLU ? 64 : 128;  // outputs per Q tile
+  const int64_t t256 = static_cast<int64_t>(max_tiles) * ((p.n + per256 - 1) / per256);
+  const int64_t t128 = static_cast<int64_t>(max_tiles) * ((p.n + per128 - 1) / per128);
+  const int sms = sm_count();
+  const int64_t cost256 = ((t256 + sms - 1) / sms) * 110, cost128 = ((t128 + sms - 1) / sms) * 100;
+  const int n_rows = EPI == EPI_GLU ? 2 * p.n : p.n;
+  if (cost256 <= cost128) return launch_tile<T, 256, false, EPI>(dtype, p.x, p.w, p.y, p.m, n_rows, p.k, st, &p, max_tiles);
+  return launch_tile<T, 128, false, EPI>(dtype, p.x, p.w, p.y, p.m, n_rows, p.k, st, &p, max_tiles);
 }
 
 // prefill with the epilogue fused: the same tile choice, counted in output tiles
@@ -461,6 +524,26 @@ int gemm_tcgen05_fused_launch(int dtype, int epi, const LinearParams& p, int64_t
 
 bool gemm_tcgen05_supports(int64_t m, int n, int k) {
   return m >= 1 && m < (1ll << 31) && n >= 8 && n % 8 == 0 && k >= 8 && k % 8 == 0;
+}
+
+int gemm_tcgen05_f32_launch(int dtype, const void* a, const void* w, float* c, int64_t m, int n, int k, cudaStream_t st) {
+  return dtype == LRI_BF16 ? launch_f32<__nv_bfloat16>(dtype, a, w, c, m, n, k, st)
+                           : launch_f32<__half>(dtype, a, w, c, m, n, k, st);
+}
+
+bool gemm_tcgen05_experts_supports(int epi, const LinearParams& p) {
+  const int64_t rows = p.ex.pairs * p.ex.matrix_rows;
+  return (epi == EPI_GLU || epi == EPI_PLAIN) && gemm_tcgen05_supports(p.m, p.n, p.k) && rows < (1ll << 31) &&
+         aligned16(p.x) && aligned16(p.w) && aligned16(p.y);
+}
+int gemm_tcgen05_experts_launch(int dtype, int epi, const LinearParams& p, int max_tiles, cudaStream_t st) {
+  if (!gemm_tcgen05_experts_supports(epi, p) || p.ex.tiles == nullptr || max_tiles < 1)
+    return fail(LRI_ERR_ARG, "gemm: expert tiles not available for this shape");
+  if (epi == EPI_GLU)
+    return dtype == LRI_BF16 ? launch_experts<__nv_bfloat16, EPI_GLU>(dtype, p, max_tiles, st)
+                             : launch_experts<__half, EPI_GLU>(dtype, p, max_tiles, st);
+  return dtype == LRI_BF16 ? launch_experts<__nv_bfloat16, EPI_PLAIN>(dtype, p, max_tiles, st)
+                           : launch_experts<__half, EPI_PLAIN>(dtype, p, max_tiles, st);
 }
 
 int gemm_tcgen05_launch(int dtype, const void* a, const void* w, void* c, int64_t m, int n, int k, cudaStream_t st) {

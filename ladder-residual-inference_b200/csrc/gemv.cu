@@ -7,6 +7,8 @@
 // through shared memory; the few threads holding the final sums run the fused epilogue:
 //   PLAIN   store (optionally + addend)                       wo / w2 / LM head
 //   SWIGLU  rows (j, I + j) -> silu(gate) * up                 w1
+//   F32     store the fp32 sums                                 projections that feed fp32 arithmetic
+//   GLU     as SWIGLU with the clamped unit of an expert         one (token, expert) pair per grid.y slice
 //   QKV     rotate adjacent pairs, scatter q / k-cache / v-cache   wqkv
 //   ARGMAX  no logits stored: arg-max over rows and ranks           LM head, greedy decoding (argmax.cuh)
 #include <cstdlib>
@@ -27,13 +29,22 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
   const int K = p.k;
   const T* __restrict__ w = static_cast<const T*>(p.w);
   const T* __restrict__ x = static_cast<const T*>(p.x);
+  constexpr bool kPairs = M == 1 && (EPI == EPI_GLU || EPI == EPI_PLAIN);  // forms that take expert weights
+  const int64_t pair = blockIdx.y;
+  if (kPairs && p.ex.pairs > 0) {
+    // the matrix is chosen by the preceding kernels: nothing can be streamed before they are done
+    pdl_launch_dependents();
+    pdl_wait();
+    w += static_cast<int64_t>(p.ex.experts[pair]) * p.ex.matrix_rows * K;
+    x += (pair / p.ex.rows_per_input) * K;
+  }
 
   // weight rows of this CTA (clamped: rows past the end recompute the last row and are not stored)
   const T* wrow[R];
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     int64_t row;
-    if (EPI == EPI_SWIGLU) {
+    if (EPI == EPI_SWIGLU || EPI == EPI_GLU) {
       int64_t j = static_cast<int64_t>(blockIdx.x) * (R / 2) + (r >> 1);
       j = j < p.n ? j : p.n - 1;
       row = (r & 1) ? p.n + j : j;  // even slot: up row j, odd slot: gate row I + j
@@ -68,8 +79,10 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
   // begin its own prologue, and only then wait for the activations to be complete.
   int c0 = warp;
   load_w(c0);
-  pdl_launch_dependents();
-  pdl_wait();
+  if (!kPairs || p.ex.pairs == 0) {
+    pdl_launch_dependents();
+    pdl_wait();
+  }
   while (true) {
     uint4 xv[U][M];
 #pragma unroll
@@ -147,12 +160,25 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
     s0 += red[wi][m * R + 2 * j];
     s1 += red[wi][m * R + 2 * j + 1];
   }
+  if (EPI == EPI_F32) {
+    const int64_t n = static_cast<int64_t>(blockIdx.x) * R + 2 * j;
+    float* y = static_cast<float*>(p.y) + static_cast<int64_t>(m) * p.n;
+    if (n < p.n) y[n] = s0;
+    if (n + 1 < p.n) y[n + 1] = s1;
+    return;
+  }
+  if (EPI == EPI_GLU) {
+    const int64_t jj = static_cast<int64_t>(blockIdx.x) * (R / 2) + j;
+    const float sc = p.ex.row_scale[pair];
+    if (jj < p.n) static_cast<T*>(p.y)[pair * p.n + jj] = Num<T>::from_f(clamped_glu(sc * s1, sc * s0, p.ex.glu));
+    return;
+  }
   // the projection's own rounding to the storage type (nn.Linear output)
   const float v0 = rnd<T>(s0), v1 = rnd<T>(s1);
 
   if (EPI == EPI_PLAIN) {
     const int64_t n = static_cast<int64_t>(blockIdx.x) * R + 2 * j;
-    T* y = static_cast<T*>(p.y) + static_cast<int64_t>(m) * p.n;
+    T* y = static_cast<T*>(p.y) + (kPairs && p.ex.pairs > 0 ? pair : static_cast<int64_t>(m)) * p.n;
     const T* add = p.addend ? static_cast<const T*>(p.addend) + static_cast<int64_t>(m) * p.n : nullptr;
     const float o0 = n < p.n ? rnd<T>(add ? v0 + Num<T>::to_f(add[n]) : v0) : 0.f;
     const float o1 = n + 1 < p.n ? rnd<T>(add ? v1 + Num<T>::to_f(add[n + 1]) : v1) : 0.f;
@@ -186,9 +212,10 @@ int launch_gemv(const LinearParams& p, cudaStream_t st) {
   const int nchunks = (p.k + 255) >> 8;
   int W = (nchunks + U - 1) / U;
   W = W < 1 ? 1 : (W > kGemvMaxWarps ? kGemvMaxWarps : W);
-  const int64_t per_cta = EPI == EPI_SWIGLU ? R / 2 : R;
+  const int64_t per_cta = EPI == EPI_SWIGLU || EPI == EPI_GLU ? R / 2 : R;
   const int64_t grid = (p.n + per_cta - 1) / per_cta;
-  LRI_CUDA(launch_pdl(gemv_kernel<T, M, R, U, EPI>, dim3(static_cast<unsigned>(grid)), dim3(W * 32), 0, st, p));
+  const unsigned pairs = p.ex.pairs > 0 ? static_cast<unsigned>(p.ex.pairs) : 1u;
+  LRI_CUDA(launch_pdl(gemv_kernel<T, M, R, U, EPI>, dim3(static_cast<unsigned>(grid), pairs), dim3(W * 32), 0, st, p));
   LRI_LAUNCH_CHECK("gemv_kernel");
   return LRI_OK;
 }
@@ -234,6 +261,11 @@ int dispatch_epi(int epi, const LinearParams& p, cudaStream_t st) {
     case EPI_PLAIN: return dispatch_m<T, EPI_PLAIN>(p, st);
     case EPI_SWIGLU: return dispatch_m<T, EPI_SWIGLU>(p, st);
     case EPI_ARGMAX: return dispatch_m<T, EPI_ARGMAX>(p, st);
+    case EPI_F32: return dispatch_m<T, EPI_F32>(p, st);
+    case EPI_GLU: {  // one row per expert pair
+      if (rows_per_cta(p) == 8) return launch_gemv<T, 1, 8, 2, EPI_GLU>(p, st);
+      return launch_gemv<T, 1, 4, 4, EPI_GLU>(p, st);
+    }
     default: return dispatch_m<T, EPI_QKV>(p, st);
   }
 }

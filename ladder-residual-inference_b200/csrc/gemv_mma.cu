@@ -166,6 +166,13 @@ __global__ void __launch_bounds__(kMmaMaxWarps * 32) gemv_mma_kernel(const Linea
       for (int q = 0; q < 2; ++q) {
         const int tok = t * 8 + 2 * c + q;
         if (tok >= p.m) continue;
+        if (EPI == EPI_F32) {
+          const int64_t n = (static_cast<int64_t>(blockIdx.x) * MT + mt) * 16 + 2 * a;
+          float* y = static_cast<float*>(p.y) + static_cast<int64_t>(tok) * p.n;
+          if (n < p.n) y[n] = fin[t][q];
+          if (n + 1 < p.n) y[n + 1] = fin[t][2 + q];
+          continue;
+        }
         const float v0 = rnd<T>(fin[t][q]);      // row0 of this thread
         const float v1 = rnd<T>(fin[t][2 + q]);  // row1
         if (EPI == EPI_SWIGLU) {
@@ -218,6 +225,7 @@ int dispatch(int epi, const LinearParams& p, cudaStream_t st) {
   const bool one = p.m <= 8;
   switch (epi) {
     case EPI_PLAIN: return one ? launch_tiles<T, 1, EPI_PLAIN>(p, st) : launch_tiles<T, 2, EPI_PLAIN>(p, st);
+    case EPI_F32: return one ? launch_tiles<T, 1, EPI_F32>(p, st) : launch_tiles<T, 2, EPI_F32>(p, st);
     case EPI_SWIGLU: return one ? launch_tiles<T, 1, EPI_SWIGLU>(p, st) : launch_tiles<T, 2, EPI_SWIGLU>(p, st);
     default: return one ? launch_tiles<T, 1, EPI_QKV>(p, st) : launch_tiles<T, 2, EPI_QKV>(p, st);
   }

@@ -6,7 +6,9 @@
 
 namespace lri {
 
-enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_QKV = 2, EPI_ARGMAX = 3 };
+// EPI_F32: like PLAIN with an fp32 output (no rounding, no addend).  EPI_GLU: like SWIGLU (weight rows [up | gate])
+// with the clamped gated linear unit in fp32 and a scale per input row (mixture-of-experts feed-forward).
+enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_QKV = 2, EPI_ARGMAX = 3, EPI_F32 = 4, EPI_GLU = 5 };
 constexpr int kGemvMaxRows = 8;
 
 // Producer side of the split all-reduce, fused into the epilogue of a row-parallel projection:
@@ -19,6 +21,19 @@ struct PushArgs {
   size_t region_off;              // offset of the channel's line region inside an inbox
   int64_t slot_bytes;             // bytes of one (buffer, source rank) slot
   int world, rank, enabled;
+};
+
+// Mixture of experts: the weight matrix of a row (or of a tile of rows) is chosen on the device.
+//   pairs > 0  streaming kernel, one (token, choice) pair per grid.y slice: matrix experts[pair], input row
+//              pair / rows_per_input, output row pair
+//   tiles      tcgen05 kernel: tiles[0] = number of 128-row tiles in use, tiles[1 + t] = matrix of tile t
+struct ExpertArgs {
+  const int* experts;
+  int pairs, rows_per_input;
+  const int* tiles;
+  int64_t matrix_rows;     // weight rows of one expert
+  const float* row_scale;  // GLU epilogue: factor on the input of a pair (or of a row of the tiled input)
+  GluParams glu;
 };
 
 struct LinearParams {
@@ -38,6 +53,7 @@ struct LinearParams {
   int64_t smax, table_rows;
   int table_gathered;  // rope_table row s belongs to token s (rows already gathered by position)
   PushArgs push;       // PLAIN epilogue of the SIMT kernel only
+  ExpertArgs ex;       // expert weights chosen on the device
   ArgmaxArgs am;       // ARGMAX epilogue of the SIMT kernel: greedy choice instead of stored logits
 };
 
@@ -91,6 +107,18 @@ inline int streaming_launch(int dtype, int epi, const LinearParams& p, cudaStrea
   return gemv_mma_launch(dtype, epi, p, st);
 }
 bool prefer_simt_gemv();
+
+// Any shape, alignment and storage type (fp32 included), SIMT fp32 arithmetic: y = x W^T with y in the storage
+// type or, out_f32, in fp32; addend may be NULL (linear_generic.cu).
+int gemm_generic_launch(int dtype, const void* x, const void* w, const void* addend, void* y, bool out_f32, int64_t m,
+                        int n, int k, cudaStream_t st);
+
+// tcgen05 GEMM over tiles of rows that each use one expert's matrix; p.m = rows of the tiled input (a multiple
+// of 128), p.n outputs (GLU: hidden size), p.ex.tiles set, max_tiles = upper bound of tiles[0].
+bool gemm_tcgen05_experts_supports(int epi, const LinearParams& p);
+int gemm_tcgen05_experts_launch(int dtype, int epi, const LinearParams& p, int max_tiles, cudaStream_t st);
+// fp32 output of the plain tcgen05 GEMM
+int gemm_tcgen05_f32_launch(int dtype, const void* a, const void* w, float* c, int64_t m, int n, int k, cudaStream_t st);
 
 // C[m, n] = A[m, k] * W[n, k]^T, C in `dtype`, any m.  backend: lri_gemm_backend.
 int gemm_launch(int dtype, const void* a, const void* w, void* c, int64_t m, int n, int k, cudaStream_t st);

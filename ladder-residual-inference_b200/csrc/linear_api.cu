@@ -45,6 +45,7 @@ const OptionSpec kOptionSpecs[OPT_COUNT] = {
     {"attn_prefill_tc", "LRI_ATTN_PREFILL_TC", 1, 0, 1},
     {"gemm_reserve_sms", "LRI_GEMM_RESERVE_SMS", 0, 0, 64},
     {"attn_head_tile", "LRI_ATTN_HEAD_TILE", 0, 0, 4},
+    {"moe_stream_pairs", "LRI_MOE_STREAM_PAIRS", 32, 0, 65535},
 };
 
 bool option_value_ok(int which, int v) {
@@ -346,6 +347,12 @@ static int check_common(const char* who, int dtype, const void* x, const void* w
 
 extern "C" int lri_linear(int dtype, const void* x, const void* w, const void* addend, void* y, int64_t M, int N,
                           int K, void* workspace, size_t workspace_bytes, lri_stream_t stream) {
+  if (dtype == LRI_FP32 || (K > 0 && K % 8 != 0)) {
+    LRI_REQUIRE(dtype >= LRI_BF16 && dtype <= LRI_FP32, LRI_ERR_UNSUPPORTED, "linear: dtype %d", dtype);
+    LRI_REQUIRE(x && w && y, LRI_ERR_ARG, "linear: NULL pointer");
+    LRI_REQUIRE(M >= 0 && N > 0 && K > 0, LRI_ERR_ARG, "linear: M=%lld N=%d K=%d", (long long)M, N, K);
+    return M == 0 ? LRI_OK : gemm_generic_launch(dtype, x, w, addend, y, false, M, N, K, static_cast<cudaStream_t>(stream));
+  }
   int rc = check_common("linear", dtype, x, w, M, K);
   if (rc != LRI_OK) return rc;
   LRI_REQUIRE(y != nullptr && N > 0, LRI_ERR_ARG, "linear: y is NULL or N=%d", N);
@@ -372,6 +379,30 @@ extern "C" int lri_linear(int dtype, const void* x, const void* w, const void* a
   LRI_REQUIRE((M * N) % 8 == 0 && aligned16(y) && aligned16(addend), LRI_ERR_ALIGN,
               "linear: addend path needs M*N %% 8 == 0 and 16-byte aligned y, addend");
   return add_rows_launch(dtype, y, addend, M * N, st);
+}
+
+extern "C" size_t lri_linear_f32_workspace_bytes(int64_t M, int N) {
+  return M < 0 || N <= 0 ? 0 : streamk_bytes(EPI_F32, M, N);
+}
+
+extern "C" int lri_linear_f32(int dtype, const void* x, const void* w, float* y, int64_t M, int N, int K, void* workspace,
+                              size_t workspace_bytes, lri_stream_t stream) {
+  LRI_REQUIRE(dtype >= LRI_BF16 && dtype <= LRI_FP32, LRI_ERR_UNSUPPORTED, "linear_f32: dtype %d", dtype);
+  LRI_REQUIRE(x && w && y, LRI_ERR_ARG, "linear_f32: NULL pointer");
+  LRI_REQUIRE(M >= 0 && M < (1ll << 31) && N > 0 && K > 0, LRI_ERR_ARG, "linear_f32: M=%lld N=%d K=%d", (long long)M, N, K);
+  if (M == 0) return LRI_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dtype == LRI_FP32 || K % 8 != 0 || !aligned16(x) || !aligned16(w))
+    return gemm_generic_launch(dtype, x, w, nullptr, y, true, M, N, K, st);
+  LinearParams p{};
+  p.x = x, p.w = w, p.y = y, p.m = static_cast<int>(M), p.n = N, p.k = K;
+  if (M <= streaming_rows()) return streaming_launch(dtype, EPI_F32, p, st, prefer_simt_gemv());
+  if (streamk_rows(M) && gemm_streamk_supports(EPI_F32, p, workspace, workspace_bytes))
+    return gemm_streamk_launch(dtype, EPI_F32, p, workspace, workspace_bytes, st);
+  if (M <= kGemvMmaMaxRows) return streaming_launch(dtype, EPI_F32, p, st, prefer_simt_gemv());
+  if (current_gemm_backend() != LRI_GEMM_SIMT && N % 8 == 0 && aligned16(y))
+    return gemm_tcgen05_f32_launch(dtype, x, w, y, M, N, K, st);
+  return gemm_generic_launch(dtype, x, w, nullptr, y, true, M, N, K, st);
 }
 
 extern "C" int lri_streamk_plan(int64_t M, int N, int K, int* tiles, int* k_tiles, int* max_segments, int* ctas,

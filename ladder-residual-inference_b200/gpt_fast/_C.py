@@ -69,6 +69,35 @@ _SIGNATURES = {
     "lri_lm_head_argmax_scratch_bytes": (c_size_t, []),
     "lri_lm_head_argmax": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int64, c_void_p, c_void_p,
                                    c_size_t, c_void_p, c_size_t, c_void_p, c_size_t, c_int, c_void_p]),
+    "lri_linear_f32_workspace_bytes": (c_size_t, [c_int64, c_int]),
+    "lri_linear_f32": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p, c_size_t, c_void_p]),
+    "lri_gated_norm_add": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int64, c_void_p, c_int64, c_void_p,
+                                   c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_void_p]),
+    "lri_embed_norm": (c_int, [c_int, c_void_p, c_void_p, c_int, c_int64, c_void_p, c_void_p, c_float, c_void_p, c_int64,
+                               c_int, c_void_p]),
+    "lri_latent_prepare": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_void_p, c_float, c_void_p, c_int64,
+                                   c_void_p, c_int, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, c_void_p,
+                                   c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_latent_window": (c_int, [c_int, c_void_p, c_int64, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
+                                  c_void_p, c_void_p]),
+    "lri_head_linear": (c_int, [c_int, c_void_p, c_int64, c_int64, c_void_p, c_int, c_void_p, c_int64, c_int64, c_int64,
+                                c_int, c_int, c_int, c_void_p]),
+    "lri_window_attention": (c_int, [c_int, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, c_int64, c_void_p,
+                                     c_int64, c_int64, c_void_p, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_int,
+                                     c_int, c_int64, c_int64, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_hgrn2_workspace_bytes": (c_size_t, [c_int, c_int, c_int, c_int, c_int, c_int]),
+    "lri_hgrn2": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_float,
+                          c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_size_t,
+                          c_void_p]),
+    "lri_moe_packs": (c_int, [c_int, c_int64, c_int, c_int, c_int]),
+    "lri_moe_max_tiles": (c_int64, [c_int64, c_int, c_int]),
+    "lri_moe_route": (c_int, [c_void_p, c_int64, c_int, c_int, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
+    "lri_moe_pack": (c_int, [c_int, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
+    "lri_moe_gateup": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_void_p, c_void_p,
+                               c_int64, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p]),
+    "lri_moe_down": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int,
+                             c_void_p]),
     "lri_comm_status": (c_int, [c_void_p, c_void_p]),
     "lri_comm_destroy": (c_int, [c_void_p]),
 }
@@ -80,7 +109,7 @@ for _name, (_res, _args) in _SIGNATURES.items():
 
 EXPORTED_SYMBOLS = tuple(_SIGNATURES)
 
-BF16, FP16 = 0, 1
+BF16, FP16, FP32 = 0, 1, 2
 GEMM_AUTO, GEMM_TCGEN05, GEMM_SIMT = 0, 1, 2
 
 
@@ -90,6 +119,11 @@ def dtype_code(dtype: torch.dtype) -> int:
     if dtype == torch.float16:
         return FP16
     raise TypeError(f"the sm_100a kernels take bfloat16 or float16 tensors, not {dtype}")
+
+
+def dtype_code_any(dtype: torch.dtype) -> int:
+    """dtype_code for the entry points that also run in fp32."""
+    return FP32 if dtype == torch.float32 else dtype_code(dtype)
 
 
 def check(status: int) -> None:

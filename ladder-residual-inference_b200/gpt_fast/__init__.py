@@ -7,6 +7,7 @@ from .gpt_dense_TP import GPTDense
 from .gpt_desync_TP import GPTDesync
 from .gpt_ladder_TP import GPTLadder
 from .gpt_parallel_TP import GPTParallel
+from .gpt_patevik_TP import GPTPatevik
 from .tp import maybe_init_dist
 
-__all__ = ["GPTDense", "GPTDesync", "GPTLadder", "GPTParallel", "maybe_init_dist"]
+__all__ = ["GPTDense", "GPTDesync", "GPTLadder", "GPTParallel", "GPTPatevik", "maybe_init_dist"]

@@ -50,7 +50,7 @@ class Engine:
         cfg, t = self.cfg, self.comm.world
         self.nh, self.nkv, self.hd = cfg.n_head // t, cfg.n_local_heads // t, cfg.head_dim
         self.inter = cfg.intermediate_size // t
-        self.d = cfg.dim
+        self.d, self.dtype = cfg.dim, dtype
         self.max_batch, self.max_seq = max_batch, max_seq
         rows = max_batch * max_seq
         self.max_rows = rows
@@ -74,22 +74,9 @@ class Engine:
         # wo and w2 may run at the same time on two streams: one workspace each (w2's also serves the LM head)
         self.ws_wo = workspace(self.ops.linear_workspace_bytes, self.d)
         self.ws_w2 = workspace(self.ops.linear_workspace_bytes, self.d)
-        self.ws_head = workspace(self.ops.linear_workspace_bytes, cfg.vocab_size)
-        # vocabulary-parallel greedy head (decode_greedy): this rank's slice of the output rows
-        self.vocab_per_rank = -(-cfg.vocab_size // (8 * t)) * 8
-        self.vocab_lo = min(cfg.vocab_size, self.comm.rank * self.vocab_per_rank)
-        self.vocab_hi = min(cfg.vocab_size, self.vocab_lo + self.vocab_per_rank)
-        self.head_logits = torch.empty(max_batch * self.vocab_per_rank, dtype=dtype, device=device)
-        self.head_best = torch.empty(t, max_batch, 2, dtype=torch.float32, device=device)
-        # fused greedy head (projection + arg-max over rows and ranks in one launch): needs peer memory
-        # for the exchange, i.e. one rank or the P2P communicator; NCCL-only groups use the torch ops below
-        self.head_tokens = torch.zeros(max_batch, dtype=torch.int32, device=device)
-        self.fused_head = hasattr(self.ops, "lm_head_argmax") and self.resid.is_cuda and max_batch <= 64 and \
-            (t == 1 or getattr(self.comm, "handle", None) is not None)
-        if self.fused_head:
-            self.head_scratch = torch.zeros(self.ops.lm_head_argmax_scratch_bytes(), dtype=torch.uint8, device=device)
         nbytes = self.ops.attn_decode_scratch_bytes(max_batch, self.nh, self.nkv, self.hd, _MAX_SPLITS)
         self.scratch = torch.zeros(max(nbytes, 16), dtype=torch.uint8, device=device)
+        self._setup_head(max_batch, device, dtype)
         # ladder decode runs the attention and MLP chains of a layer on two streams (LRI_LADDER_OVERLAP=0: one)
         self.overlap_sublayers = (self.family == "ladder" and self.resid.is_cuda and
                                   os.environ.get("LRI_LADDER_OVERLAP", "1") != "0")
@@ -100,6 +87,27 @@ class Engine:
             self.side_stream = torch.cuda.Stream()
             self._events = [torch.cuda.Event() for _ in range(2 * cfg.n_layer + 2)]
         self.ready = True
+
+    def _setup_head(self, max_batch, device, dtype):
+        """Buffers of the output projection and of the token choice."""
+        cfg, t = self.cfg, self.comm.world
+        n = max(self.ops.linear_workspace_bytes(self.max_rows, cfg.vocab_size),
+                self.ops.linear_workspace_bytes(min(self.max_rows, 64), cfg.vocab_size))
+        self.ws_head = torch.empty(n, dtype=torch.uint8, device=device) if n else None
+        # vocabulary-parallel greedy head (decode_greedy): this rank's slice of the output rows
+        self.vocab_per_rank = -(-cfg.vocab_size // (8 * t)) * 8
+        self.vocab_lo = min(cfg.vocab_size, self.comm.rank * self.vocab_per_rank)
+        self.vocab_hi = min(cfg.vocab_size, self.vocab_lo + self.vocab_per_rank)
+        self.head_logits = torch.empty(max_batch * self.vocab_per_rank, dtype=dtype, device=device)
+        self.head_best = torch.empty(t, max_batch, 2, dtype=torch.float32, device=device)
+        # fused greedy head (projection + arg-max over rows and ranks in one launch): needs peer memory
+        # for the exchange, i.e. one rank or the P2P communicator; NCCL-only groups use the torch ops below
+        self.head_tokens = torch.zeros(max_batch, dtype=torch.int32, device=device)
+        self.fused_head = hasattr(self.ops, "lm_head_argmax") and self.resid.is_cuda and max_batch <= 64 and \
+            dtype in (torch.bfloat16, torch.float16) and cfg.dim % 8 == 0 and \
+            (t == 1 or getattr(self.comm, "handle", None) is not None)
+        if self.fused_head:
+            self.head_scratch = torch.zeros(self.ops.lm_head_argmax_scratch_bytes(), dtype=torch.uint8, device=device)
 
     # ------------------------------------------------------------------------------------------
     def _attention(self, att, w_qkv, rows, B, S, pos, out, push=0):
@@ -164,15 +172,19 @@ class Engine:
         if input_pos.dtype not in (torch.int32, torch.int64):
             input_pos = input_pos.to(torch.int64)
         rows = B * S
+        self._body(idx, rows, B, S, input_pos)
+        return B, S, rows
+
+    def _body(self, idx, rows, B, S, input_pos):
+        """Embedding, layers and final norm; leaves the normalised hidden states in self.normed."""
         self._splits = decode_splits(B, self.nh, self.nkv, self.model.max_seq_length, self.hd) if S == 1 else 1
         self.ops.embedding(self.model.tok_embeddings.weight, idx, self.resid)
         getattr(self, "_run_" + self.family)(rows, B, S, input_pos)
-        return B, S, rows
 
     @torch.no_grad()
     def forward(self, idx, input_pos):
         B, S, rows = self._trunk(idx, input_pos)
-        logits = torch.empty(B, S, self.cfg.vocab_size, dtype=self.resid.dtype, device=self.resid.device)
+        logits = torch.empty(B, S, self.cfg.vocab_size, dtype=self.dtype, device=self.resid.device)
         self.ops.linear(self.normed, self.model.output.weight, logits, rows, workspace=self.ws_head)
         return logits
 
@@ -184,7 +196,7 @@ class Engine:
         most of the LM-head work (32 x 4096 positions x 128256 logits = 33.6 GB of output)."""
         B, S, rows = self._trunk(idx, input_pos)
         last = self.normed[:rows].view(B, S, self.d)[:, -1].contiguous()
-        logits = torch.empty(B, 1, self.cfg.vocab_size, dtype=self.resid.dtype, device=self.resid.device)
+        logits = torch.empty(B, 1, self.cfg.vocab_size, dtype=self.dtype, device=self.resid.device)
         self.ops.linear(last, self.model.output.weight, logits, B, workspace=self.ws_head)
         return logits
 
@@ -251,7 +263,7 @@ class Engine:
         assert S == 1, "forward_sample is a decode step (one position per sequence)"
         t, V = self.comm.world, self.cfg.vocab_size
         n = self.vocab_hi - self.vocab_lo
-        dtype, dev = self.resid.dtype, self.resid.device
+        dtype, dev = self.dtype, self.resid.device
         local = self.head_logits[: B * max(n, 1)].view(B, max(n, 1))
         if n > 0:
             self.ops.linear(self.normed, self.model.output.weight[self.vocab_lo:self.vocab_hi], local, B,

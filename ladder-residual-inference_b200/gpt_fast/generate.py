@@ -41,10 +41,11 @@ class DeviceLoop:
                 self.pos.add_(1)
 
     def _graph(self, n: int) -> torch.cuda.CUDAGraph:
-        """Graph of n consecutive steps; captured once (the warm-up steps advance the position, which
-        the caller's start() sets afterwards)."""
+        """Graph of n consecutive steps; captured once.  The warm-up step advances token, position and any
+        recurrent state; all are put back."""
         if n not in self._graphs:
             tok0, pos0 = self.tok.clone(), self.pos.clone()
+            state0 = [s.clone() for s in self.model.recurrent_state()]
             side = torch.cuda.Stream()
             side.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(side):
@@ -53,6 +54,8 @@ class DeviceLoop:
             torch.cuda.synchronize()
             self.tok.copy_(tok0)
             self.pos.copy_(pos0)
+            for s, s0 in zip(self.model.recurrent_state(), state0):
+                s.copy_(s0)
             g = torch.cuda.CUDAGraph()
             with torch.cuda.graph(g):
                 self._steps(n)

@@ -1,4 +1,5 @@
-"""Hugging Face Llama / LlamaLadder checkpoints -> the fused, sharded parameter layout of this package.
+"""Checkpoints -> the fused, sharded parameter layout of this package: Hugging Face Llama / LlamaLadder, and Patevik.
+`load_model(path)` picks the model class from the folder's config.json.
 
 The reference has no loader (every rank draws its own random shard, benchmark.py:242-243); the only
 conversion it carries is the load hook that fuses separate wq / wk / wv into wqkv
@@ -77,6 +78,132 @@ def hf_to_local(hf: Dict[str, Tensor], config, rank: int, world: int, family: st
     return out
 
 
+def _fuse_branch(get, name: str, branch, parts, rank: int, world: int) -> Dict[str, Tensor]:
+    """Parameters of one gated residual branch; `parts` lists (tensor, "rows" or "all") of the sublayer's input rows."""
+    rows = [get(f"{name}.gate")] + [_rows(t, rank, world) if how == "rows" else t for t, how in parts]
+    total = branch.in_proj.weight.shape[0]
+    have = sum(r.shape[0] for r in rows)
+    if have < total:
+        rows.append(torch.zeros(total - have, rows[0].shape[1], dtype=rows[0].dtype))
+    return {"in_proj.weight": torch.cat(rows), "gate_bias": get(f"{name}.gate_bias"), "pre_norm": get(f"{name}.pre"),
+            "post_norm": get(f"{name}.post")}
+
+
+def patevik_to_local(w: Dict[str, Tensor], model, rank: int, world: int) -> Dict[str, Tensor]:
+    """Patevik checkpoint tensors -> state dict of rank `rank` of `world` for GPTPatevik's module tree:
+
+        in_proj   rows [gate of the branch | sublayer's input rows of the rank | zero rows]
+        expand    rows [W_uk of the rank's heads | W_uv of the rank's heads]
+        w1, w2    stacked experts, rows [up | gate] and columns of the rank's slice of the expert width
+    """
+    out = {"tok_embeddings.weight": w["embed"], "norm.weight": w["final.norm"], "output.weight": w["head"]}
+    for i, block in enumerate(model.layers):
+        p = f"l{i}."
+        names = {"mixer.gate": "rg1", "mixer.gate_bias": "rg1.b", "mixer.pre": "norm1", "mixer.post": "norm1b",
+                 "mlp.gate": "rg2", "mlp.gate_bias": "rg2.b", "mlp.pre": "norm2", "mlp.post": "norm2b"}
+
+        def get(k):
+            return w[p + names[k]]
+
+        mixer = block.mixer.sublayer
+        parts = [(w[f"{p}mix.{t}"], how) for t, how in mixer.tensors().items()]
+        for k, v in _fuse_branch(get, "mixer", block.mixer, parts, rank, world).items():
+            out[f"layers.{i}.mixer.{k}"] = v
+        dst = f"layers.{i}.mixer.sublayer."
+        out[dst + "wo.weight"] = _cols(w[p + "mix.o"], rank, world)
+        if mixer.kind == "latent_attention":
+            out[dst + "latent_norm"] = w[p + "mix.dkv.norm"]
+            out[dst + "expand.weight"] = torch.cat([_rows(w[p + "mix.uk"], rank, world), _rows(w[p + "mix.uv"], rank, world)])
+        else:
+            out[dst + "f_bias"] = _rows(w[p + "mix.f.b"], rank, world)
+            out[dst + "lower"] = _rows(w[p + "mix.lower"], rank, world)
+            out[dst + "norm"] = w[p + "mix.norm"]
+        if block.mlp is None:
+            continue
+        moe = block.mlp.sublayer
+        for k, v in _fuse_branch(get, "mlp", block.mlp, [(w[p + "mlp.router"], "all")], rank, world).items():
+            out[f"layers.{i}.mlp.{k}"] = v
+        dst = f"layers.{i}.mlp.sublayer."
+        experts = [f"{p}mlp.e{e}." for e in range(moe.experts)]
+        out[dst + "w1"] = torch.stack([torch.cat([_rows(w[e + "up"], rank, world), _rows(w[e + "gate"], rank, world)])
+                                       for e in experts])
+        out[dst + "w2"] = torch.stack([_cols(w[e + "down"], rank, world) for e in experts])
+    return out
+
+
+def _read_safetensors(path: str) -> Dict[str, Tensor]:
+    from safetensors.torch import load_file
+    files = sorted(glob.glob(os.path.join(path, "*.safetensors"))) if os.path.isdir(path) else [path]
+    if not files:
+        raise FileNotFoundError(f"no *.safetensors under {path}")
+    out: Dict[str, Tensor] = {}
+    for f in files:
+        out.update(load_file(f))
+    return out
+
+
+def _copy_parameters(model, local: Dict[str, Tensor]) -> None:
+    params = dict(model.named_parameters())
+    missing = sorted(set(params) - set(local))
+    if missing:
+        raise KeyError(f"checkpoint has no tensor for {missing[:4]}{' ...' if len(missing) > 4 else ''}")
+    with torch.no_grad():
+        for name, p in params.items():
+            src = local[name]
+            if tuple(src.shape) != tuple(p.shape):
+                raise ValueError(f"{name}: checkpoint shard {tuple(src.shape)} vs parameter {tuple(p.shape)}")
+            p.copy_(src.to(device=p.device, dtype=p.dtype))
+
+
+def _patevik_class(config: dict):
+    from .gpt_patevik_TP import GPTPatevik, ModelArgs
+    return GPTPatevik, ModelArgs.from_config(config)
+
+
+def _llama_class(path_or_config):
+    """Llama checkpoints run the ladder family when the config names ladder layers, the dense family otherwise."""
+    from . import gpt_dense_TP, gpt_ladder_TP
+    kw = model_args_from_hf_config(path_or_config)
+    if "ladder_layers" in kw:
+        return gpt_ladder_TP.GPTLadder, gpt_ladder_TP.ModelArgs(**kw)
+    return gpt_dense_TP.GPTDense, gpt_dense_TP.ModelArgs(**kw)
+
+
+def model_class(path: str):
+    """(model class, model args) of the checkpoint folder `path`, by its config.json: `architecture` for designs with
+    their own format, otherwise the Hugging Face Llama fields."""
+    with open(os.path.join(path, "config.json")) as f:
+        config = json.load(f)
+    name = config.get("architecture")
+    if name is None:
+        return _llama_class(path)
+    known = {"Patevik": _patevik_class}
+    if name not in known:
+        raise ValueError(f"unknown architecture {name!r}; known: {sorted(known)}")
+    return known[name](config)
+
+
+def load_model(path: str, dtype=torch.bfloat16, device="cuda", max_batch_size: Optional[int] = None,
+               max_seq_length: Optional[int] = None):
+    """Model of the checkpoint folder `path` on `device`, in `dtype`, this rank's shard; caches set up when both
+    sizes are given."""
+    cls, args = model_class(path)
+    if dtype not in cls.dtypes:
+        raise TypeError(f"{cls.__name__} runs in {[str(d) for d in cls.dtypes]}, not {dtype}")
+    with torch.device("meta"):
+        model = cls(args)
+    model = model.to(dtype=dtype).to_empty(device=device).eval()
+    rank, world = dist.get_rank(), dist.get_world_size()
+    tensors = _read_safetensors(path)
+    if cls.family == "patevik":
+        _copy_parameters(model, patevik_to_local(tensors, model, rank, world))
+    else:
+        load_hf_state_dict(model, tensors, rank, world)
+    if max_batch_size is not None and max_seq_length is not None:
+        model.setup_caches(max_batch_size=max_batch_size, max_seq_length=max_seq_length)
+    return model
+
+
 def model_args_from_hf_config(path: str) -> Dict[str, object]:
     """ModelArgs keyword arguments from the config.json of a Hugging Face Llama / LlamaLadder
     checkpoint directory (field names: transformers' LlamaConfig; `ladder_layers` as normalised by
@@ -109,25 +236,9 @@ def load_hf_state_dict(model, hf: Dict[str, Tensor], rank: Optional[int] = None,
     rank = dist.get_rank() if rank is None else rank
     world = dist.get_world_size() if world is None else world
     local = hf_to_local(hf, model.config, rank, world, model.family)
-    params = dict(model.named_parameters())
-    missing = sorted(set(params) - set(local))
-    if missing:
-        raise KeyError(f"checkpoint has no tensor for {missing[:4]}{' ...' if len(missing) > 4 else ''}")
-    with torch.no_grad():
-        for name, p in params.items():
-            src = local[name]
-            if tuple(src.shape) != tuple(p.shape):
-                raise ValueError(f"{name}: checkpoint shard {tuple(src.shape)} vs parameter {tuple(p.shape)}")
-            p.copy_(src.to(device=p.device, dtype=p.dtype))
+    _copy_parameters(model, local)
 
 
 def load_hf_checkpoint(model, path: str, rank: Optional[int] = None, world: Optional[int] = None) -> None:
     """`path`: a directory of *.safetensors shards (or one file) in Hugging Face Llama naming."""
-    from safetensors.torch import load_file
-    files = sorted(glob.glob(os.path.join(path, "*.safetensors"))) if os.path.isdir(path) else [path]
-    if not files:
-        raise FileNotFoundError(f"no *.safetensors under {path}")
-    hf: Dict[str, Tensor] = {}
-    for f in files:
-        hf.update(load_file(f))
-    load_hf_state_dict(model, hf, rank, world)
+    load_hf_state_dict(model, _read_safetensors(path), rank, world)

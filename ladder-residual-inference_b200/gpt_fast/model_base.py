@@ -58,6 +58,8 @@ class TPModelBase(nn.Module):
     code use.  forward(idx [B, S], input_pos [S]) -> logits [B, S, vocab]."""
 
     family = ""
+    engine_class = Engine
+    dtypes = (torch.bfloat16, torch.float16)  # storage types the family's kernels run
 
     def __init__(self, config, blocks) -> None:
         super().__init__()
@@ -75,32 +77,39 @@ class TPModelBase(nn.Module):
     def setup_caches(self, max_batch_size, max_seq_length):
         if self.max_seq_length >= max_seq_length and self.max_batch_size >= max_batch_size:
             return
-        cfg = self.config
-        world = dist.get_world_size()
-        head_dim = cfg.dim // cfg.n_head
         max_seq_length = find_multiple(max_seq_length, 8)
         self.max_seq_length = max_seq_length
         self.max_batch_size = max_batch_size
         dtype = self.output.weight.dtype
         device = self.output.weight.device
+        self._setup_layer_caches(max_batch_size, max_seq_length, dtype, device)
+        self._engine = self.engine_class(self, self.family)
+        self._engine.setup(max_batch_size, max_seq_length, device, dtype)
+
+    def _setup_layer_caches(self, max_batch_size, max_seq_length, dtype, device):
+        cfg = self.config
+        head_dim = cfg.dim // cfg.n_head
         for b in self.layers:
-            b.attention.kv_cache = KVCache(max_batch_size, max_seq_length, cfg.n_local_heads // world, head_dim,
-                                           dtype).to(device)
+            b.attention.kv_cache = KVCache(max_batch_size, max_seq_length, cfg.n_local_heads // dist.get_world_size(),
+                                           head_dim, dtype).to(device)
         self.freqs_cis = precompute_freqs_cis(cfg.block_size, head_dim, cfg.rope_base, dtype,
                                               cfg.rope_scaling).to(device).contiguous()
         # kept because callers of the reference may read it; the kernels derive causality from input_pos
         self.causal_mask = torch.tril(torch.ones(max_seq_length, max_seq_length, dtype=torch.bool, device=device))
-        self._engine = Engine(self, self.family)
-        self._engine.setup(max_batch_size, max_seq_length, device, dtype)
+
+    def recurrent_state(self):
+        """Tensors a step reads and overwrites, so that repeating a step needs them restored (none for attention
+        caches: rewriting a position with the same values changes nothing)."""
+        return []
 
     def forward(self, idx: Tensor, input_pos: Optional[Tensor] = None) -> Tensor:
-        assert self.freqs_cis is not None, "Caches must be initialized first"
+        assert self._engine is not None, "Caches must be initialized first"
         return self._engine.forward(idx, input_pos)
 
     def prefill_last(self, idx: Tensor, input_pos: Tensor) -> Tensor:
         """forward(idx, input_pos)[:, -1:] without computing the other positions' logits (no
         counterpart in the reference, whose forward always projects every position)."""
-        assert self.freqs_cis is not None, "Caches must be initialized first"
+        assert self._engine is not None, "Caches must be initialized first"
         return self._engine.forward_last(idx, input_pos)
 
     def decode_greedy(self, idx: Tensor, input_pos: Tensor) -> Tensor:
@@ -108,7 +117,7 @@ class TPModelBase(nn.Module):
         `forward(idx, input_pos)[:, -1].argmax(-1)` but with the output projection split by
         vocabulary over the tensor-parallel ranks (no counterpart in the reference, which
         samples from the replicated logits, benchmark.py:74-92)."""
-        assert self.freqs_cis is not None, "Caches must be initialized first"
+        assert self._engine is not None, "Caches must be initialized first"
         return self._engine.forward_greedy(idx, input_pos)
 
     def decode_sample(self, idx: Tensor, input_pos: Tensor, temperature: float = 1.0, top_k: Optional[int] = None,
@@ -116,7 +125,7 @@ class TPModelBase(nn.Module):
         """One sampled next token per sequence, int32 [B, 1], by the reference's rule
         (`sample(model(idx, input_pos), temperature, top_k)[0]`, benchmark.py:56-92), computed on the
         vocabulary-split output projection; see Engine.forward_sample."""
-        assert self.freqs_cis is not None, "Caches must be initialized first"
+        assert self._engine is not None, "Caches must be initialized first"
         return self._engine.forward_sample(idx, input_pos, temperature, top_k, generator)
 
 

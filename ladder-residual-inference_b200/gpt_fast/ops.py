@@ -40,7 +40,7 @@ class CudaOps:
         _C.require_cuda(x, w, out)
         n, k = w.shape
         ws_ptr, ws_bytes = (workspace.data_ptr(), workspace.numel() * workspace.element_size()) if workspace is not None else (None, 0)
-        _C.check(_C.lib.lri_linear(_C.dtype_code(x.dtype), x.data_ptr(), w.data_ptr(), _C.ptr(addend), out.data_ptr(),
+        _C.check(_C.lib.lri_linear(_C.dtype_code_any(x.dtype), x.data_ptr(), w.data_ptr(), _C.ptr(addend), out.data_ptr(),
                                    rows, n, k, ws_ptr, ws_bytes, _C.stream_handle()))
 
     @staticmethod
@@ -117,6 +117,141 @@ class CudaOps:
             _C.check(_C.lib.lri_attn_prefill(code, q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                                              input_pos.data_ptr(), i64, out.data_ptr(), B, S, n_head, n_kv, head_dim,
                                              smax, _C.stream_handle()))
+
+
+    # ---- layers with an fp32 residual stream ---------------------------------------------------------
+    @staticmethod
+    def linear_f32(x, w, out, rows, workspace=None):
+        """out (fp32) = x w^T, unrounded."""
+        _C.require_cuda(x, w, out)
+        n, k = w.shape
+        ws_ptr, ws_bytes = (workspace.data_ptr(), workspace.numel() * workspace.element_size()) if workspace is not None else (None, 0)
+        _C.check(_C.lib.lri_linear_f32(_C.dtype_code_any(x.dtype), x.data_ptr(), w.data_ptr(), out.data_ptr(), rows, n, k,
+                                       ws_ptr, ws_bytes, _C.stream_handle()))
+
+    @staticmethod
+    def linear_f32_workspace_bytes(rows, n):
+        return _C.lib.lri_linear_f32_workspace_bytes(rows, n)
+
+    @staticmethod
+    def embed_norm(table, idx, resid, weight, eps, normed):
+        _C.require_cuda(table, idx, resid)
+        if idx.dtype not in (torch.int32, torch.int64):
+            idx = idx.to(torch.int64)
+        idx = idx.contiguous()
+        _C.check(_C.lib.lri_embed_norm(_C.dtype_code_any(table.dtype), table.data_ptr(), idx.data_ptr(),
+                                       int(idx.dtype == torch.int64), table.shape[0], resid.data_ptr(), _C.ptr(weight),
+                                       float(eps), _C.ptr(normed), idx.numel(), table.shape[1], _C.stream_handle()))
+
+    @staticmethod
+    def gated_norm_add(resid, y, gate, gate_ld, gate_bias, post_weight, eps, next_weight, normed, rows, n_slots=1,
+                       slots=None, y_rows=None):
+        """resid += post norm of the gated sum over slots of y; normed = norm of the new residual.  `gate` is a
+        view that starts at the gate's first column of an fp32 buffer with row pitch gate_ld."""
+        _C.require_cuda(resid, y)
+        _C.check(_C.lib.lri_gated_norm_add(_C.dtype_code_any(y.dtype), resid.data_ptr(), y.data_ptr(), _C.ptr(slots), n_slots,
+                                           y_rows if y_rows is not None else rows * n_slots, _C.ptr(gate), gate_ld,
+                                           _C.ptr(gate_bias), _C.ptr(post_weight), float(eps), resid.data_ptr(),
+                                           _C.ptr(next_weight), _C.ptr(normed), rows, resid.shape[-1], _C.stream_handle()))
+
+    @staticmethod
+    def sum_slots(y, rows, n_slots, slots, y_rows, out):
+        """out[r] = sum of the rows slots[r, :] of y (slots None: rows r * n_slots ...), rounded once."""
+        _C.require_cuda(y, out)
+        _C.check(_C.lib.lri_gated_norm_add(_C.dtype_code_any(y.dtype), None, y.data_ptr(), _C.ptr(slots), n_slots, y_rows, None, 0,
+                                           None, None, 0.0, None, None, out.data_ptr(), rows, out.shape[-1],
+                                           _C.stream_handle()))
+
+    # ---- latent attention ------------------------------------------------------------------------------
+    @staticmethod
+    def latent_prepare(proj, ld, q_off, kv_off, norm_weight, eps, table, input_pos, qn, qn_pitch, qr, qr_pitch, cache, B, S,
+                       heads, dim, rot_dim, rank):
+        """qn_pitch, qr_pitch: (row, head) element pitches of the unrotated and the rotated part of q."""
+        _C.require_cuda(proj, norm_weight, table, input_pos, qn, qr, cache)
+        _C.check(_C.lib.lri_latent_prepare(
+            _C.dtype_code_any(cache.dtype), proj.data_ptr(), ld, q_off, kv_off, norm_weight.data_ptr(), float(eps),
+            table.data_ptr(), table.shape[0], input_pos.data_ptr(), int(input_pos.dtype == torch.int64), qn.data_ptr(),
+            qn_pitch[0], qn_pitch[1], qr.data_ptr(), qr_pitch[0], qr_pitch[1], cache.data_ptr(), cache.shape[1], B, S, heads,
+            dim, rot_dim, rank, _C.stream_handle()))
+
+    @staticmethod
+    def latent_window(cache, rank, rot_dim, input_pos, B, history, rows, latent, k_rot):
+        _C.require_cuda(cache, input_pos, latent, k_rot)
+        _C.check(_C.lib.lri_latent_window(_C.dtype_code_any(cache.dtype), cache.data_ptr(), cache.shape[1], rank, rot_dim,
+                                          input_pos.data_ptr(), int(input_pos.dtype == torch.int64), B, history, rows,
+                                          latent.data_ptr(), k_rot.data_ptr(), _C.stream_handle()))
+
+    @staticmethod
+    def head_linear(x, x_pitch, w, transposed, y, y_pitch, rows, heads, n_in, n_out):
+        """y[row, head] = W[head] x[row, head]; pitches are (row, head) in elements."""
+        _C.require_cuda(x, w, y)
+        _C.check(_C.lib.lri_head_linear(_C.dtype_code_any(w.dtype), x.data_ptr(), x_pitch[0], x_pitch[1], w.data_ptr(),
+                                        int(transposed), y.data_ptr(), y_pitch[0], y_pitch[1], rows, heads, n_in, n_out,
+                                        _C.stream_handle()))
+
+    @staticmethod
+    def window_attention(q, q_pitch, k, k_pitch, k2, k2_pitch, v, v_pitch, out, input_pos, history, k_rows, window, scale, B,
+                         S, heads, d1, d2, dv):
+        """q_pitch (row, head); k_pitch, v_pitch (batch, row, head); k2_pitch (batch, row), in elements."""
+        _C.require_cuda(q, k, k2, v, out, input_pos)
+        _C.check(_C.lib.lri_window_attention(
+            _C.dtype_code_any(q.dtype), q.data_ptr(), *q_pitch, k.data_ptr(), *k_pitch, k2.data_ptr(), *k2_pitch,
+            v.data_ptr(), *v_pitch, out.data_ptr(), input_pos.data_ptr(), int(input_pos.dtype == torch.int64), history,
+            k_rows, window, float(scale), B, S, heads, d1, d2, dv, _C.stream_handle()))
+
+    # ---- recurrence ----------------------------------------------------------------------------------------
+    @staticmethod
+    def hgrn2_workspace_bytes(dtype, B, S, heads, dim, vdim):
+        return _C.lib.lri_hgrn2_workspace_bytes(_C.dtype_code_any(dtype), B, S, heads, dim, vdim)
+
+    @staticmethod
+    def hgrn2(proj, ld, q_off, f_off, v_off, f_bias, lower, norm_weight, eps, state, input_pos, out, B, S, heads, dim, vdim,
+              workspace):
+        _C.require_cuda(proj, f_bias, lower, norm_weight, state, input_pos, out, workspace)
+        _C.check(_C.lib.lri_hgrn2(
+            _C.dtype_code_any(out.dtype), proj.data_ptr(), ld, q_off, f_off, v_off, f_bias.data_ptr(), lower.data_ptr(),
+            norm_weight.data_ptr(), float(eps), state.data_ptr(), input_pos.data_ptr(), int(input_pos.dtype == torch.int64),
+            out.data_ptr(), B, S, heads, dim, vdim, workspace.data_ptr(), workspace.numel() * workspace.element_size(),
+            _C.stream_handle()))
+
+    # ---- mixture of experts -----------------------------------------------------------------------------------
+    @staticmethod
+    def moe_packs(dtype, rows, top, dim, ff):
+        return bool(_C.lib.lri_moe_packs(_C.dtype_code_any(dtype), rows, top, dim, ff))
+
+    @staticmethod
+    def moe_max_tiles(rows, top, experts):
+        return _C.lib.lri_moe_max_tiles(rows, top, experts)
+
+    @staticmethod
+    def moe_route(logits, ld, experts, top, rows, ids, scores, counts=None, rank=None):
+        _C.require_cuda(logits, ids, scores)
+        _C.check(_C.lib.lri_moe_route(logits.data_ptr(), ld, experts, top, rows, ids.data_ptr(), scores.data_ptr(),
+                                      _C.ptr(counts), _C.ptr(rank), _C.stream_handle()))
+
+    @staticmethod
+    def moe_pack(x, rows, top, experts, ids, scores, rank, counts, first_row, tiles, packed, row_scale, slots):
+        _C.require_cuda(x, packed)
+        _C.check(_C.lib.lri_moe_pack(_C.dtype_code(x.dtype), x.data_ptr(), rows, x.shape[-1], top, experts, ids.data_ptr(),
+                                     scores.data_ptr(), rank.data_ptr(), counts.data_ptr(), first_row.data_ptr(),
+                                     tiles.data_ptr(), packed.data_ptr(), row_scale.data_ptr(), slots.data_ptr(),
+                                     _C.stream_handle()))
+
+    @staticmethod
+    def moe_gateup(x, w1, hidden, ids, scores, pairs, top, glu, tiles=None, row_scale=None, max_tiles=0):
+        """w1 [experts, 2 ff, dim]; glu = (alpha, limit, offset); with `tiles` x and hidden are packed rows."""
+        _C.require_cuda(x, w1, hidden)
+        experts, two_ff, dim = w1.shape
+        _C.check(_C.lib.lri_moe_gateup(_C.dtype_code_any(x.dtype), x.data_ptr(), w1.data_ptr(), hidden.data_ptr(), _C.ptr(ids),
+                                       _C.ptr(scores), pairs, top, _C.ptr(tiles), _C.ptr(row_scale), max_tiles, experts,
+                                       two_ff // 2, dim, *[float(g) for g in glu], _C.stream_handle()))
+
+    @staticmethod
+    def moe_down(hidden, w2, y, ids, pairs, tiles=None, max_tiles=0):
+        _C.require_cuda(hidden, w2, y)
+        experts, dim, ff = w2.shape
+        _C.check(_C.lib.lri_moe_down(_C.dtype_code_any(hidden.dtype), hidden.data_ptr(), w2.data_ptr(), y.data_ptr(),
+                                     _C.ptr(ids), pairs, _C.ptr(tiles), max_tiles, experts, dim, ff, _C.stream_handle()))
 
 
 def decode_splits(B, n_head, n_kv, smax, head_dim=128):

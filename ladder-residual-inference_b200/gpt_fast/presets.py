@@ -61,6 +61,25 @@ ARCH = {
                                    vocab_size=128256, rope_base=500000, rope_scaling=_LLAMA31_SCALING),
 }
 
+
+
+def _layer_list(n_layer, width, heads, dim, vdim, kv_rank, rot_dim, window, experts, top, ff, vocab, rope_base=500000.0):
+    """Alternating HGRN2 and latent-attention layers of one size, each with a mixture of experts."""
+    mlp = dict(kind="moe", expert=dict(ff=ff, limit=7.0), router=dict(experts=experts, top=top))
+    recurrent = dict(type="hgrn2", mixer=dict(heads=heads, dim=dim, vdim=vdim), mlp=mlp)
+    latent = dict(type="latent_attention", mlp=mlp,
+                  mixer=dict(heads=heads, dim=dim, vdim=vdim, kv_rank=kv_rank, rot_dim=rot_dim, mask=dict(size=window),
+                             rot=dict(base=rope_base, dims=rot_dim), scale=(dim + rot_dim) ** -0.5))
+    return dict(vocab_size=vocab, dim=width, layers=[deepcopy(latent if i % 2 else recurrent) for i in range(n_layer)])
+
+
+# Layer-list designs.  The active parameters of a layer's feed-forward are those of the Llama shape of the same name.
+LAYER_LISTS = {
+    "patevik-tiny": _layer_list(4, 192, 3, 32, 64, 48, 32, 40, 6, 2, 96, 512),
+    "patevik-1b": _layer_list(16, 2048, 32, 64, 64, 256, 32, 1024, 8, 2, 4096, 128256),
+    "patevik-8b": _layer_list(32, 4096, 32, 128, 128, 512, 64, 4096, 8, 2, 7168, 128256),
+}
+
 _COMMON = ["CodeLlama-7b-Python-hf", "1b", "3b", "7B", "13B", "30B", "34B", "70B", "Mistral-7B", "stories15M",
            "stories110M", "llama-3.2-1b", "llama-3.2-3b", "llama-3-8b", "llama-3-70b", "llama-3.1-405b",
            "ladder-llama-1b", "ladder-llama-405b-kv8"]
@@ -76,7 +95,9 @@ def _every_other_mlp(n_layer):
 
 
 def family_presets(family):
-    """Returns {preset name: ModelArgs kwargs} for 'ladder', 'dense', 'parallel' or 'desync'."""
+    """Returns {preset name: ModelArgs kwargs} for 'ladder', 'dense', 'parallel', 'desync' or 'patevik'."""
+    if family == "patevik":
+        return deepcopy(LAYER_LISTS)
     out = {}
 
     def add(name, arch=None, **extra):
