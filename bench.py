@@ -1,7 +1,7 @@
 """Decode-throughput bench of the tensor-parallel Ladder-Llama step on B200.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--batch B] [--preset llama-3-8b]
-                    [--family ladder] [--impl ours|reference] [--mode decode|prefill|kernels]
+                    [--family ladder|...|patevik] [--impl ours|reference] [--mode decode|prefill|kernels]
     python -m torch.distributed.run --nnodes=1 --nproc-per-node N --master-addr 127.0.0.1 \
         --master-port P bench.py --gpus N ...
 
@@ -67,8 +67,11 @@ def parse_args(argv=None):
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--repeats", type=int, default=5, help="repeats of the K-step timed region (median reported)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--family", default="ladder", choices=["ladder", "dense", "parallel", "desync"])
-    ap.add_argument("--preset", default="llama-3-8b")
+    ap.add_argument("--family", default="ladder", choices=["ladder", "dense", "parallel", "desync", "patevik"],
+                    help="patevik (presets patevik-8b, patevik-1b): decode and prompt throughput of the layer-list design "
+                         "beside the dense Llama model of equal width, depth and active parameters, one line for both; "
+                         "with --mode kernels a table of every op of a decode step and of a prompt pass against its roofline")
+    ap.add_argument("--preset", default=None, help="default: llama-3-8b (patevik-8b for --family patevik)")
     ap.add_argument("--batch", type=int, default=1)
     ap.add_argument("--prompt", type=int, default=1024)
     ap.add_argument("--dtype", default="bf16", choices=["bf16", "fp16"])
@@ -100,7 +103,10 @@ def parse_args(argv=None):
     ap.add_argument("--reps", type=int, default=20)
     ap.add_argument("--json", default="")
     ap.add_argument("--eager", action="store_true", help="kernels mode: launch from Python instead of replaying a graph")
-    return ap.parse_args(argv)
+    args = ap.parse_args(argv)
+    if args.preset is None:
+        args.preset = "patevik-8b" if args.family == "patevik" else "llama-3-8b"
+    return args
 
 
 def _peaks():
@@ -363,7 +369,10 @@ def workload_config(args, a, note=None):
 # our arm
 # ---------------------------------------------------------------------------------------------
 
-FAMILY_CLASS = {"ladder": "GPTLadder", "dense": "GPTDense", "parallel": "GPTParallel", "desync": "GPTDesync"}
+FAMILY_CLASS = {"ladder": "GPTLadder", "dense": "GPTDense", "parallel": "GPTParallel", "desync": "GPTDesync",
+                "patevik": "GPTPatevik"}
+# dense Llama shape of equal width, depth, vocabulary and active feed-forward parameters
+EQUAL_SIZE = {"patevik-8b": "llama-3-8b", "patevik-1b": "ladder-llama-1b"}
 
 
 class DecodeLoop:
@@ -378,6 +387,7 @@ class DecodeLoop:
         self.tok = first.clone()
         self.pos = torch.tensor([T], dtype=torch.int32, device=dev)
         self.nxt = torch.empty_like(self.tok)
+        self.state0 = [s.clone() for s in model.recurrent_state()]  # a step at position T starts from here
         self.graph = None
         self.use_graph = use_graph
 
@@ -417,6 +427,8 @@ class DecodeLoop:
     def reset(self):
         self.tok.copy_(self.first)
         self.pos.fill_(self.T)
+        for s, s0 in zip(self.model.recurrent_state(), self.state0):
+            s.copy_(s0)
 
 
 def build_model(gpt_fast, family, preset, dtype, dev, share_with=None):
@@ -432,6 +444,9 @@ def build_model(gpt_fast, family, preset, dtype, dev, share_with=None):
         return model.eval()
     model = model.to(dtype=dtype).to_empty(device=dev).eval()
     torch.manual_seed(1234)  # same stream on every rank: replicated parameters are identical
+    if hasattr(model, "init_random_"):
+        model.init_random_(0.02)
+        return model
     with torch.no_grad():
         for p in model.parameters():
             torch.nn.init.normal_(p, mean=0.0, std=0.02)
@@ -639,6 +654,99 @@ def run_ours(args):
         line["cpu_baseline"] = {"value": tps, "unit": UNIT, "cores": cores, "kind": "port",
                                 "sample": cpu_sample_text(a, args.cpu_layers, T, B, steps_cpu, warm_cpu, 1)}
         line["cpu_baseline_config1"] = cpu_config1_baseline()
+    print(json.dumps(line), flush=True)
+
+
+def run_layer_family(args):
+    """Decode and prompt throughput of a layer-list model and of the dense Llama model of equal size, same batch, prompt
+    and kernels' conventions; or (--mode kernels) every op of both against its roofline."""
+    import torch
+    import gpt_fast
+    from gpt_fast import _C, op_bench
+    assert args.gpus == 1, "the layer-list comparison runs on one GPU"
+    if args.preset not in EQUAL_SIZE:
+        raise SystemExit(f"--family patevik takes --preset {' or '.join(EQUAL_SIZE)}")
+    dev = torch.device("cuda", torch.cuda.current_device())
+    dtype = torch.bfloat16 if args.dtype == "bf16" else torch.float16
+    B, T, K, W, R = args.batch, args.prompt, args.steps, args.warmup, max(1, args.repeats)
+    hbm, _ = measured_hbm_peak()
+    tensor, _ = measured_tensor_peak()
+    g = torch.Generator().manual_seed(1234)
+    arms = [("patevik", args.preset)] + ([] if args.no_compare else [("dense", EQUAL_SIZE[args.preset])])
+    out = {}
+    sampler = ClockSampler(torch.cuda.current_device())
+    for family, preset in arms:
+        model = build_model(gpt_fast, family, preset, dtype, dev)
+        model.setup_caches(max_batch_size=B, max_seq_length=T + W + K + 24)
+        x = torch.randint(0, model.config.vocab_size, (B, T), generator=g).to(dev)
+        positions = torch.arange(T, device=dev)
+
+        def prompt():
+            with torch.no_grad():
+                return model.prefill_last(x, positions)
+
+        first = prompt()[:, -1].float().argmax(-1, keepdim=True).to(torch.int32)
+        if args.mode == "kernels":
+            experts = model.config.layers[0]["mlp"]["router"]["experts"] if family == "patevik" else None
+            tok, pos = first.clone(), torch.tensor([T], dtype=torch.int32, device=dev)
+            wanted = [w for w in args.only.split(",") if w]
+            for label, step, pos0 in (("decode", lambda: model.decode_greedy(tok, pos), T), ("prompt", prompt, 0)):
+                calls = [c for c in op_bench.record(model._engine, step) if not wanted or any(c[0][0] == w for w in wanted)]
+                for r in op_bench.time_calls(calls, pos0, hbm, tensor, experts):
+                    print(json.dumps({"model": f"{family}:{preset}", "step": label, "batch": B, "prompt": T, **r}), flush=True)
+            del model
+            torch.cuda.empty_cache()
+            continue
+        c0 = _C.lib.lri_launch_count()
+        prompt()
+        prompt_launches = _C.lib.lri_launch_count() - c0
+
+        def timed(n, body):
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            for _ in range(n):
+                body()
+            e1.record()
+            torch.cuda.synchronize()
+            return e0.elapsed_time(e1) / n
+
+        for _ in range(3):
+            prompt()
+        sampler.start()
+        time.sleep(0.25)
+        t0 = time.time()
+        prompt_ms = statistics.median(timed(4, prompt) for _ in range(R))
+        loop = DecodeLoop(model, B, T, first, args.head, 1, not args.no_graph)
+        c0 = _C.lib.lri_launch_count()
+        loop.step()
+        launches = _C.lib.lri_launch_count() - c0
+        loop.capture()
+        runs = []
+        for _ in range(R):
+            loop.reset()
+            for _ in range(W):
+                loop.run()
+            runs.append(timed(K, loop.run))
+        clocks = sampler.stop(t0, time.time())
+        decode_ms = statistics.median(runs)
+        _C.check(_C.lib.lri_gemm_status())
+        out[family] = {"preset": preset, "decode_tokens_per_s": B / decode_ms * 1e3, "decode_ms_per_step": decode_ms,
+                       "prompt_tokens_per_s": B * T / prompt_ms * 1e3, "prompt_ms": prompt_ms,
+                       "launches_per_decode_step": int(launches), "launches_per_prompt": int(prompt_launches), "clocks": clocks,
+                       "weight_bytes": sum(p.numel() * p.element_size() for p in model.parameters())}
+        del loop, model
+        torch.cuda.empty_cache()
+    if args.mode == "kernels":
+        return
+    line = {"metric": METRIC, "value": out["patevik"]["decode_tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": K, "warmup": W,
+            "ms_per_step": out["patevik"]["decode_ms_per_step"], "higher_is_better": True, "vs_baseline": None, "dtype": args.dtype,
+            "data": "synthetic", "models": out,
+            "config": {"workload": f"patevik:{args.preset}, batch {B}, prompt {T} random ids (logits of the last position), greedy "
+                                   f"decode from there, random weights", "batch": B, "context": T,
+                       "l2": "inputs larger than L2: every step streams GBs of weights, no flush"}}
+    if "dense" in out:
+        line["vs_dense"] = {k: out["patevik"][k] / out["dense"][k] for k in ("decode_tokens_per_s", "prompt_tokens_per_s")}
     print(json.dumps(line), flush=True)
 
 
@@ -1037,6 +1145,8 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         run_reference_arm(args)
+    elif args.family == "patevik":
+        run_layer_family(args)
     elif args.mode == "comm":
         run_comm(args)
     elif args.mode == "kernels":

@@ -65,7 +65,9 @@ int lri_set_gemm_backend(int backend);
  * kernel), gemm_reserve_sms (LRI_GEMM_RESERVE_SMS: SMs
  * the persistent prefill GEMM leaves free for a collective running beside it, 0..64), attn_head_tile
  * (LRI_ATTN_HEAD_TILE: query heads of a KV group per CTA of the cluster decode attention, 0 choose, 1, 2, 4),
- * moe_stream_pairs (LRI_MOE_STREAM_PAIRS: (token, expert) pairs up to which experts run as streaming projections).  Unknown
+ * moe_stream_pairs (LRI_MOE_STREAM_PAIRS: (token, expert) pairs up to which experts run as streaming projections),
+ * window_tc (LRI_WINDOW_TC: 0 keeps sliding-window attention on the plain kernel), hgrn2_blocks
+ * (LRI_HGRN2_BLOCKS: 0 keeps the HGRN2 recurrence token by token).  Unknown
  * names and values an option does not take return LRI_ERR_ARG.  No counterpart in the reference
  * (its only switches are benchmark.py's command-line flags). */
 int lri_set_option(const char* name, int value);
@@ -320,13 +322,17 @@ int lri_head_linear(int dtype, const void* x, int64_t x_row, int64_t x_head, con
                     lri_stream_t stream);
 /* Softmax attention of query (row, head) = [d1 | d2] over the key rows j = [k (d1) | k2 (d2, shared by the heads)]
  * at positions input_pos[0] - history + j (history < 0: position j) with 0 <= position of the query - position of the key < window_size.
- * Row j of v has dv elements.  Pitches in elements; a head pitch of 0 shares a row among the heads. */
+ * Row j of v has dv elements.  Pitches in elements; a head pitch of 0 shares a row among the heads.
+ * 16-bit types: prompt portions (16 tokens on, dim and vdim up to 128, rot_dim up to 64, multiples of 8) run on tcgen05;
+ * single tokens over shared rows (k == v, k2 right behind k, d1 = dv up to 512, multiples of 16) on mma.sync, with
+ * scratch for the results of splits (keys = most keys a query sees); everything else on a plain kernel. */
+size_t lri_window_attention_scratch_bytes(int B, int heads, int dv, int64_t keys);
 int lri_window_attention(int dtype, const void* q, int64_t q_row, int64_t q_head, const void* k, int64_t k_batch,
                          int64_t k_row, int64_t k_head, const void* k2, int64_t k2_batch, int64_t k2_row,
                          const void* v, int64_t v_batch, int64_t v_row, int64_t v_head, void* out,
                          const void* input_pos, int pos_is_i64, int history, int64_t k_rows,
                          int64_t window_size, float scale, int B, int S, int heads, int d1, int d2, int dv,
-                         lri_stream_t stream);
+                         void* scratch, size_t scratch_bytes, lri_stream_t stream);
 
 /* ---- HGRN2 recurrence -----------------------------------------------------------------------------
  * proj [B*S, ld] fp32 holds q, f, v at the given offsets.  f = lower + (1 - lower) sigmoid(f + f_bias), q = silu(q);
@@ -348,10 +354,10 @@ int64_t lri_moe_max_tiles(int64_t rows, int top, int experts);
 int lri_moe_route(const float* logits, int64_t ld, int experts, int top, int64_t rows, int32_t* ids,
                   float* scores, int32_t* counts, int32_t* rank, lri_stream_t stream);
 /* Packs the rows of x by expert into tiles of 128: tiles = {count, expert of each}, packed rows and their scores,
- * slots [rows * top] = packed row of each pair.  Leaves counts at zero. */
+ * slots [rows * top] = packed row of each pair; the buffers hold max_tiles tiles.  Leaves counts at zero. */
 int lri_moe_pack(int dtype, const void* x, int64_t rows, int dim, int top, int experts, const int32_t* ids,
                  const float* scores, const int32_t* rank, int32_t* counts, int32_t* first_row, int32_t* tiles,
-                 void* packed, float* row_scale, int32_t* slots, lri_stream_t stream);
+                 int64_t max_tiles, void* packed, float* row_scale, int32_t* slots, lri_stream_t stream);
 /* hidden = g sigmoid(alpha g) (u + offset), g = min(s gate, limit), u = clamp(s up, -limit, limit) with the score s
  * of the pair and gate, up the two products with w1 [experts, 2 ff, dim] = [up | gate].  tiles == NULL: x [rows, dim],
  * hidden [pairs, ff]; else x and hidden are packed rows. */

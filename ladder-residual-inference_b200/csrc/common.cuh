@@ -64,6 +64,8 @@ enum Option {
   OPT_GEMM_RESERVE_SMS, // LRI_GEMM_RESERVE_SMS  SMs the persistent prefill GEMM leaves free (for a collective running beside it)
   OPT_ATTN_HEAD_TILE,   // LRI_ATTN_HEAD_TILE  query heads per CTA of the cluster decode-attention kernel: 1, 2, 4 (0 = choose)
   OPT_MOE_STREAM_PAIRS, // LRI_MOE_STREAM_PAIRS  (token, expert) pairs up to which experts run as streaming projections
+  OPT_WINDOW_TC,        // LRI_WINDOW_TC      0: sliding-window attention always on the plain kernel
+  OPT_HGRN2_BLOCKS,     // LRI_HGRN2_BLOCKS   0: the HGRN2 recurrence always runs token by token
   OPT_COUNT
 };
 int option(int which);

@@ -48,7 +48,8 @@ __device__ __forceinline__ void store_v(T* p, const float (&f)[VEC]) {
   }
 }
 
-template <typename T, int VEC, int NV, int THREADS>
+// PRE (few rows): the kernel is a chain of load latencies, so everything that can be loaded at once is.
+template <typename T, int VEC, int NV, int THREADS, bool PRE>
 __global__ void __launch_bounds__(THREADS) gated_norm_add_kernel(const GatedNormParams p) {
   __shared__ float part[33];
   const int64_t row = blockIdx.x;
@@ -57,9 +58,28 @@ __global__ void __launch_bounds__(THREADS) gated_norm_add_kernel(const GatedNorm
   const T* bias = static_cast<const T*>(p.gate_bias);
   const T* wpost = static_cast<const T*>(p.post_weight);
   const T* wnext = static_cast<const T*>(p.next_weight);
+  // constants of the model: fetched while the preceding kernel drains
+  [[maybe_unused]] float cb[NV][VEC], cp[NV][VEC], cn[NV][VEC];
+  if constexpr (PRE) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int v = threadIdx.x + i * THREADS;
+      if (v >= nvec) continue;
+      if (p.gate) load_v<T, VEC>(bias + v * VEC, cb[i]);
+      if (wpost) load_v<T, VEC>(wpost + v * VEC, cp[i]);
+      if (wnext) load_v<T, VEC>(wnext + v * VEC, cn[i]);
+    }
+  }
   pdl_launch_dependents();
   pdl_wait();
   float t[NV][VEC];
+  [[maybe_unused]] float res[NV][VEC];
+  if constexpr (PRE) {
+    if (p.resid)
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (threadIdx.x + i * THREADS < nvec) load_v<float, VEC>(p.resid + row * dim + (threadIdx.x + i * THREADS) * VEC, res[i]);
+  }
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -80,7 +100,12 @@ __global__ void __launch_bounds__(THREADS) gated_norm_add_kernel(const GatedNorm
     if (p.gate) {
       float g[VEC], b[VEC];
       load_v<float, VEC>(p.gate + row * p.gate_ld + v * VEC, g);
-      load_v<T, VEC>(bias + v * VEC, b);
+      if constexpr (PRE) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) b[e] = cb[i][e];
+      } else {
+        load_v<T, VEC>(bias + v * VEC, b);
+      }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) t[i][e] *= sigmoid_f(g[e] + b[e]);
     }
@@ -96,13 +121,23 @@ __global__ void __launch_bounds__(THREADS) gated_norm_add_kernel(const GatedNorm
     if (v >= nvec) continue;
     if (wpost) {
       float w[VEC];
-      load_v<T, VEC>(wpost + v * VEC, w);
+      if constexpr (PRE) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) w[e] = cp[i][e];
+      } else {
+        load_v<T, VEC>(wpost + v * VEC, w);
+      }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) t[i][e] *= inv * w[e];
     }
     if (p.resid) {
       float r[VEC];
-      load_v<float, VEC>(p.resid + row * dim + v * VEC, r);
+      if constexpr (PRE) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) r[e] = res[i][e];
+      } else {
+        load_v<float, VEC>(p.resid + row * dim + v * VEC, r);
+      }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) t[i][e] += r[e];
     }
@@ -127,16 +162,21 @@ __global__ void __launch_bounds__(THREADS) gated_norm_add_kernel(const GatedNorm
     const int v = threadIdx.x + i * THREADS;
     if (v >= nvec) continue;
     float w[VEC];
-    load_v<T, VEC>(wnext + v * VEC, w);
+    if constexpr (PRE) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) w[e] = cn[i][e];
+    } else {
+      load_v<T, VEC>(wnext + v * VEC, w);
+    }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) w[e] *= t[i][e] * inv;
     store_v<T, VEC>(out + v * VEC, w);
   }
 }
 
-template <typename T, int VEC, int NV, int THREADS>
+template <typename T, int VEC, int NV, int THREADS, bool PRE = false>
 int launch(const GatedNormParams& p, int64_t rows, cudaStream_t st) {
-  LRI_CUDA(launch_pdl(gated_norm_add_kernel<T, VEC, NV, THREADS>, dim3(static_cast<unsigned>(rows)), dim3(THREADS), 0, st, p));
+  LRI_CUDA(launch_pdl(gated_norm_add_kernel<T, VEC, NV, THREADS, PRE>, dim3(static_cast<unsigned>(rows)), dim3(THREADS), 0, st, p));
   LRI_LAUNCH_CHECK("gated_norm_add_kernel");
   return LRI_OK;
 }
@@ -154,8 +194,8 @@ int dispatch(const GatedNormParams& p, int64_t rows, cudaStream_t st) {
   }
   const int nvec = p.dim / 8;
   if (rows <= 16 && nvec > 256) {  // few rows: the kernel is one thread's latency chain, spread the row
-    if (nvec <= 512) return launch<T, 8, 1, 512>(p, rows, st);
-    if (nvec <= 1024) return launch<T, 8, 1, 1024>(p, rows, st);
+    if (nvec <= 512) return launch<T, 8, 1, 512, true>(p, rows, st);
+    if (nvec <= 1024) return launch<T, 8, 1, 1024, true>(p, rows, st);
     return launch<T, 8, 2, 1024>(p, rows, st);
   }
   if (nvec <= 128) return launch<T, 8, 1, 128>(p, rows, st);

@@ -4,29 +4,15 @@
 //   S_t[c, e] = f_t[c] S_{t-1}[c, e] + (1 - f_t[c]) v_t[e]
 //   o_t[e] = sum_c q_t[c] S_t[c, e]                         then RMSNorm over e, one weight for all heads
 //
-// The projections arrive in fp32; gates, state and sums stay fp32.  The state of sequence b and head h is
+// Here the token-by-token form: single tokens, short portions, fp32 models and sizes the block form does not take.
+// The projections arrive in fp32; gates, state and sums stay fp32, v is taken in the storage type.  The state of sequence b and head h is
 // [C, E] in `state`; a call whose first position is 0 starts from zero, any other continues what the previous call left.
-#include "linear.cuh"
+#include "hgrn2.cuh"
 
 namespace lri {
 namespace {
 
 constexpr int kWarps = 8;
-
-struct Hgrn2Params {
-  const float* proj;  // [B * S, ld]: q_raw at q_off, f_raw at f_off, v at v_off
-  int64_t ld, q_off, f_off, v_off;
-  const void* f_bias;  // [H * C]
-  const void* lower;   // [H * C]
-  const void* norm_w;  // [E]
-  float eps;
-  float* state;        // [B_max, H, C, E]
-  const void* input_pos;
-  int pos_is_i64;
-  void* out;     // [B * S, H * E]
-  float* o_raw;  // [B * S, H * E] when the columns of a head are cut over CTAs, else NULL
-  int S, H, C, E;
-};
 
 // Grid (column slices, heads, sequences).  A warp owns the state rows c = warp, warp + 8, ... and its lanes the
 // columns of the slice, VEC each; the rows of a thread stay in registers over all tokens of the call.
@@ -66,13 +52,12 @@ __global__ void __launch_bounds__(kWarps * 32) hgrn2_steps_kernel(const Hgrn2Par
     const float* pr = p.proj + row * p.ld;
     for (int c = threadIdx.x; c < C; c += kWarps * 32) {
       qs[c] = silu_f(pr[p.q_off + h * C + c]);
-      const float low = Num<T>::to_f(lower[c]);
-      fs[c] = low + (1.0f - low) * sigmoid_f(pr[p.f_off + h * C + c] + Num<T>::to_f(bias[c]));
+      fs[c] = forget_gate(pr[p.f_off + h * C + c], Num<T>::to_f(bias[c]), Num<T>::to_f(lower[c]));
     }
     float v[VEC], o[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
-      v[e] = live ? pr[p.v_off + h * E + e0 + e] : 0.f;
+      v[e] = live ? rnd<T>(pr[p.v_off + h * E + e0 + e]) : 0.f;
       o[e] = 0.f;
     }
     __syncthreads();
@@ -198,9 +183,11 @@ constexpr int kMaxChannels = 512;
 using namespace lri;
 
 extern "C" size_t lri_hgrn2_workspace_bytes(int dtype, int B, int S, int heads, int dim, int vdim) {
-  (void)dtype, (void)dim;
-  if (B <= 0 || S <= 0 || heads <= 0 || vdim <= 0) return 0;
-  return static_cast<size_t>(B) * S * heads * vdim * sizeof(float);
+  (void)dtype;
+  if (B <= 0 || S <= 0 || heads <= 0 || dim <= 0 || vdim <= 0) return 0;
+  const size_t raw = static_cast<size_t>(B) * S * heads * vdim * sizeof(float);
+  const size_t blocks = hgrn2_blocks_workspace_bytes(B, S, heads, dim, vdim);
+  return raw > blocks ? raw : blocks;
 }
 
 extern "C" int lri_hgrn2(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t f_off, int64_t v_off,
@@ -223,6 +210,7 @@ extern "C" int lri_hgrn2(int dtype, const float* proj, int64_t ld, int64_t q_off
   p.input_pos = input_pos, p.pos_is_i64 = pos_is_i64, p.out = out, p.o_raw = static_cast<float*>(workspace);
   p.S = S, p.H = heads, p.C = dim, p.E = vdim;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (option(OPT_HGRN2_BLOCKS) && hgrn2_blocks_supports(dtype, p, B)) return hgrn2_blocks_launch(dtype, p, B, workspace, st);
   if (dtype == LRI_BF16) return steps<__nv_bfloat16>(p, B, st);
   if (dtype == LRI_FP16) return steps<__half>(p, B, st);
   return steps<float>(p, B, st);

@@ -8,12 +8,14 @@
 //                    are expanded to per-head keys and values by one projection)
 //   head_linear      per-head matrices: q^T W_uk (the query in latent coordinates) and W_uv o (single-token form: scores
 //                    and sums run on the cached latents themselves)
-//   window_attention softmax attention over a sliding window for either form, any size and type
+//   window_attention softmax attention over a sliding window for either form: tcgen05 for prompt portions
+//                    (latent_attention_tc.cu), mma.sync for single tokens (latent_decode.cu), and here the plain kernel
+//                    for any size and type
+#include "latent_attention.cuh"
 #include "linear.cuh"
 
 namespace lri {
 
-// tcgen05 form of the prompt attention (latent_attention_tc.cu)
 namespace {
 
 // ---- rotation, norm, cache write ---------------------------------------------------------------------
@@ -33,6 +35,7 @@ struct PrepareParams {
   void* cache;  // [B, smax, r + dr]
   int64_t smax;
   int S, H, dn, dr, r;
+  int vec;  // 8-element accesses of q are aligned
 };
 
 // Grid (rows, 1 + head groups): slice 0 writes the cache row, the others 8 heads of q each.
@@ -64,6 +67,32 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const PrepareParams
     return;
   }
   const int h0 = (blockIdx.y - 1) * 8, h1 = min(h0 + 8, p.H);
+  if (p.vec) {
+    // items of 8 unrotated elements, then of 4 rotated pairs
+    const int plain = p.dn >> 3, per_head = plain + (half >> 2);
+    for (int i = threadIdx.x; i < (h1 - h0) * per_head; i += 256) {
+      const int h = h0 + i / per_head, u = i % per_head;
+      const float* q = pr + p.q_off + static_cast<int64_t>(h) * (p.dn + p.dr);
+      if (u < plain) {
+        float f[8];
+        load8<float>(q + u * 8, f);
+        store8<T>(static_cast<T*>(p.qn) + row * p.qn_row + h * p.qn_head + u * 8, f);
+        continue;
+      }
+      const int e = (u - plain) * 4;
+      T* qr = static_cast<T*>(p.qr) + row * p.qr_row + h * p.qr_head;
+      const float4 x = *reinterpret_cast<const float4*>(q + p.dn + e), y = *reinterpret_cast<const float4*>(q + p.dn + half + e);
+      const float4 t0 = *reinterpret_cast<const float4*>(cs + 2 * e), t1 = *reinterpret_cast<const float4*>(cs + 2 * e + 4);
+      const float a[4] = {x.x, x.y, x.z, x.w}, b2[4] = {y.x, y.y, y.z, y.w};
+      const float c[4] = {t0.x, t0.z, t1.x, t1.z}, sn[4] = {t0.y, t0.w, t1.y, t1.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        qr[e + j] = Num<T>::from_f(a[j] * c[j] - b2[j] * sn[j]);
+        qr[half + e + j] = Num<T>::from_f(b2[j] * c[j] + a[j] * sn[j]);
+      }
+    }
+    return;
+  }
   for (int h = h0 + (threadIdx.x >> 5); h < h1; h += 8) {
     const int lane = threadIdx.x & 31;
     const float* q = pr + p.q_off + static_cast<int64_t>(h) * (p.dn + p.dr);
@@ -144,26 +173,137 @@ __global__ void __launch_bounds__(256) head_linear_generic_kernel(const HeadLine
   if (lane == 0) (static_cast<T*>(p.y) + row * p.y_row + h * p.y_head)[j] = Num<T>::from_f(acc);
 }
 
-// ---- attention over a sliding window, any size ---------------------------------------------------------------
-struct WindowParams {
-  const void* q;  // [d1 | d2] at q + row * q_row + head * q_head
-  int64_t q_row, q_head;
-  const void* k;  // d1 elements at k + b * k_batch + j * k_row + head * k_head
-  int64_t k_batch, k_row, k_head;
-  const void* k2;  // d2 elements at k2 + b * k2_batch + j * k2_row, shared by the heads
-  int64_t k2_batch, k2_row;
-  const void* v;  // dv elements
-  int64_t v_batch, v_row, v_head;
-  void* out;  // [rows, H * dv]
-  const void* input_pos;
-  int pos_is_i64;
-  int history;  // key row j holds position pos0 - history + j; history < 0: position j
-  int64_t k_rows;
-  int64_t window;
-  float scale;
-  int S, H, d1, d2, dv;
-};
+// transposed, 16-byte loads: a CTA owns 64 outputs of a head; 8 threads cover them with 8 outputs each, the 32 thread groups
+// take the inputs i = group, group + 32, ...; M rows share the weights.  The weights of the first four inputs of a thread are requested
+// before the wait for the preceding kernel.
+template <typename T, int M>
+__global__ void __launch_bounds__(256) head_linear_t_kernel(const HeadLinearParams p) {
+  __shared__ float red[8][M][64];
+  const int h = blockIdx.y, cg = threadIdx.x & 7, ig = threadIdx.x >> 3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int j0 = blockIdx.x * 64 + cg * 8;
+  const int64_t row0 = static_cast<int64_t>(blockIdx.z) * M;
+  const T* w = static_cast<const T*>(p.w) + static_cast<int64_t>(h) * p.in * p.out + j0;
+  const bool live = j0 < p.out;
+  uint4 wv[4];
+  auto load_w = [&](int i0) {
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int i = i0 + ig + 32 * u;
+      wv[u] = live && i < p.in ? ld_stream16(w + static_cast<int64_t>(i) * p.out) : make_uint4(0, 0, 0, 0);
+    }
+  };
+  load_w(0);
+  pdl_launch_dependents();
+  pdl_wait();
+  const T* x = static_cast<const T*>(p.x) + row0 * p.x_row + h * p.x_head;
+  float acc[M][8] = {};
+  for (int i0 = 0; i0 < p.in; i0 += 128) {
+    if (i0 > 0) load_w(i0);
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int i = i0 + ig + 32 * u;
+      if (i >= p.in) break;
+      float f[8];
+      unpack8<T>(wv[u], f);
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        const float xv = row0 + m < p.rows ? Num<T>::to_f(x[m * p.x_row + i]) : 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[m][e] = fmaf(f[e], xv, acc[m][e]);
+      }
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < M; ++m)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float v = acc[m][e];
+      v += __shfl_xor_sync(0xffffffffu, v, 8);
+      v += __shfl_xor_sync(0xffffffffu, v, 16);
+      if (lane < 8) red[warp][m][cg * 8 + e] = v;
+    }
+  __syncthreads();
+  for (int i = threadIdx.x; i < M * 64; i += 256) {
+    const int m = i >> 6, c = i & 63;
+    if (row0 + m >= p.rows || blockIdx.x * 64 + c >= p.out) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int wi = 0; wi < 8; ++wi) v += red[wi][m][c];
+    (static_cast<T*>(p.y) + (row0 + m) * p.y_row + h * p.y_head)[blockIdx.x * 64 + c] = Num<T>::from_f(v);
+  }
+}
 
+// rows of W contiguous, 16-byte loads: a warp owns 4 outputs of a head, its lanes 8 inputs each per step
+template <typename T, int M>
+__global__ void __launch_bounds__(256) head_linear_kernel(const HeadLinearParams p) {
+  const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int j0 = blockIdx.x * 32 + warp * 4;
+  const int64_t row0 = static_cast<int64_t>(blockIdx.z) * M;
+  const T* w = static_cast<const T*>(p.w) + static_cast<int64_t>(h) * p.out * p.in;
+  uint4 wv[2][4];
+  auto load_w = [&](int i0) {
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = i0 + u * 256 + lane * 8;
+#pragma unroll
+      for (int r = 0; r < 4; ++r)
+        wv[u][r] = j0 + r < p.out && i < p.in ? ld_stream16(w + static_cast<int64_t>(j0 + r) * p.in + i) : make_uint4(0, 0, 0, 0);
+    }
+  };
+  load_w(0);
+  pdl_launch_dependents();
+  pdl_wait();
+  const T* x = static_cast<const T*>(p.x) + row0 * p.x_row + h * p.x_head;
+  float acc[M][4] = {};
+  for (int i0 = 0; i0 < p.in; i0 += 512) {
+    if (i0 > 0) load_w(i0);
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = i0 + u * 256 + lane * 8;
+      if (i >= p.in) break;
+      float xf[M][8];
+#pragma unroll
+      for (int m = 0; m < M; ++m) load8<T>(x + (row0 + m < p.rows ? m : 0) * p.x_row + i, xf[m]);
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        float f[8];
+        unpack8<T>(wv[u][r], f);
+#pragma unroll
+        for (int m = 0; m < M; ++m)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc[m][r] = fmaf(f[e], xf[m][e], acc[m][r]);
+      }
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < M; ++m)
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+      const float v = warp_sum(acc[m][r]);
+      if (lane == 0 && row0 + m < p.rows && j0 + r < p.out)
+        (static_cast<T*>(p.y) + (row0 + m) * p.y_row + h * p.y_head)[j0 + r] = Num<T>::from_f(v);
+    }
+}
+
+template <typename T, int M>
+int launch_head_linear(const HeadLinearParams& p, int heads, bool transposed, cudaStream_t st) {
+  const unsigned h = static_cast<unsigned>(heads), z = static_cast<unsigned>((p.rows + M - 1) / M);
+  if (transposed)
+    LRI_CUDA(launch_pdl(head_linear_t_kernel<T, M>, dim3((p.out + 63) / 64, h, z), dim3(256), 0, st, p));
+  else
+    LRI_CUDA(launch_pdl(head_linear_kernel<T, M>, dim3((p.out + 31) / 32, h, z), dim3(256), 0, st, p));
+  LRI_LAUNCH_CHECK("head_linear_kernel");
+  return LRI_OK;
+}
+template <typename T>
+int head_linear(const HeadLinearParams& p, int heads, bool transposed, cudaStream_t st) {
+  if (p.rows <= 1) return launch_head_linear<T, 1>(p, heads, transposed, st);
+  if (p.rows <= 2) return launch_head_linear<T, 2>(p, heads, transposed, st);
+  return launch_head_linear<T, 4>(p, heads, transposed, st);
+}
+
+// ---- attention over a sliding window, any size ---------------------------------------------------------------
 // One warp per (token, head).  A lane scores one key at a time, then the warp adds the 32 keys' values, lanes over the
 // value columns.
 template <typename T, int NV>
@@ -274,6 +414,8 @@ extern "C" int lri_latent_prepare(int dtype, const float* proj, int64_t ld, int6
   p.table = rope_table, p.table_rows = table_rows, p.input_pos = input_pos, p.pos_is_i64 = pos_is_i64;
   p.qn = qn, p.qn_row = qn_row, p.qn_head = qn_head, p.qr = qr, p.qr_row = qr_row, p.qr_head = qr_head;
   p.cache = cache, p.smax = smax, p.S = S, p.H = heads, p.dn = dim, p.dr = rot_dim, p.r = rank;
+  p.vec = dim % 8 == 0 && rot_dim % 8 == 0 && ld % 8 == 0 && q_off % 8 == 0 && qn_row % 8 == 0 && qn_head % 8 == 0 && aligned16(proj) &&
+          aligned16(qn) && aligned16(rope_table);
   LRI_CUDA(launch_pdl(LRI_BY_TYPE(dtype, latent_prepare_kernel), dim3(static_cast<unsigned>(rows), 1 + (heads + 7) / 8), dim3(256), 0,
                       static_cast<cudaStream_t>(stream), p));
   LRI_LAUNCH_CHECK("latent_prepare_kernel");
@@ -315,6 +457,9 @@ extern "C" int lri_head_linear(int dtype, const void* x, int64_t x_row, int64_t 
   p.x = x, p.x_row = x_row, p.x_head = x_head, p.w = w, p.y = y, p.y_row = y_row, p.y_head = y_head;
   p.rows = static_cast<int>(rows), p.in = in, p.out = out;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dtype != LRI_FP32 && in % 8 == 0 && out % 8 == 0 && x_row % 8 == 0 && x_head % 8 == 0 && aligned16(x) && aligned16(w))
+    return dtype == LRI_BF16 ? head_linear<__nv_bfloat16>(p, heads, transposed != 0, st)
+                             : head_linear<__half>(p, heads, transposed != 0, st);
   const unsigned h = static_cast<unsigned>(heads), m = static_cast<unsigned>(rows);
   if (transposed)
     LRI_CUDA(launch_pdl(LRI_BY_TYPE(dtype, head_linear_t_generic_kernel), dim3((out + 127) / 128, h, m), dim3(128), 0, st, p));
@@ -324,11 +469,16 @@ extern "C" int lri_head_linear(int dtype, const void* x, int64_t x_row, int64_t 
   return LRI_OK;
 }
 
+extern "C" size_t lri_window_attention_scratch_bytes(int B, int heads, int dv, int64_t keys) {
+  return B > 0 && heads > 0 && dv > 0 && keys > 0 ? latent_decode_scratch_bytes(B, heads, dv, keys) : 0;
+}
+
 extern "C" int lri_window_attention(int dtype, const void* q, int64_t q_row, int64_t q_head, const void* k, int64_t k_batch,
                                     int64_t k_row, int64_t k_head, const void* k2, int64_t k2_batch, int64_t k2_row, const void* v,
                                     int64_t v_batch, int64_t v_row, int64_t v_head, void* out, const void* input_pos,
                                     int pos_is_i64, int history, int64_t k_rows, int64_t window_size, float scale, int B, int S,
-                                    int heads, int d1, int d2, int dv, lri_stream_t stream) {
+                                    int heads, int d1, int d2, int dv, void* scratch, size_t scratch_bytes,
+                                    lri_stream_t stream) {
   LRI_REQUIRE(dtype_ok(dtype), LRI_ERR_UNSUPPORTED, "window_attention: dtype %d", dtype);
   LRI_REQUIRE(q && k && k2 && v && out && input_pos, LRI_ERR_ARG, "window_attention: NULL pointer");
   LRI_REQUIRE(B >= 0 && S >= 0 && heads > 0 && d1 > 0 && d2 >= 0 && dv > 0 && k_rows > 0 && window_size > 0, LRI_ERR_ARG,
@@ -342,6 +492,10 @@ extern "C" int lri_window_attention(int dtype, const void* q, int64_t q_row, int
   p.out = out, p.input_pos = input_pos, p.pos_is_i64 = pos_is_i64, p.history = history, p.k_rows = k_rows;
   p.window = window_size, p.scale = scale, p.S = S, p.H = heads, p.d1 = d1, p.d2 = d2, p.dv = dv;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (option(OPT_WINDOW_TC)) {
+    if (latent_decode_supports(dtype, p)) return latent_decode_launch(dtype, p, B, scratch, scratch_bytes, st);
+    if (window_attention_tc_supports(dtype, p, B)) return window_attention_tc_launch(dtype, p, B, st);
+  }
   if (dtype == LRI_BF16) return window<__nv_bfloat16>(p, rows, st);
   if (dtype == LRI_FP16) return window<__half>(p, rows, st);
   return window<float>(p, rows, st);

@@ -16,6 +16,7 @@ bool gemm_tcgen05_supports(int64_t m, int n, int k);
 int gemm_tcgen05_launch(int dtype, const void* a, const void* w, void* c, int64_t m, int n, int k, cudaStream_t st);
 int gemm_tcgen05_status_read_and_clear(int* status_out);
 int attn_prefill_tc_status_read_and_clear(int* status_out);
+int window_attention_tc_status_read_and_clear(int* status_out);
 bool gemm_tcgen05_fused_supports(int epi, const LinearParams& p, int64_t m);
 int gemm_tcgen05_fused_launch(int dtype, int epi, const LinearParams& p, int64_t m, cudaStream_t st);
 
@@ -46,6 +47,8 @@ const OptionSpec kOptionSpecs[OPT_COUNT] = {
     {"gemm_reserve_sms", "LRI_GEMM_RESERVE_SMS", 0, 0, 64},
     {"attn_head_tile", "LRI_ATTN_HEAD_TILE", 0, 0, 4},
     {"moe_stream_pairs", "LRI_MOE_STREAM_PAIRS", 32, 0, 65535},
+    {"window_tc", "LRI_WINDOW_TC", 1, 0, 1},
+    {"hgrn2_blocks", "LRI_HGRN2_BLOCKS", 1, 0, 1},
 };
 
 bool option_value_ok(int which, int v) {
@@ -332,6 +335,10 @@ extern "C" int lri_gemm_status(void) {
   if (rc != LRI_OK) return rc;
   if (v != 0 || v2 != 0)
     return fail(LRI_ERR_TIMEOUT, "tcgen05 GEMM: a bounded mbarrier wait gave up (site %d)", v != 0 ? v : v2);
+  if (v3 == 0) {
+    rc = window_attention_tc_status_read_and_clear(&v3);
+    if (rc != LRI_OK) return rc;
+  }
   if (v3 != 0) return fail(LRI_ERR_TIMEOUT, "tcgen05 prefill attention: a bounded mbarrier wait gave up (site %d)", v3);
   return LRI_OK;
 }

@@ -59,7 +59,7 @@ moe_route_kernel(const float* logits, int64_t ld, int experts, int top, int64_t 
 
 // One CTA: tile list and first packed row of every expert from the counts, which are left at zero.
 __global__ void __launch_bounds__(1024)
-moe_plan_kernel(int experts, int32_t* counts, int32_t* first_row, int32_t* tiles) {
+moe_plan_kernel(int experts, int max_tiles, int32_t* counts, int32_t* first_row, int32_t* tiles) {
   __shared__ int scan[kMaxExperts];
   pdl_launch_dependents();
   pdl_wait();
@@ -77,20 +77,21 @@ moe_plan_kernel(int experts, int32_t* counts, int32_t* first_row, int32_t* tiles
   if (e < experts) {
     counts[e] = 0;
     first_row[e] = t0 * kTileRows;
-    for (int t = 0; t < mine; ++t) tiles[1 + t0 + t] = e;
+    for (int t = 0; t < mine && t0 + t < max_tiles; ++t) tiles[1 + t0 + t] = e;
   }
-  if (e == kMaxExperts - 1) tiles[0] = scan[e];
+  if (e == kMaxExperts - 1) tiles[0] = scan[e] < max_tiles ? scan[e] : max_tiles;
 }
 
 // One CTA per pair: packed row, its scale, and where the combine step finds the pair's result.
 __global__ void __launch_bounds__(128)
 moe_gather_kernel(const uint4* x, int vecs, int top, const int32_t* ids,
                   const float* scores, const int32_t* rank, const int32_t* first_row,
-                  uint4* packed, float* row_scale, int32_t* slots) {
+                  int64_t packed_rows, uint4* packed, float* row_scale, int32_t* slots) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t pair = blockIdx.x;
   const int64_t dst = first_row[ids[pair]] + rank[pair];
+  if (dst < 0 || dst >= packed_rows) return;  // ranks of another call: nothing is written outside the buffers
   const uint4* src = x + (pair / top) * vecs;
   for (int v = threadIdx.x; v < vecs; v += 128) packed[dst * vecs + v] = src[v];
   if (threadIdx.x == 0) {
@@ -178,7 +179,7 @@ extern "C" int lri_moe_route(const float* logits, int64_t ld, int experts, int t
 
 extern "C" int lri_moe_pack(int dtype, const void* x, int64_t rows, int dim, int top, int experts, const int32_t* ids,
                             const float* scores, const int32_t* rank, int32_t* counts, int32_t* first_row, int32_t* tiles,
-                            void* packed, float* row_scale, int32_t* slots, lri_stream_t stream) {
+                            int64_t max_tiles, void* packed, float* row_scale, int32_t* slots, lri_stream_t stream) {
   LRI_REQUIRE(dtype == LRI_BF16 || dtype == LRI_FP16, LRI_ERR_UNSUPPORTED, "moe_pack: dtype %d", dtype);
   LRI_REQUIRE(x && ids && scores && rank && counts && first_row && tiles && packed && row_scale && slots, LRI_ERR_ARG,
               "moe_pack: NULL pointer");
@@ -186,11 +187,14 @@ extern "C" int lri_moe_pack(int dtype, const void* x, int64_t rows, int dim, int
               "moe_pack: dim=%d must be a multiple of 8 and the rows 16-byte aligned", dim);
   LRI_REQUIRE(experts >= 1 && experts <= kMaxExperts, LRI_ERR_UNSUPPORTED, "moe_pack: %d experts", experts);
   LRI_REQUIRE(rows > 0 && rows * top < (1ll << 31), LRI_ERR_ARG, "moe_pack: rows=%lld", (long long)rows);
+  LRI_REQUIRE(max_tiles >= lri_moe_max_tiles(rows, top, experts), LRI_ERR_ARG, "moe_pack: room for %lld tiles, %lld needed",
+              (long long)max_tiles, (long long)lri_moe_max_tiles(rows, top, experts));
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  LRI_CUDA(launch_pdl(moe_plan_kernel, dim3(1), dim3(kMaxExperts), 0, st, experts, counts, first_row, tiles));
+  LRI_CUDA(launch_pdl(moe_plan_kernel, dim3(1), dim3(kMaxExperts), 0, st, experts,
+                      static_cast<int>(max_tiles), counts, first_row, tiles));
   LRI_LAUNCH_CHECK("moe_plan_kernel");
   LRI_CUDA(launch_pdl(moe_gather_kernel, dim3(static_cast<unsigned>(rows * top)), dim3(128), 0, st,
-                      static_cast<const uint4*>(x), dim / 8, top, ids, scores, rank, first_row, static_cast<uint4*>(packed),
+                      static_cast<const uint4*>(x), dim / 8, top, ids, scores, rank, first_row, max_tiles * kTileRows, static_cast<uint4*>(packed),
                       row_scale, slots));
   LRI_LAUNCH_CHECK("moe_gather_kernel");
   return LRI_OK;

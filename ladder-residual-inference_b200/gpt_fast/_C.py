@@ -84,7 +84,9 @@ _SIGNATURES = {
                                 c_int, c_int, c_int, c_void_p]),
     "lri_window_attention": (c_int, [c_int, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, c_int64, c_void_p,
                                      c_int64, c_int64, c_void_p, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_int,
-                                     c_int, c_int64, c_int64, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+                                     c_int, c_int64, c_int64, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_size_t,
+                                     c_void_p]),
+    "lri_window_attention_scratch_bytes": (c_size_t, [c_int, c_int, c_int, c_int64]),
     "lri_hgrn2_workspace_bytes": (c_size_t, [c_int, c_int, c_int, c_int, c_int, c_int]),
     "lri_hgrn2": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_float,
                           c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_size_t,
@@ -93,7 +95,7 @@ _SIGNATURES = {
     "lri_moe_max_tiles": (c_int64, [c_int64, c_int, c_int]),
     "lri_moe_route": (c_int, [c_void_p, c_int64, c_int, c_int, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
     "lri_moe_pack": (c_int, [c_int, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
+                             c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p]),
     "lri_moe_gateup": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_void_p, c_void_p,
                                c_int64, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p]),
     "lri_moe_down": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int,

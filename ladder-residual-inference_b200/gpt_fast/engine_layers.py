@@ -55,10 +55,14 @@ class LayerEngine(Engine):
             self.win_latent = buf(rows, max(m.rank for m in latent))
             self.win_rot = buf(rows, max(m.rot_dim for m in latent))
             self.win_kv = buf(rows, max(m.heads * (m.dim + m.vdim) for m in latent))
+            # fewer sequences are cut into more splits: the largest batch is not the largest scratch
+            size = max(ops.window_attention_scratch_bytes(b, m.heads, m.rank, min(m.window, max_seq))
+                       for m in latent for b in range(1, max_batch + 1))
+            self.attn_scratch = torch.empty(max(size, 16), dtype=torch.uint8, device=device)
             self.ws_expand = workspace(ops.linear_workspace_bytes, self.win_kv.shape[1])
         if hgrn:
-            size = max(max(ops.hgrn2_workspace_bytes(dtype, max_batch, s, m.heads, m.dim, m.vdim) for s in (1, max_seq))
-                       for m in hgrn)
+            size = max(ops.hgrn2_workspace_bytes(dtype, b, max_seq, m.heads, m.dim, m.vdim)
+                       for m in hgrn for b in range(1, max_batch + 1))
             self.ws_hgrn = torch.empty(max(size, 16), dtype=torch.uint8, device=device)
         if moes:
             def most(f):
@@ -100,7 +104,7 @@ class LayerEngine(Engine):
             ops.head_linear(self.q, (H * dn, dn), w_k, True, ql, (H * row_len, row_len), B, H, dn, r)
             ops.window_attention(ql, (H * row_len, row_len), cache, (smax * row_len, row_len, 0), cache.view(-1)[r:],
                                  (smax * row_len, row_len), cache, (smax * row_len, row_len, 0), ol, pos, -1, smax,
-                                 m.window, m.scale, B, 1, H, r, dr, r)
+                                 m.window, m.scale, B, 1, H, r, dr, r, self.attn_scratch)
             ops.head_linear(ol, (H * r, r), w_v, False, self.y, (H * dv, dv), B, H, r, dv)
             return
         # prompt portion: the visible latents are expanded to per-head keys and values
@@ -133,7 +137,7 @@ class LayerEngine(Engine):
         tiles = ops.moe_max_tiles(rows, m.top, m.experts)
         ops.moe_route(logits, self.ld, m.experts, m.top, rows, self.moe_ids, self.moe_scores, self.moe_counts, self.moe_rank)
         ops.moe_pack(self.normed, rows, m.top, m.experts, self.moe_ids, self.moe_scores, self.moe_rank, self.moe_counts,
-                     self.moe_first, self.moe_tiles, self.moe_packed, self.moe_scale, self.moe_slots)
+                     self.moe_first, self.moe_tiles, tiles, self.moe_packed, self.moe_scale, self.moe_slots)
         ops.moe_gateup(self.moe_packed, m.w1, self.moe_hidden, None, None, pairs, m.top, m.glu, tiles=self.moe_tiles,
                        row_scale=self.moe_scale, max_tiles=tiles)
         ops.moe_down(self.moe_hidden, m.w2, self.moe_out, None, pairs, tiles=self.moe_tiles, max_tiles=tiles)

@@ -191,13 +191,18 @@ class CudaOps:
 
     @staticmethod
     def window_attention(q, q_pitch, k, k_pitch, k2, k2_pitch, v, v_pitch, out, input_pos, history, k_rows, window, scale, B,
-                         S, heads, d1, d2, dv):
+                         S, heads, d1, d2, dv, scratch=None):
         """q_pitch (row, head); k_pitch, v_pitch (batch, row, head); k2_pitch (batch, row), in elements."""
         _C.require_cuda(q, k, k2, v, out, input_pos)
         _C.check(_C.lib.lri_window_attention(
             _C.dtype_code_any(q.dtype), q.data_ptr(), *q_pitch, k.data_ptr(), *k_pitch, k2.data_ptr(), *k2_pitch,
             v.data_ptr(), *v_pitch, out.data_ptr(), input_pos.data_ptr(), int(input_pos.dtype == torch.int64), history,
-            k_rows, window, float(scale), B, S, heads, d1, d2, dv, _C.stream_handle()))
+            k_rows, window, float(scale), B, S, heads, d1, d2, dv, _C.ptr(scratch),
+            scratch.numel() * scratch.element_size() if scratch is not None else 0, _C.stream_handle()))
+
+    @staticmethod
+    def window_attention_scratch_bytes(B, heads, dv, keys):
+        return _C.lib.lri_window_attention_scratch_bytes(B, heads, dv, keys)
 
     # ---- recurrence ----------------------------------------------------------------------------------------
     @staticmethod
@@ -230,11 +235,11 @@ class CudaOps:
                                       _C.ptr(counts), _C.ptr(rank), _C.stream_handle()))
 
     @staticmethod
-    def moe_pack(x, rows, top, experts, ids, scores, rank, counts, first_row, tiles, packed, row_scale, slots):
+    def moe_pack(x, rows, top, experts, ids, scores, rank, counts, first_row, tiles, max_tiles, packed, row_scale, slots):
         _C.require_cuda(x, packed)
         _C.check(_C.lib.lri_moe_pack(_C.dtype_code(x.dtype), x.data_ptr(), rows, x.shape[-1], top, experts, ids.data_ptr(),
                                      scores.data_ptr(), rank.data_ptr(), counts.data_ptr(), first_row.data_ptr(),
-                                     tiles.data_ptr(), packed.data_ptr(), row_scale.data_ptr(), slots.data_ptr(),
+                                     tiles.data_ptr(), max_tiles, packed.data_ptr(), row_scale.data_ptr(), slots.data_ptr(),
                                      _C.stream_handle()))
 
     @staticmethod
