@@ -78,14 +78,23 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
                : "memory");
 }
 
+// Gates by the special-function unit: a few units in the last place of fp32.
+__device__ __forceinline__ float gate(float raw, float bias, float low) {
+  return low + (1.0f - low) * __fdividef(1.0f, 1.0f + __expf(-(raw + bias)));
+}
+__device__ __forceinline__ float silu(float x) { return x * __fdividef(1.0f, 1.0f + __expf(-x)); }
+
 template <int CP>
 struct Smem {
   static constexpr int kPitchC = CP + 8;      // bf16 rows of q", k"
   static constexpr int kPitchE = kMaxE + 8;   // bf16 rows of v
   static constexpr int kPitchA = kBlock + 8;  // bf16 rows of A
-  float raw[2][kBlock * (2 * CP + kMaxE)];    // q, f, v of a block as they arrive
-  float q[kBlock][CP], f[kBlock][CP];
-  float bias[CP], low[CP], F[CP];
+  alignas(16) float raw[2][kBlock * (2 * CP + kMaxE)];    // q, f, v of a block as they arrive
+  alignas(16) float q[kBlock][CP];
+  alignas(16) float f[kBlock][CP];
+  alignas(16) float bias[CP];
+  alignas(16) float low[CP];
+  alignas(16) float F[CP];
   float o[2][kBlock][kMaxE + 4];  // per half of the channels
   alignas(16) bf16 qd[kTerms][kBlock * kPitchC];
   alignas(16) bf16 kd[kTerms][kBlock * kPitchC];
@@ -123,19 +132,17 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
   pdl_launch_dependents();
   pdl_wait();
 
-  const int vc = C / 4, ve = E / 4, per_row = 2 * vc + ve;
+  // warp t works on token t of a block, a lane on 4 consecutive channels (or values)
+  const int x4 = lane * 4;
   auto fetch = [&](int s0, int buf) {
-    for (int i = tid; i < kBlock * per_row; i += kThreads) {
-      const int t = i / per_row, r = i - t * per_row;
-      if (s0 + t >= s_end) continue;
-      const float* row = p.proj + (static_cast<int64_t>(b) * p.S + s0 + t) * p.ld;
-      float* dst = sm.raw[buf] + t * (2 * CP + kMaxE);
-      if (r < vc) {
-        if (FULL) cp_async16(dst + r * 4, row + p.q_off + h * C + r * 4);
-      } else if (r < 2 * vc)
-        cp_async16(dst + CP + (r - vc) * 4, row + p.f_off + h * C + (r - vc) * 4);
-      else
-        cp_async16(dst + 2 * CP + (r - 2 * vc) * 4, row + p.v_off + h * E + (r - 2 * vc) * 4);
+    if (s0 + warp < s_end) {
+      const float* row = p.proj + (static_cast<int64_t>(b) * p.S + s0 + warp) * p.ld + x4;
+      float* dst = sm.raw[buf] + warp * (2 * CP + kMaxE) + x4;
+      if (x4 < C) {
+        if (FULL) cp_async16(dst, row + p.q_off + h * C);
+        cp_async16(dst + CP, row + p.f_off + h * C);
+      }
+      if (x4 < E) cp_async16(dst + 2 * CP, row + p.v_off + h * E);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -182,20 +189,32 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
     const float* raw = sm.raw[buf];
     if (s0 + kBlock < s_end) fetch(s0 + kBlock, buf ^ 1);
     // ---- gates, activations, v terms ----
-    for (int i = tid; i < kBlock * CP; i += kThreads) {
-      const int t = i / CP, c = i - t * CP;
-      float f = 1.f, q = 0.f;
-      if (c < C && s0 + t < s_end) {
-        f = forget_gate(raw[t * (2 * CP + kMaxE) + CP + c], sm.bias[c], sm.low[c]);
-        if (FULL) q = silu_f(raw[t * (2 * CP + kMaxE) + c]);
+    {
+      const bool in = s0 + warp < s_end;
+      const float* rw = raw + warp * (2 * CP + kMaxE) + x4;
+      if (x4 < CP) {
+        float4 f = make_float4(1.f, 1.f, 1.f, 1.f), q = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (in && x4 < C) {
+          const float4 fr = *reinterpret_cast<const float4*>(rw + CP);
+          const float4 bi = *reinterpret_cast<const float4*>(&sm.bias[x4]), lo = *reinterpret_cast<const float4*>(&sm.low[x4]);
+          f.x = gate(fr.x, bi.x, lo.x), f.y = gate(fr.y, bi.y, lo.y), f.z = gate(fr.z, bi.z, lo.z), f.w = gate(fr.w, bi.w, lo.w);
+          if (FULL) {
+            const float4 qr = *reinterpret_cast<const float4*>(rw);
+            q = make_float4(silu(qr.x), silu(qr.y), silu(qr.z), silu(qr.w));
+          }
+        }
+        *reinterpret_cast<float4*>(&sm.f[warp][x4]) = f;
+        if (FULL) *reinterpret_cast<float4*>(&sm.q[warp][x4]) = q;
       }
-      sm.f[t][c] = f;
-      if (FULL) sm.q[t][c] = q;
-    }
-    for (int i = tid; i < kBlock * E; i += kThreads) {
-      const int t = i / E, e = i - t * E;
-      split_store<kVTerms>(&sm.v[0][t * Smem<CP>::kPitchE + e], kBlock * Smem<CP>::kPitchE,
-                           s0 + t < s_end ? rnd<T>(raw[t * (2 * CP + kMaxE) + 2 * CP + e]) : 0.f);
+      if (x4 < E) {
+        const float4 x = in ? *reinterpret_cast<const float4*>(rw + 2 * CP) : make_float4(0.f, 0.f, 0.f, 0.f);
+        uint32_t lo[kTerms], hi[kTerms];
+        split2(rnd<T>(x.x), rnd<T>(x.y), lo);
+        split2(rnd<T>(x.z), rnd<T>(x.w), hi);
+#pragma unroll
+        for (int i = 0; i < kVTerms; ++i)
+          *reinterpret_cast<uint2*>(&sm.v[i][warp * Smem<CP>::kPitchE + x4]) = make_uint2(lo[i], hi[i]);
+      }
     }
     __syncthreads();
     // ---- running products: thread (channel, k" or q", first or last 8 tokens) ----
@@ -243,11 +262,13 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
         float x = 0.f;
         if (t >= s) {
 #pragma unroll
-          for (int j = 0; j < kPer; ++j) {
-            const int c = lane + 32 * j;
-            const float f = sm.f[t][c];
-            d[j] = t == s ? 1.f - f : d[j] * f;
-            x = fmaf(sm.q[t][c], d[j], x);
+          for (int j = 0; j < kPer; j += 2) {
+            const float2 f = *reinterpret_cast<const float2*>(&sm.f[t][lane * kPer + j]);
+            const float2 q = *reinterpret_cast<const float2*>(&sm.q[t][lane * kPer + j]);
+            d[j] = t == s ? 1.f - f.x : d[j] * f.x;
+            d[j + 1] = t == s ? 1.f - f.y : d[j + 1] * f.y;
+            x = fmaf(q.x, d[j], x);
+            x = fmaf(q.y, d[j + 1], x);
           }
         }
         a[t] = x;

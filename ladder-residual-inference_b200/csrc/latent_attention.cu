@@ -35,10 +35,11 @@ struct PrepareParams {
   void* cache;  // [B, smax, r + dr]
   int64_t smax;
   int S, H, dn, dr, r;
+  int heads_per_cta;
   int vec;  // 8-element accesses of q are aligned
 };
 
-// Grid (rows, 1 + head groups): slice 0 writes the cache row, the others 8 heads of q each.
+// Grid (rows, 1 + head groups): slice 0 writes the cache row, the others some heads of q each.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(const PrepareParams p) {
   __shared__ float part[33];
@@ -66,7 +67,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const PrepareParams
     }
     return;
   }
-  const int h0 = (blockIdx.y - 1) * 8, h1 = min(h0 + 8, p.H);
+  const int h0 = (blockIdx.y - 1) * p.heads_per_cta, h1 = min(h0 + p.heads_per_cta, p.H);
   if (p.vec) {
     // items of 8 unrotated elements, then of 4 rotated pairs
     const int plain = p.dn >> 3, per_head = plain + (half >> 2);
@@ -416,7 +417,10 @@ extern "C" int lri_latent_prepare(int dtype, const float* proj, int64_t ld, int6
   p.cache = cache, p.smax = smax, p.S = S, p.H = heads, p.dn = dim, p.dr = rot_dim, p.r = rank;
   p.vec = dim % 8 == 0 && rot_dim % 8 == 0 && ld % 8 == 0 && q_off % 8 == 0 && qn_row % 8 == 0 && qn_head % 8 == 0 && aligned16(proj) &&
           aligned16(qn) && aligned16(rope_table);
-  LRI_CUDA(launch_pdl(LRI_BY_TYPE(dtype, latent_prepare_kernel), dim3(static_cast<unsigned>(rows), 1 + (heads + 7) / 8), dim3(256), 0,
+  // many rows: one CTA takes the heads of a row (few rows: more CTAs, shorter chains)
+  p.heads_per_cta = rows >= 256 ? (heads < 64 ? heads : 64) : 8;
+  LRI_CUDA(launch_pdl(LRI_BY_TYPE(dtype, latent_prepare_kernel),
+                      dim3(static_cast<unsigned>(rows), 1 + (heads + p.heads_per_cta - 1) / p.heads_per_cta), dim3(256), 0,
                       static_cast<cudaStream_t>(stream), p));
   LRI_LAUNCH_CHECK("latent_prepare_kernel");
   return LRI_OK;

@@ -62,12 +62,15 @@ __global__ void __launch_bounds__(kThreads) latent_decode_kernel(const DecodePar
 
   const int vecs = p.row_len / 8;
   const T* qg = static_cast<const T*>(p.q) + b * p.q_row;
-  for (int i = threadIdx.x; i < kHeads * vecs; i += kThreads) {
-    const int h = i / vecs, v = i - h * vecs;
-    uint4 val = make_uint4(0, 0, 0, 0);
-    if (h0 + h < p.H) val = *reinterpret_cast<const uint4*>(qg + (h0 + h) * p.q_head + v * 8);
-    *reinterpret_cast<uint4*>(qs + h * pitch + v * 8) = val;
-  }
+  // (a warp copies whole rows; the wait for the first tile of keys covers the queries too)
+  for (int h = warp; h < kHeads; h += kWarps)
+    for (int v = lane; v < vecs; v += 32) {
+      T* dst = qs + h * pitch + v * 8;
+      if (h0 + h < p.H)
+        cp_async16(dst, qg + (h0 + h) * p.q_head + v * 8);
+      else
+        *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+    }
   if (threadIdx.x < kHeads) m_s[threadIdx.x] = -INFINITY, l_s[threadIdx.x] = 0.f;
   float acc[kMaxUnits][2][4];
 #pragma unroll
@@ -81,28 +84,44 @@ __global__ void __launch_bounds__(kThreads) latent_decode_kernel(const DecodePar
 
   for (int64_t t = t0; t < t1; ++t) {
     __syncthreads();  // the previous tile has been consumed (first pass: nothing)
-    for (int i = threadIdx.x; i < kKeys * vecs; i += kThreads) {
-      const int j = i / vecs, v = i - j * vecs;
+#pragma unroll
+    for (int i = 0; i < kKeys / kWarps; ++i) {
+      const int j = warp * (kKeys / kWarps) + i;
       const int64_t row = t * kKeys + j;
-      T* dst = ks + j * pitch + v * 8;
-      if (row <= hi)
-        cp_async16(dst, kg + row * p.row_len + v * 8);
-      else
-        *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+      T* dst = ks + j * pitch;
+      const T* src = kg + row * p.row_len;
+      for (int v = lane; v < vecs; v += 32) {
+        if (row <= hi)
+          cp_async16(dst + v * 8, src + v * 8);
+        else
+          *reinterpret_cast<uint4*>(dst + v * 8) = make_uint4(0, 0, 0, 0);
+      }
     }
     cp_async_wait_all();
     __syncthreads();
     // scores of 16 heads x this warp's 8 keys
     {
-      float c[4] = {0.f, 0.f, 0.f, 0.f};
+      float c[4] = {0.f, 0.f, 0.f, 0.f}, c2[4] = {0.f, 0.f, 0.f, 0.f};  // two chains of products
       const T* qa = qs + (lane & 15) * pitch + (lane >> 4) * 8;
-      const T* kb = ks + (warp * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 8;
-      for (int k = 0; k < p.row_len; k += 16) {
+      const T* kb = ks + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 8;
+      int k = 0;
+#pragma unroll 4
+      for (; k + 32 <= p.row_len; k += 32) {
+        uint32_t a[8], bb[4];
+        ldmatrix_x4(qa + k, a[0], a[1], a[2], a[3]);
+        ldmatrix_x4(qa + k + 16, a[4], a[5], a[6], a[7]);
+        ldmatrix_x4(kb + k, bb[0], bb[1], bb[2], bb[3]);
+        mma16816<T>(c, a[0], a[1], a[2], a[3], bb[0], bb[1]);
+        mma16816<T>(c2, a[4], a[5], a[6], a[7], bb[2], bb[3]);
+      }
+      if (k < p.row_len) {
         uint32_t a0, a1, a2, a3, b0, b1;
         ldmatrix_x4(qa + k, a0, a1, a2, a3);
-        ldmatrix_x2(kb + k, b0, b1);
+        ldmatrix_x2(ks + (warp * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 8 + k, b0, b1);
         mma16816<T>(c, a0, a1, a2, a3, b0, b1);
       }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) c[e] += c2[e];
       const int row = lane >> 2, col = warp * 8 + 2 * (lane & 3);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
