@@ -1,4 +1,5 @@
 """Patevik on the GPU: every mechanism alone and whole models against the plain oracle, in fp32 (sharp), bf16 and fp16."""
+import copy
 import json
 import os
 import subprocess
@@ -313,25 +314,26 @@ def test_router_ties_take_the_lowest_expert():
 
 
 # ---- whole models ------------------------------------------------------------------------------------------------
-LIMIT = {torch.float32: (2e-5, 2e-4), torch.bfloat16: (2e-2, 1e-1), torch.float16: (4e-3, 4e-2)}  # median, 97 % of the positions
+LIMIT = {torch.float32: (2e-5, 2e-4), torch.bfloat16: (2e-2, 6e-2), torch.float16: (4e-3, 2e-2)}  # median and largest error
 
 
 def _close(got, ref, dtype, what=""):
     e = pu.row_err(got, ref).flatten()
-    med, most = LIMIT[dtype]
-    # (a close router decision may go the other way in 16 bits: the tail of the positions has no limit)
-    assert torch.isfinite(e).all() and e.median() < med and torch.quantile(e, 0.97) < most, (what, e.median(), torch.quantile(e, 0.97), e.max())
-    if dtype == torch.float32:
-        assert e.max() < most, (what, e.max())
+    assert torch.isfinite(e).all() and e.median() < LIMIT[dtype][0] and e.max() < LIMIT[dtype][1], (what, e.median(), e.max())
 
 
 _CACHE = {}
 
 
-def _case(name, n=150, seed=1):
-    key = (name, n, seed)
+def _case(name, dtype, n=150, seed=1):
+    """(config, weights, tokens, oracle logits).  In 16 bits a close router decision may go the other way, which no limit
+    could tell from a fault: there every token uses all experts (the choice itself is tested in fp32 and alone)."""
+    key = (name, dtype == torch.float32, n, seed)
     if key not in _CACHE:
-        cfg = pu.CONFIGS[name]
+        cfg = copy.deepcopy(pu.CONFIGS[name])
+        for layer in cfg["layers"]:
+            if layer["mlp"] and dtype != torch.float32:
+                layer["mlp"]["router"]["top"] = layer["mlp"]["router"]["experts"]
         w = pu.weights(cfg, 7)
         toks = pu.tokens(cfg, n, seed)
         _CACHE[key] = (cfg, w, toks, pu.reference(cfg, w, toks))
@@ -342,7 +344,7 @@ def _case(name, n=150, seed=1):
 @pytest.mark.parametrize("name", list(pu.CONFIGS))
 @pytest.mark.parametrize("cuts", [[150], [1], [2], [100, 1], [3, 2, 64, 16, 17, 1], [65, 7]], ids=str)
 def test_model_prompts_portions_and_single_tokens(name, dtype, cuts):
-    cfg, w, toks, ref = _case(name)
+    cfg, w, toks, ref = _case(name, dtype)
     model = pu.build(cfg, w, dtype, "cuda", 1, 152)
     _close(pu.feed(model, toks[None], cuts)[0], ref, dtype, cuts)
 
@@ -351,7 +353,7 @@ def test_model_prompts_portions_and_single_tokens(name, dtype, cuts):
 @pytest.mark.parametrize("name", ["uneven", "tiles"])
 def test_batches_and_reused_rows(name, dtype):
     """Rows of a batch do not see one another; a row that served a longer sequence serves another from position 0."""
-    cfg, w, toks, ref = _case(name)
+    cfg, w, toks, ref = _case(name, dtype)
     model = pu.build(cfg, w, dtype, "cuda", 3, 152)
     rows = torch.stack([toks[:90], pu.tokens(cfg, 90, 11), pu.tokens(cfg, 90, 12)])
     refs = torch.stack([pu.reference(cfg, w, r) for r in rows])
@@ -380,8 +382,9 @@ def test_window_edge_reaches_the_logits(dtype):
             model = pu.build(cfg, w, dtype, "cuda", 1, n)
             cuts = [qpos, 1] if decoded else [n]
             a, b = (pu.feed(model, t[None], cuts)[0, qpos] for t in (base, moved))
-            assert (torch.equal(a, b) or not seen) and ((a - b).abs().max() > 1e-4 or not seen), (decoded, gap)
-            if not seen:
+            if seen:
+                assert (a - b).abs().max() > 1e-2, (decoded, gap)
+            else:
                 assert torch.equal(a, b), (decoded, gap)
             assert pu.row_err(b[None], pu.reference(cfg, w, moved)[qpos][None]).max() < LIMIT[dtype][1]
 
@@ -391,7 +394,7 @@ def test_long_greedy_decoding_through_the_device_loop(dtype):
     """DeviceLoop (captured steps, state put back after the warm-up) against the oracle fed the same tokens: every
     chosen token is the oracle's best, or within rounding of it."""
     from gpt_fast.generate import DeviceLoop
-    cfg, w, toks, _ = _case("tiles")
+    cfg, w, toks, _ = _case("tiles", dtype)
     model = pu.build(cfg, w, dtype, "cuda", 2, 240)
     prompt = torch.stack([toks[:30], pu.tokens(cfg, 30, 31)])
     pos = torch.arange(30, dtype=torch.int32, device="cuda")
@@ -413,7 +416,7 @@ def test_long_greedy_decoding_through_the_device_loop(dtype):
 
 
 def test_sampling_and_last_logits():
-    cfg, w, toks, ref = _case("uneven")
+    cfg, w, toks, ref = _case("uneven", torch.bfloat16)
     model = pu.build(cfg, w, torch.bfloat16, "cuda", 1, 152)
     pos = torch.arange(60, dtype=torch.int32, device="cuda")
     last = model.prefill_last(toks[None, :60].cuda(), pos)[0, 0].float().cpu()
@@ -431,7 +434,7 @@ def test_sampling_and_last_logits():
 def test_checkpoint_folder_and_trace_replay(tmp_path):
     """bin/trace_run on a checkpoint folder: two requests one after the other, portions and single tokens."""
     import numpy as np
-    cfg, w, toks, ref = _case("uneven")
+    cfg, w, toks, ref = _case("uneven", torch.float32)
     pu.save(cfg, w, tmp_path / "model")
     os.makedirs(tmp_path / "out")
     other = pu.tokens(cfg, 40, 77)
