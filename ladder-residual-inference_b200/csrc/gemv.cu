@@ -8,7 +8,7 @@
 //   PLAIN   store (optionally + addend)                       wo / w2 / LM head
 //   SWIGLU  rows (j, I + j) -> silu(gate) * up                 w1
 //   F32     store the fp32 sums                                 projections that feed fp32 arithmetic
-//   GLU     as SWIGLU with the clamped unit of an expert         one (token, expert) pair per grid.y slice
+//   GLU     as SWIGLU with the clamped unit of an expert         one (token, expert) pair per grid.x slice
 //   QKV     rotate adjacent pairs, scatter q / k-cache / v-cache   wqkv
 //   ARGMAX  no logits stored: arg-max over rows and ranks           LM head, greedy decoding (argmax.cuh)
 #include <cstdlib>
@@ -30,8 +30,11 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
   const T* __restrict__ w = static_cast<const T*>(p.w);
   const T* __restrict__ x = static_cast<const T*>(p.x);
   constexpr bool kPairs = M == 1 && (EPI == EPI_GLU || EPI == EPI_PLAIN);  // forms that take expert weights
-  const int64_t pair = blockIdx.y;
-  if (kPairs && p.ex.pairs > 0) {
+  const bool by_pair = kPairs && p.ex.pairs > 0;
+  // pairs are the fast grid dimension: those that share an expert read its rows at about the same time
+  const int64_t pair = by_pair ? blockIdx.x : 0;
+  const int64_t tile = by_pair ? blockIdx.y : blockIdx.x;
+  if (by_pair) {
     // the matrix is chosen by the preceding kernels: nothing can be streamed before they are done
     pdl_launch_dependents();
     pdl_wait();
@@ -45,11 +48,11 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
   for (int r = 0; r < R; ++r) {
     int64_t row;
     if (EPI == EPI_SWIGLU || EPI == EPI_GLU) {
-      int64_t j = static_cast<int64_t>(blockIdx.x) * (R / 2) + (r >> 1);
+      int64_t j = tile * (R / 2) + (r >> 1);
       j = j < p.n ? j : p.n - 1;
       row = (r & 1) ? p.n + j : j;  // even slot: up row j, odd slot: gate row I + j
     } else {
-      row = static_cast<int64_t>(blockIdx.x) * R + r;
+      row = tile * R + r;
       row = row < p.n ? row : p.n - 1;
     }
     wrow[r] = w + row * K;
@@ -79,7 +82,7 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
   // begin its own prologue, and only then wait for the activations to be complete.
   int c0 = warp;
   load_w(c0);
-  if (!kPairs || p.ex.pairs == 0) {
+  if (!by_pair) {
     pdl_launch_dependents();
     pdl_wait();
   }
@@ -133,7 +136,7 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
         s1 += red[wi][m * R + 2 * j + 1];
       }
       // compare what the projection would have stored: logits rounded to the storage type
-      const int64_t n = static_cast<int64_t>(blockIdx.x) * R + 2 * j;
+      const int64_t n = tile * R + 2 * j;
       unsigned long long k = 0ull;
       if (n < p.n) k = argmax_key(rnd<T>(s0), p.am.index_offset + n);
       if (n + 1 < p.n) {
@@ -161,14 +164,14 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
     s1 += red[wi][m * R + 2 * j + 1];
   }
   if (EPI == EPI_F32) {
-    const int64_t n = static_cast<int64_t>(blockIdx.x) * R + 2 * j;
+    const int64_t n = tile * R + 2 * j;
     float* y = static_cast<float*>(p.y) + static_cast<int64_t>(m) * p.n;
     if (n < p.n) y[n] = s0;
     if (n + 1 < p.n) y[n + 1] = s1;
     return;
   }
   if (EPI == EPI_GLU) {
-    const int64_t jj = static_cast<int64_t>(blockIdx.x) * (R / 2) + j;
+    const int64_t jj = tile * (R / 2) + j;
     const float sc = p.ex.row_scale[pair];
     if (jj < p.n) static_cast<T*>(p.y)[pair * p.n + jj] = Num<T>::from_f(clamped_glu(sc * s1, sc * s0, p.ex.glu));
     return;
@@ -177,8 +180,8 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
   const float v0 = rnd<T>(s0), v1 = rnd<T>(s1);
 
   if (EPI == EPI_PLAIN) {
-    const int64_t n = static_cast<int64_t>(blockIdx.x) * R + 2 * j;
-    T* y = static_cast<T*>(p.y) + (kPairs && p.ex.pairs > 0 ? pair : static_cast<int64_t>(m)) * p.n;
+    const int64_t n = tile * R + 2 * j;
+    T* y = static_cast<T*>(p.y) + (by_pair ? pair : static_cast<int64_t>(m)) * p.n;
     const T* add = p.addend ? static_cast<const T*>(p.addend) + static_cast<int64_t>(m) * p.n : nullptr;
     const float o0 = n < p.n ? rnd<T>(add ? v0 + Num<T>::to_f(add[n]) : v0) : 0.f;
     const float o1 = n + 1 < p.n ? rnd<T>(add ? v1 + Num<T>::to_f(add[n + 1]) : v1) : 0.f;
@@ -198,10 +201,10 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
                        : "memory");
     }
   } else if (EPI == EPI_SWIGLU) {
-    const int64_t jj = static_cast<int64_t>(blockIdx.x) * (R / 2) + j;
+    const int64_t jj = tile * (R / 2) + j;
     if (jj < p.n) static_cast<T*>(p.y)[static_cast<int64_t>(m) * p.n + jj] = swiglu_rounded<T>(v0, v1);
   } else {
-    const int64_t n = static_cast<int64_t>(blockIdx.x) * R + 2 * j;  // even
+    const int64_t n = tile * R + 2 * j;  // even
     if (n >= p.n) return;
     qkv_epilogue_pair<T>(p, m, n, v0, v1);
   }
@@ -215,7 +218,8 @@ int launch_gemv(const LinearParams& p, cudaStream_t st) {
   const int64_t per_cta = EPI == EPI_SWIGLU || EPI == EPI_GLU ? R / 2 : R;
   const int64_t grid = (p.n + per_cta - 1) / per_cta;
   const unsigned pairs = p.ex.pairs > 0 ? static_cast<unsigned>(p.ex.pairs) : 1u;
-  LRI_CUDA(launch_pdl(gemv_kernel<T, M, R, U, EPI>, dim3(static_cast<unsigned>(grid), pairs), dim3(W * 32), 0, st, p));
+  const dim3 dims = p.ex.pairs > 0 ? dim3(pairs, static_cast<unsigned>(grid)) : dim3(static_cast<unsigned>(grid));
+  LRI_CUDA(launch_pdl(gemv_kernel<T, M, R, U, EPI>, dims, dim3(W * 32), 0, st, p));
   LRI_LAUNCH_CHECK("gemv_kernel");
   return LRI_OK;
 }

@@ -94,12 +94,13 @@ struct Smem {
   alignas(16) float f[kBlock][CP];
   alignas(16) float bias[CP];
   alignas(16) float low[CP];
-  alignas(16) float F[CP];
+  alignas(16) float F[2][CP];
+  alignas(16) float w[kMaxE];
   float o[2][kBlock][kMaxE + 4];  // per half of the channels
-  alignas(16) bf16 qd[kTerms][kBlock * kPitchC];
-  alignas(16) bf16 kd[kTerms][kBlock * kPitchC];
-  alignas(16) bf16 v[2][kBlock * kPitchE];
-  alignas(16) bf16 a[kTerms][kBlock * kPitchA];
+  alignas(16) bf16 qd[2][kTerms][kBlock * kPitchC];
+  alignas(16) bf16 kd[2][kTerms][kBlock * kPitchC];
+  alignas(16) bf16 v[2][2][kBlock * kPitchE];
+  alignas(16) bf16 a[2][kTerms][kBlock * kPitchA];
 };
 
 // Grid (segments, heads, sequences).  FULL: outputs and the sequence's final state; otherwise the segment's contribution.
@@ -122,12 +123,13 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
     sm.bias[c] = c < C ? Num<T>::to_f(static_cast<const T*>(p.f_bias)[h * C + c]) : 0.f;
     sm.low[c] = c < C ? Num<T>::to_f(static_cast<const T*>(p.lower)[h * C + c]) : 0.f;
   }
+  for (int e = tid; e < E; e += kThreads) sm.w[e] = Num<T>::to_f(static_cast<const T*>(p.norm_w)[e]);
   static_assert(kWarps == kBlock && kThreads == 4 * 128, "work is dealt to warps by token and to threads by channel");
   // channels past C stay zero in the arrays that the products read
   if (C < CP)
-    for (int i = tid; i < kTerms * kBlock * Smem<CP>::kPitchC; i += kThreads) {
-      (&sm.qd[0][0])[i] = __float2bfloat16_rn(0.f);
-      (&sm.kd[0][0])[i] = __float2bfloat16_rn(0.f);
+    for (int i = tid; i < 2 * kTerms * kBlock * Smem<CP>::kPitchC; i += kThreads) {
+      (&sm.qd[0][0][0])[i] = __float2bfloat16_rn(0.f);
+      (&sm.kd[0][0][0])[i] = __float2bfloat16_rn(0.f);
     }
   pdl_launch_dependents();
   pdl_wait();
@@ -146,7 +148,6 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  fetch(s_begin, 0);
 
   // ---- state before the segment ----
   float st[kTiles][4];
@@ -182,42 +183,37 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
   }
   float decay = 1.f;  // thread c: product of all gates of the segment (first pass)
 
-  int buf = 0;
-  for (int s0 = s_begin; s0 < s_end; s0 += kBlock, buf ^= 1) {
-    asm volatile("cp.async.wait_all;" ::: "memory");
-    __syncthreads();  // the block has arrived, the previous block's shared arrays have been read
-    const float* raw = sm.raw[buf];
-    if (s0 + kBlock < s_end) fetch(s0 + kBlock, buf ^ 1);
-    // ---- gates, activations, v terms ----
-    {
-      const bool in = s0 + warp < s_end;
-      const float* rw = raw + warp * (2 * CP + kMaxE) + x4;
-      if (x4 < CP) {
-        float4 f = make_float4(1.f, 1.f, 1.f, 1.f), q = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (in && x4 < C) {
-          const float4 fr = *reinterpret_cast<const float4*>(rw + CP);
-          const float4 bi = *reinterpret_cast<const float4*>(&sm.bias[x4]), lo = *reinterpret_cast<const float4*>(&sm.low[x4]);
-          f.x = gate(fr.x, bi.x, lo.x), f.y = gate(fr.y, bi.y, lo.y), f.z = gate(fr.z, bi.z, lo.z), f.w = gate(fr.w, bi.w, lo.w);
-          if (FULL) {
-            const float4 qr = *reinterpret_cast<const float4*>(rw);
-            q = make_float4(silu(qr.x), silu(qr.y), silu(qr.z), silu(qr.w));
-          }
+  // ---- steps of a block; buf = parity of the block ----
+  // gates, activations, v terms (each thread reads what it fetched itself)
+  auto gates = [&](int s0, int buf) {
+    const bool in = s0 + warp < s_end;
+    const float* rw = sm.raw[buf] + warp * (2 * CP + kMaxE) + x4;
+    if (x4 < CP) {
+      float4 f = make_float4(1.f, 1.f, 1.f, 1.f), q = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (in && x4 < C) {
+        const float4 fr = *reinterpret_cast<const float4*>(rw + CP);
+        const float4 bi = *reinterpret_cast<const float4*>(&sm.bias[x4]), lo = *reinterpret_cast<const float4*>(&sm.low[x4]);
+        f.x = gate(fr.x, bi.x, lo.x), f.y = gate(fr.y, bi.y, lo.y), f.z = gate(fr.z, bi.z, lo.z), f.w = gate(fr.w, bi.w, lo.w);
+        if (FULL) {
+          const float4 qr = *reinterpret_cast<const float4*>(rw);
+          q = make_float4(silu(qr.x), silu(qr.y), silu(qr.z), silu(qr.w));
         }
-        *reinterpret_cast<float4*>(&sm.f[warp][x4]) = f;
-        if (FULL) *reinterpret_cast<float4*>(&sm.q[warp][x4]) = q;
       }
-      if (x4 < E) {
-        const float4 x = in ? *reinterpret_cast<const float4*>(rw + 2 * CP) : make_float4(0.f, 0.f, 0.f, 0.f);
-        uint32_t lo[kTerms], hi[kTerms];
-        split2(rnd<T>(x.x), rnd<T>(x.y), lo);
-        split2(rnd<T>(x.z), rnd<T>(x.w), hi);
-#pragma unroll
-        for (int i = 0; i < kVTerms; ++i)
-          *reinterpret_cast<uint2*>(&sm.v[i][warp * Smem<CP>::kPitchE + x4]) = make_uint2(lo[i], hi[i]);
-      }
+      *reinterpret_cast<float4*>(&sm.f[warp][x4]) = f;
+      if (FULL) *reinterpret_cast<float4*>(&sm.q[warp][x4]) = q;
     }
-    __syncthreads();
-    // ---- running products: thread (channel, k" or q", first or last 8 tokens) ----
+    if (x4 < E) {
+      const float4 x = in ? *reinterpret_cast<const float4*>(rw + 2 * CP) : make_float4(0.f, 0.f, 0.f, 0.f);
+      uint32_t lo[kTerms], hi[kTerms];
+      split2(rnd<T>(x.x), rnd<T>(x.y), lo);
+      split2(rnd<T>(x.z), rnd<T>(x.w), hi);
+#pragma unroll
+      for (int i = 0; i < kVTerms; ++i)
+        *reinterpret_cast<uint2*>(&sm.v[buf][i][warp * Smem<CP>::kPitchE + x4]) = make_uint2(lo[i], hi[i]);
+    }
+  };
+  auto products = [&](int buf) {
+    // running products: thread (channel, k" or q", first or last 8 tokens)
     {
       constexpr int kH = kBlock / 2;
       const int c = tid & 127, part = tid >> 7, t0 = (part & 1) * kH;
@@ -230,15 +226,15 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
 #pragma unroll
           for (int i = kH - 1; i >= 0; --i) {
             const float f = sm.f[t0 + i][c];
-            split_store(&sm.kd[0][(t0 + i) * Smem<CP>::kPitchC + c], kBlock * Smem<CP>::kPitchC, (1.f - f) * r);
+            split_store(&sm.kd[buf][0][(t0 + i) * Smem<CP>::kPitchC + c], kBlock * Smem<CP>::kPitchC, (1.f - f) * r);
             r *= f;
           }
           if (t0 == 0) {
-            sm.F[c] = r;
+            sm.F[buf][c] = r;
             decay *= r;
           }
         } else if (c < CP) {
-          sm.F[c] = 1.f;
+          sm.F[buf][c] = 1.f;
         }
       } else if (FULL && c < C) {
         float r = 1.f;
@@ -248,53 +244,53 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
 #pragma unroll
         for (int i = 0; i < kH; ++i) {
           r *= sm.f[t0 + i][c];
-          split_store(&sm.qd[0][(t0 + i) * Smem<CP>::kPitchC + c], kBlock * Smem<CP>::kPitchC, sm.q[t0 + i][c] * r);
+          split_store(&sm.qd[buf][0][(t0 + i) * Smem<CP>::kPitchC + c], kBlock * Smem<CP>::kPitchC, sm.q[t0 + i][c] * r);
         }
       }
     }
-    // ---- A[t, s]: warp s, lanes over channels ----
-    if (FULL) {
-      constexpr int kPer = CP / 32;
-      const int s = warp;
-      float d[kPer] = {}, a[kBlock];
+    if (!FULL) return;
+    // A[t, s]: warp s, lanes over channels
+    constexpr int kPer = CP / 32;
+    const int s = warp;
+    float d[kPer] = {}, a[kBlock];
 #pragma unroll
-      for (int t = 0; t < kBlock; ++t) {
-        float x = 0.f;
-        if (t >= s) {
+    for (int t = 0; t < kBlock; ++t) {
+      float x = 0.f;
+      if (t >= s) {
 #pragma unroll
-          for (int j = 0; j < kPer; j += 2) {
-            const float2 f = *reinterpret_cast<const float2*>(&sm.f[t][lane * kPer + j]);
-            const float2 q = *reinterpret_cast<const float2*>(&sm.q[t][lane * kPer + j]);
-            d[j] = t == s ? 1.f - f.x : d[j] * f.x;
-            d[j + 1] = t == s ? 1.f - f.y : d[j + 1] * f.y;
-            x = fmaf(q.x, d[j], x);
-            x = fmaf(q.y, d[j + 1], x);
-          }
+        for (int j = 0; j < kPer; j += 2) {
+          const float2 f = *reinterpret_cast<const float2*>(&sm.f[t][lane * kPer + j]);
+          const float2 q = *reinterpret_cast<const float2*>(&sm.q[t][lane * kPer + j]);
+          d[j] = t == s ? 1.f - f.x : d[j] * f.x;
+          d[j + 1] = t == s ? 1.f - f.y : d[j + 1] * f.y;
+          x = fmaf(q.x, d[j], x);
+          x = fmaf(q.y, d[j + 1], x);
         }
-        a[t] = x;
       }
-      // sums over the lanes: each exchange halves the values a lane holds
-      int t_mine = 0;
-#pragma unroll
-      for (int n = kBlock / 2, o = 16; n >= 1; n >>= 1, o >>= 1) {
-        const bool up = lane & o;
-#pragma unroll
-        for (int i = 0; i < n; ++i) {
-          const float give = up ? a[i] : a[i + n];
-          a[i] = (up ? a[i + n] : a[i]) + __shfl_xor_sync(0xffffffffu, give, o);
-        }
-        t_mine = t_mine * 2 + (up ? 1 : 0);
-      }
-      a[0] += __shfl_xor_sync(0xffffffffu, a[0], 1);
-      if ((lane & 1) == 0) split_store(&sm.a[0][t_mine * Smem<CP>::kPitchA + s], kBlock * Smem<CP>::kPitchA, a[0]);
+      a[t] = x;
     }
-    __syncthreads();
+    // sums over the lanes: each exchange halves the values a lane holds
+    int t_mine = 0;
+#pragma unroll
+    for (int n = kBlock / 2, o = 16; n >= 1; n >>= 1, o >>= 1) {
+      const bool up = lane & o;
+#pragma unroll
+      for (int i = 0; i < n; ++i) {
+        const float give = up ? a[i] : a[i + n];
+        a[i] = (up ? a[i + n] : a[i]) + __shfl_xor_sync(0xffffffffu, give, o);
+      }
+      t_mine = t_mine * 2 + (up ? 1 : 0);
+    }
+    a[0] += __shfl_xor_sync(0xffffffffu, a[0], 1);
+    if ((lane & 1) == 0) split_store(&sm.a[buf][0][t_mine * Smem<CP>::kPitchA + s], kBlock * Smem<CP>::kPitchA, a[0]);
+  };
+  auto tensor = [&](int buf) {
     if (live) {
       // V^T: rows of E, 16 tokens deep
       uint32_t va[kVTerms][4];
 #pragma unroll
       for (int i = 0; i < kVTerms; ++i)
-        ldmatrix_x4_trans(&sm.v[i][((lane & 7) + ((lane >> 4) & 1) * 8) * Smem<CP>::kPitchE + e0 + ((lane >> 3) & 1) * 8], va[i][0],
+        ldmatrix_x4_trans(&sm.v[buf][i][((lane & 7) + ((lane >> 4) & 1) * 8) * Smem<CP>::kPitchE + e0 + ((lane >> 3) & 1) * 8], va[i][0],
                           va[i][1], va[i][2], va[i][3]);
       if (FULL) {
         float o[2][4] = {};
@@ -311,7 +307,7 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
           uint32_t b[kTerms][4];  // tokens 0-7: [0], [1]; tokens 8-15: [2], [3]
 #pragma unroll
           for (int i = 0; i < kTerms; ++i)
-            ldmatrix_x4(&sm.qd[i][((lane & 7) + (lane >> 4) * 8) * Smem<CP>::kPitchC + c0 + k * 16 + ((lane >> 3) & 1) * 8], b[i][0], b[i][1],
+            ldmatrix_x4(&sm.qd[buf][i][((lane & 7) + (lane >> 4) * 8) * Smem<CP>::kPitchC + c0 + k * 16 + ((lane >> 3) & 1) * 8], b[i][0], b[i][1],
                         b[i][2], b[i][3]);
 #pragma unroll
           for (int n = 0; n < 2; ++n) {
@@ -325,7 +321,7 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
           uint32_t b[kTerms][4];
 #pragma unroll
           for (int i = 0; i < kTerms; ++i)
-            ldmatrix_x4(&sm.a[i][((lane & 7) + (lane >> 4) * 8) * Smem<CP>::kPitchA + ((lane >> 3) & 1) * 8], b[i][0], b[i][1], b[i][2],
+            ldmatrix_x4(&sm.a[buf][i][((lane & 7) + (lane >> 4) * 8) * Smem<CP>::kPitchA + ((lane >> 3) & 1) * 8], b[i][0], b[i][1], b[i][2],
                         b[i][3]);
           // each half of the channels adds this product for half of the tokens
           uint32_t b0[kTerms], b1[kTerms];
@@ -347,10 +343,10 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
         uint32_t b[kTerms][4];  // channels c0 + 16 k .. + 7: [0], [1]; + 8 ..: [2], [3]
 #pragma unroll
         for (int i = 0; i < kTerms; ++i)
-          ldmatrix_x4_trans(&sm.kd[i][(lane & 15) * Smem<CP>::kPitchC + c0 + k * 16 + (lane >> 4) * 8], b[i][0], b[i][1], b[i][2], b[i][3]);
+          ldmatrix_x4_trans(&sm.kd[buf][i][(lane & 15) * Smem<CP>::kPitchC + c0 + k * 16 + (lane >> 4) * 8], b[i][0], b[i][1], b[i][2], b[i][3]);
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
-          const float2 F = *reinterpret_cast<const float2*>(&sm.F[c0 + k * 16 + n * 8 + cc]);
+          const float2 F = *reinterpret_cast<const float2*>(&sm.F[buf][c0 + k * 16 + n * 8 + cc]);
           float(&s)[4] = st[2 * k + n];
           s[0] *= F.x, s[1] *= F.y, s[2] *= F.x, s[3] *= F.y;
           uint32_t b0[kTerms], b1[kTerms];
@@ -360,29 +356,57 @@ __global__ void __launch_bounds__(kThreads, 1) hgrn2_blocks_kernel(const Hgrn2Pa
         }
       }
     }
-    // ---- RMSNorm over E, one token per warp ----
-    if (FULL) {
-      __syncthreads();
-      const T* w = static_cast<const T*>(p.norm_w);
-      const int t = warp;
-      if (s0 + t < s_end) {
-        float x[4], ss = 0.f;
+  };
+  // RMSNorm over E, one token per warp
+  auto norm = [&](int s0) {
+        const int t = warp;
+    if (s0 + t < s_end) {
+      float x[4], ss = 0.f;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const int e = lane * 4 + j;
-          x[j] = e < E ? sm.o[0][t][e] + sm.o[1][t][e] : 0.f;
-          ss += x[j] * x[j];
-        }
-        const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(E) + p.eps);
-        if (lane * 4 < E) {
-          T* dst = static_cast<T*>(p.out) + ((static_cast<int64_t>(b) * p.S + s0 + t) * H + h) * E + lane * 4;
-          uint2 v;
-          v.x = pack2<T>(x[0] * inv * Num<T>::to_f(w[lane * 4]), x[1] * inv * Num<T>::to_f(w[lane * 4 + 1]));
-          v.y = pack2<T>(x[2] * inv * Num<T>::to_f(w[lane * 4 + 2]), x[3] * inv * Num<T>::to_f(w[lane * 4 + 3]));
-          *reinterpret_cast<uint2*>(dst) = v;
-        }
+      for (int j = 0; j < 4; ++j) {
+        const int e = lane * 4 + j;
+        x[j] = e < E ? sm.o[0][t][e] + sm.o[1][t][e] : 0.f;
+        ss += x[j] * x[j];
+      }
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(E) + p.eps);
+      if (lane * 4 < E) {
+        T* dst = static_cast<T*>(p.out) + ((static_cast<int64_t>(b) * p.S + s0 + t) * H + h) * E + lane * 4;
+        uint2 v;
+        v.x = pack2<T>(x[0] * inv * sm.w[x4], x[1] * inv * sm.w[x4 + 1]);
+        v.y = pack2<T>(x[2] * inv * sm.w[x4 + 2], x[3] * inv * sm.w[x4 + 3]);
+        *reinterpret_cast<uint2*>(dst) = v;
       }
     }
+  };
+
+  // Two barriers a block: while the tensor products of block i run, the gates of block i + 1 are taken (half of the warps
+  // begin with the one, half with the other); then the running products of block i + 1 beside the norm of block i.
+  auto wait_fetched = [] { asm volatile("cp.async.wait_group 1;" ::: "memory"); };
+  fetch(s_begin, 0);
+  fetch(s_begin + kBlock, 1);
+  wait_fetched();
+  __syncthreads();  // bias, low
+  gates(s_begin, 0);
+  __syncthreads();
+  products(0);
+  __syncthreads();
+  int buf = 0;
+  for (int s0 = s_begin; s0 < s_end; s0 += kBlock, buf ^= 1) {
+    const bool more = s0 + kBlock < s_end;
+    fetch(s0 + 2 * kBlock, buf);
+    wait_fetched();
+#pragma unroll 1
+    for (int turn = 0; turn < 2; ++turn) {
+      if ((turn ^ (warp & 1)) == 0) {
+        if (more) gates(s0 + kBlock, buf ^ 1);
+      } else {
+        tensor(buf);
+      }
+    }
+    __syncthreads();
+    if (more) products(buf ^ 1);
+    if (FULL) norm(s0);
+    __syncthreads();
   }
   if (FULL) {
     if (seg == sg.count - 1)

@@ -38,6 +38,23 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
 }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
+// Visible rows lo .. hi and the tiles t0 .. t1 - 1 of a split
+struct TileRange {
+  int64_t lo, hi, t0, t1;
+};
+__device__ __forceinline__ TileRange tile_range(const DecodeParams& p, int split) {
+  const int64_t pos = *reinterpret_cast<const volatile int*>(p.input_pos);  // the low word of a 64-bit position too
+  TileRange r;
+  r.hi = pos < p.smax ? pos : p.smax - 1;
+  r.lo = pos - p.window + 1;
+  r.lo = r.lo < 0 ? 0 : r.lo;
+  const int64_t first = r.lo / kKeys, n = r.hi / kKeys - first + 1;
+  const int64_t per = (n + p.splits - 1) / p.splits;
+  r.t0 = first + split * per;
+  r.t1 = r.t0 + per < first + n ? r.t0 + per : first + n;
+  return r;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kThreads) latent_decode_kernel(const DecodeParams p) {
   extern __shared__ __align__(16) uint8_t ld_smem[];
@@ -49,18 +66,21 @@ __global__ void __launch_bounds__(kThreads) latent_decode_kernel(const DecodePar
   __shared__ float m_s[kHeads], l_s[kHeads], corr_s[kHeads];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int split = blockIdx.x, h0 = blockIdx.y * kHeads, b = blockIdx.z;
-  pdl_launch_dependents();
-  pdl_wait();
-  const int64_t pos = load_pos(p.input_pos, p.pos_is_i64, 0);
-  int64_t hi = pos < p.smax ? pos : p.smax - 1;
-  int64_t lo = pos - p.window + 1;
-  lo = lo < 0 ? 0 : lo;
-  const int64_t t_lo = lo / kKeys, n_tiles = hi / kKeys - t_lo + 1;
-  const int64_t per = (n_tiles + p.splits - 1) / p.splits;
-  const int64_t t0 = t_lo + split * per;
-  const int64_t t1 = t0 + per < t_lo + n_tiles ? t0 + per : t_lo + n_tiles;
-
   const int vecs = p.row_len / 8;
+  const T* kg = static_cast<const T*>(p.cache) + b * p.batch_pitch;
+  pdl_launch_dependents();
+  // Rows of earlier steps do not depend on the preceding kernel: ask the L2 for the first tile while it drains.  (Only a
+  // hint, from a position that may not be final, kept inside the cache.)
+  {
+    const TileRange g = tile_range(p, split);
+    const int64_t row = g.t0 * kKeys + (threadIdx.x >> 2);
+    if (g.t0 < g.t1 && row >= 0 && row < p.smax)
+      for (int e = (threadIdx.x & 3) * 64; e < p.row_len; e += 256)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(kg + row * p.row_len + e));
+  }
+  pdl_wait();
+  const TileRange range = tile_range(p, split);
+  const int64_t lo = range.lo, hi = range.hi, t0 = range.t0, t1 = range.t1;
   const T* qg = static_cast<const T*>(p.q) + b * p.q_row;
   // (a warp copies whole rows; the wait for the first tile of keys covers the queries too)
   for (int h = warp; h < kHeads; h += kWarps)
@@ -80,7 +100,6 @@ __global__ void __launch_bounds__(kThreads) latent_decode_kernel(const DecodePar
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[u][n][e] = 0.f;
   const int units = p.r / 16;
-  const T* kg = static_cast<const T*>(p.cache) + b * p.batch_pitch;
 
   for (int64_t t = t0; t < t1; ++t) {
     __syncthreads();  // the previous tile has been consumed (first pass: nothing)
@@ -212,6 +231,7 @@ template <typename T>
 __global__ void __launch_bounds__(128) latent_decode_merge_kernel(const DecodeParams p) {
   __shared__ float w_s[kMaxSplits];
   __shared__ float part[33];
+  __shared__ float4 sums[4][32];
   pdl_launch_dependents();
   pdl_wait();
   const int64_t bh = static_cast<int64_t>(blockIdx.y) * p.H + blockIdx.x;
@@ -228,13 +248,27 @@ __global__ void __launch_bounds__(128) latent_decode_merge_kernel(const DecodePa
   w_s[s] = w;
   __syncthreads();  // part is used again
   const float l = block_sum(w * ml.y, part);  // also orders w_s
-  const int col = blockIdx.z * 128 + threadIdx.x;
-  if (col >= p.r) return;
-  const float* o = p.part_o + bh * p.splits * p.r + col;
-  float acc = 0.f;
-#pragma unroll 16
-  for (int i = 0; i < n; ++i) acc = fmaf(w_s[i], o[static_cast<int64_t>(i) * p.r], acc);
-  static_cast<T*>(p.out)[bh * p.r + col] = Num<T>::from_f(l > 0.f ? acc / l : 0.f);
+  // 4 warps take every fourth split, a lane 4 columns: the loads of a thread are in flight together
+  const int warp = s >> 5, lane = s & 31;
+  const int col = blockIdx.z * 128 + lane * 4;
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (col < p.r) {
+    const float* o = p.part_o + bh * p.splits * p.r + col;
+#pragma unroll 8
+    for (int i = warp; i < n; i += 4) {
+      const float4 v = *reinterpret_cast<const float4*>(o + static_cast<int64_t>(i) * p.r);
+      const float wi = w_s[i];
+      acc.x = fmaf(wi, v.x, acc.x), acc.y = fmaf(wi, v.y, acc.y), acc.z = fmaf(wi, v.z, acc.z), acc.w = fmaf(wi, v.w, acc.w);
+    }
+  }
+  sums[warp][lane] = acc;
+  __syncthreads();
+  const int c = blockIdx.z * 128 + s;
+  if (c >= p.r) return;
+  float v = 0.f;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) v += reinterpret_cast<const float*>(&sums[i][0])[s];
+  static_cast<T*>(p.out)[bh * p.r + c] = Num<T>::from_f(l > 0.f ? v / l : 0.f);
 }
 
 int head_tiles(int H) { return (H + kHeads - 1) / kHeads; }

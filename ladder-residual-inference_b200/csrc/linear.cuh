@@ -24,7 +24,7 @@ struct PushArgs {
 };
 
 // Mixture of experts: the weight matrix of a row (or of a tile of rows) is chosen on the device.
-//   pairs > 0  streaming kernel, one (token, choice) pair per grid.y slice: matrix experts[pair], input row
+//   pairs > 0  streaming kernel, one (token, choice) pair per grid.x slice: matrix experts[pair], input row
 //              pair / rows_per_input, output row pair
 //   tiles      tcgen05 kernel: tiles[0] = number of 128-row tiles in use, tiles[1 + t] = matrix of tile t
 struct ExpertArgs {

@@ -46,7 +46,7 @@ const OptionSpec kOptionSpecs[OPT_COUNT] = {
     {"attn_prefill_tc", "LRI_ATTN_PREFILL_TC", 1, 0, 1},
     {"gemm_reserve_sms", "LRI_GEMM_RESERVE_SMS", 0, 0, 64},
     {"attn_head_tile", "LRI_ATTN_HEAD_TILE", 0, 0, 4},
-    {"moe_stream_pairs", "LRI_MOE_STREAM_PAIRS", 32, 0, 65535},
+    {"moe_stream_pairs", "LRI_MOE_STREAM_PAIRS", 10, 0, 65535},
     {"window_tc", "LRI_WINDOW_TC", 1, 0, 1},
     {"hgrn2_blocks", "LRI_HGRN2_BLOCKS", 1, 0, 1},
 };

@@ -28,7 +28,7 @@ def _restore_options():
     yield
     for name in (b"window_tc", b"hgrn2_blocks"):
         _C.lib.lri_set_option(name, 1)
-    _C.lib.lri_set_option(b"moe_stream_pairs", 32)
+    _C.lib.lri_set_option(b"moe_stream_pairs", 10)
     torch.cuda.synchronize()
     _C.check(_C.lib.lri_gemm_status())
 
