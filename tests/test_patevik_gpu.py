@@ -155,7 +155,7 @@ def _plant(q, k, i, j, h, strength=14.0):
 @pytest.mark.parametrize("plain", [False, True])
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("S,H,d1,d2,dv,history,pos0,window", [
-    (300, 2, 32, 16, 48, 0, 0, 72), (130, 3, 128, 64, 128, 63, 200, 64), (257, 2, 64, 32, 64, 64, 64, 65), (200, 1, 72, 8, 24, 40, 13, 100),
+    (300, 2, 40, 24, 48, 0, 0, 75), (130, 3, 128, 64, 128, 63, 200, 64), (257, 2, 64, 32, 64, 64, 64, 65), (200, 1, 72, 8, 24, 40, 13, 100),
     (520, 2, 96, 64, 128, 0, 0, 4096), (33, 2, 8, 8, 8, 0, 0, 1), (150, 2, 20, 6, 12, 30, 90, 31), (2, 3, 32, 16, 32, 20, 40, 21)])
 def test_window_attention_prompt(plain, dtype, S, H, d1, d2, dv, history, pos0, window):
     """Prompt form: the window's edges with planted keys exactly inside and exactly outside, keys before the portion,
@@ -195,7 +195,7 @@ def test_window_attention_prompt(plain, dtype, S, H, d1, d2, dv, history, pos0, 
 @pytest.mark.parametrize("plain", [False, True])
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("B,H,r,dr,smax,window,positions", [
-    (1, 4, 64, 16, 700, 72, [0, 1, 63, 64, 71, 72, 73, 127, 128, 500, 699]), (3, 5, 48, 16, 200, 64, [5, 63, 64, 199]),
+    (1, 5, 80, 32, 700, 77, [0, 1, 63, 64, 76, 77, 78, 127, 128, 500, 699]), (3, 5, 48, 16, 200, 64, [5, 63, 64, 199]),
     (2, 17, 256, 64, 500, 129, [128, 129, 300]), (1, 2, 36, 6, 90, 17, [16, 17, 80]), (2, 16, 512, 64, 300, 4096, [299]), (1, 3, 16, 16, 70, 1, [0, 64, 69])])
 def test_window_attention_single_token(plain, dtype, B, H, r, dr, smax, window, positions):
     """Single-token form on cached rows, with a planted row just inside or just outside the window."""
