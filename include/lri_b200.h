@@ -67,7 +67,8 @@ int lri_set_gemm_backend(int backend);
  * (LRI_ATTN_HEAD_TILE: query heads of a KV group per CTA of the cluster decode attention, 0 choose, 1, 2, 4),
  * moe_stream_pairs (LRI_MOE_STREAM_PAIRS: (token, expert) pairs up to which experts run as streaming projections),
  * window_tc (LRI_WINDOW_TC: 0 keeps sliding-window attention on the plain kernel), hgrn2_blocks
- * (LRI_HGRN2_BLOCKS: 0 keeps the HGRN2 recurrence token by token).  Unknown
+ * (LRI_HGRN2_BLOCKS: 0 keeps the HGRN2 recurrence token by token), scan_columns (LRI_SCAN_COLUMNS: state columns per
+ * lane of the matrix-state recurrences, 0 choose, 1, 2, 4).  Unknown
  * names and values an option does not take return LRI_ERR_ARG.  No counterpart in the reference
  * (its only switches are benchmark.py's command-line flags). */
 int lri_set_option(const char* name, int value);
@@ -369,6 +370,78 @@ int lri_moe_gateup(int dtype, const void* x, const void* w1, void* hidden, const
  * lri_gated_norm_add. */
 int lri_moe_down(int dtype, const void* hidden, const void* w2, void* y, const int32_t* ids, int64_t pairs,
                  const int32_t* tiles, int64_t max_tiles, int experts, int dim, int ff, lri_stream_t stream);
+
+/* ---- residual held as several streams (hyper-connections) ---------------------------------------------
+ * x [rows, streams, dim] fp32.  x_out_t = sum_s mix[s, t] x_s + out[t] y (all from the old streams; x_out may alias x, NULL:
+ * not stored), u = sum_s in_next[s] x_out_s (in_next NULL: plain sum), normed = RMSNorm(u) * weight rounded to `dtype`.
+ * mix [streams, streams] ([from, to]), out and in_next [streams], weight [dim] in `dtype`; up to 16 streams. */
+int lri_join_streams(int dtype, const float* x, const void* y, const void* mix, const void* out, float* x_out,
+                     const void* in_next, const void* weight, float eps, void* normed, int64_t rows, int streams, int dim,
+                     lri_stream_t stream);
+/* Starts the streams: every x_out_s = scale * table[idx], then u and normed as above. */
+int lri_embed_streams(int dtype, const void* table, const void* idx, int idx_is_i64, int64_t vocab, float scale,
+                      float* x_out, const void* in_next, const void* weight, float eps, void* normed, int64_t rows,
+                      int streams, int dim, lri_stream_t stream);
+
+/* ---- gate/up projection + clamped unit --------------------------------------------------------------------
+ * w1 [2 I, K] = [up | gate]; h = g sigmoid(alpha g) (u + offset), g = min(gate, limit), u = clamp(up, -limit, limit), from
+ * fp32 sums.  Kernels as lri_gateup_swiglu; LRI_FP32 and any K run the plain kernels. */
+size_t lri_gateup_glu_workspace_bytes(int dtype, int64_t M, int I, int K);
+int lri_gateup_glu(int dtype, const void* x, const void* w1, void* h, int64_t M, int I, int K, float alpha, float limit,
+                   float offset, void* workspace, size_t workspace_bytes, lri_stream_t stream);
+
+/* ---- grouped-query attention with whole-projection norms, windows, chunks and sinks --------------------------
+ * proj [B*S, ld] fp32 holds q (n_head heads of dim), k (n_kv of dim) and v (n_kv of vdim) at the offsets.  q and k are
+ * RMS-normed over all their elements (weights q_norm, k_norm; sums of squares over q_width, k_width elements are taken
+ * here or, sums != NULL, read from [rows, 2]), the first rot_dims of each head rotated by halves with rope_table
+ * [table_rows, rot_dims/2, 2] (fp32) at the token's position; q goes to [rows, n_head, dim], k and v to the caches
+ * [B, n_kv, smax, dim] and [B, n_kv, smax, vdim]. */
+int lri_grouped_prepare(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off,
+                        const void* q_norm, const void* k_norm, const float* sums, int q_width, int k_width, float eps,
+                        const float* rope_table, int64_t table_rows, int rot_dims, const void* input_pos, int pos_is_i64,
+                        void* q, void* k_cache, void* v_cache, int64_t smax, int B, int S, int n_head, int n_kv, int dim,
+                        int vdim, lri_stream_t stream);
+/* sums[row] = sums of squares of x[row, off1 .. off1 + n1) and x[row, off2 .. off2 + n2). */
+int lri_row_squares(const float* x, int64_t ld, int64_t off1, int n1, int64_t off2, int n2, float* sums, int64_t rows,
+                    lri_stream_t stream);
+/* Attention of the query at position p over cache positions j <= p with p - j < window (0: no window) and, chunk > 0,
+ * j / chunk == p / chunk.  sink [n_head] (NULL: none): exp(sink) joins the denominator.  out row = out_scale times the
+ * heads' results, pitch out_ld.  16-bit types: prompt portions of 16 tokens on (dim, vdim up to 128, multiples of 8) on
+ * tcgen05, single tokens on thread-block clusters; everything else on a plain kernel. */
+int lri_grouped_attention(int dtype, const void* q, const void* k_cache, const void* v_cache, const void* sink, void* out,
+                          int64_t out_ld, float out_scale, const void* input_pos, int pos_is_i64, int64_t smax,
+                          int64_t window, int64_t chunk, float scale, int B, int S, int n_head, int n_kv, int dim,
+                          int vdim, lri_stream_t stream);
+
+/* ---- matrix-state recurrences with a decay per key channel ----------------------------------------------------
+ * lri_state_scan: per sequence and head, over the tokens of the call, S <- decay * S (rows); beta != NULL (delta rule):
+ * u = beta (v - S^T k), else u = v; S <- S + k u^T; o = o_scale S^T q.  q, k [rows, kv_heads, dim] with row pitches (head h
+ * reads h / (heads / kv_heads)), v [rows, heads, vdim] with row pitch, decay [rows, heads, dim], beta [rows, heads],
+ * kq [rows, kv_heads] = k . q, o [rows, heads, vdim]; all fp32.  state [B, heads, dim, vdim] is read and written; a call that
+ * starts at position 0 starts from zero. */
+int lri_state_scan(const float* q, int64_t q_row, const float* k, int64_t k_row, const float* v, int64_t v_row,
+                   const float* decay, const float* beta, const float* kq, float* state, const void* input_pos,
+                   int pos_is_i64, float* o, float o_scale, int B, int S, int heads, int kv_heads, int dim, int vdim,
+                   lri_stream_t stream);
+/* Inputs of the gated delta rule.  proj [B*S, ld] holds q, k (kv_heads of dim), v (heads of vdim) and b (heads).  q, k, v
+ * pass a causal convolution over time per channel (conv_* [channels, taps], last column = current token) and silu, q and k
+ * become unit vectors x / sqrt(sum x^2 + 1e-6); beta = sigmoid(b); kq = k . q; z [rows, heads, dim] becomes
+ * exp(-exp(a_log) softplus(z + dt_bias)).  ring [B, taps, 2 kv_heads dim + heads vdim] keeps the last inputs of each
+ * channel (position p in slot p % taps); it is read for tokens before the call and updated. */
+int lri_delta_prepare(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, int64_t b_off,
+                      const void* conv_q, const void* conv_k, const void* conv_v, int taps, float* ring, float* z,
+                      const void* a_log, const void* dt_bias, const void* input_pos, int pos_is_i64, float* q, float* k,
+                      float* v, float* beta, float* kq, int B, int S, int heads, int kv_heads, int dim, int vdim,
+                      lri_stream_t stream);
+/* z [rows, width] <- sigmoid(z + bias)^(1 / tau). */
+int lri_logistic_decay(int dtype, float* z, const void* bias, float tau, int64_t rows, int width, lri_stream_t stream);
+/* out[row, head] = scale * RMSNorm(o[row, head]) * norm_weight * act(gate[row, head]), gate fp32 with row pitch gate_ld. */
+enum lri_gate { LRI_GATE_SIGMOID = 0, LRI_GATE_SILU = 1 };
+int lri_head_norm_gate(int dtype, const float* o, const void* norm_weight, float eps, const float* gate, int64_t gate_ld,
+                       int activation, float scale, void* out, int64_t out_ld, int64_t rows, int heads, int vdim,
+                       lri_stream_t stream);
+/* y [rows, n] = x[row, off .. off + n) rounded to `dtype`. */
+int lri_round_columns(int dtype, const float* x, int64_t ld, int64_t off, int n, void* y, int64_t rows, lri_stream_t stream);
 
 /* Reads (and clears) the device status word: LRI_OK or LRI_ERR_TIMEOUT.  Synchronises `stream`. */
 int lri_comm_status(lri_comm* comm, lri_stream_t stream);

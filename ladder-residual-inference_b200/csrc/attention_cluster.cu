@@ -12,11 +12,14 @@
 // forget, remote loads are a round trip).  After ONE cluster barrier the first CTA merges the splits
 // and writes the output; the others exit.  No scratch memory, no counters, and the grid still does
 // not depend on the position.
+//
+// MASKED: the same for key and value widths below HD, a window or chunk that bounds the visible positions from below, a
+// sink in the denominator, and a row pitch and factor of the output.
 #include <cooperative_groups.h>
 
 #include <cstdlib>
 
-#include "common.cuh"
+#include "latent_attention.cuh"
 
 namespace cg = cooperative_groups;
 
@@ -39,6 +42,12 @@ struct ClusterDecodeParams {
   int n_head, n_kv;
   int64_t smax;
   float scale_log2;
+  // MASKED
+  int dim, vdim;
+  int64_t window, chunk;
+  const void* sink;
+  int64_t out_ld;
+  float out_scale;
 };
 
 // dynamic shared memory: [NRG][GT] max, [NRG][GT] sum, [NRG][GT][HD] values (this CTA's row groups), then the
@@ -49,7 +58,7 @@ constexpr int cluster_smem_bytes() {
   return (NRG * GT * (2 + HD) + kClMaxSplits * GT * (HD + 2)) * 4;
 }
 
-template <typename T, int HD, int GT, int U>
+template <typename T, int HD, int GT, int U, bool MASKED>
 __global__ void __launch_bounds__(kClThreads) attn_decode_cluster_kernel(const ClusterDecodeParams p) {
   constexpr int LPR = HD / 8;    // lanes per cache row
   constexpr int RPW = 32 / LPR;  // row groups per warp
@@ -74,8 +83,10 @@ __global__ void __launch_bounds__(kClThreads) attn_decode_cluster_kernel(const C
   float* g_m = g_o + kClMaxSplits * GT * HD;  // [16][GT]
   float* g_l = g_m + kClMaxSplits * GT;       // [16][GT]
 
-  const T* kbase = static_cast<const T*>(p.k_cache) + (static_cast<int64_t>(b) * p.n_kv + kvh) * p.smax * HD + sl * 8;
-  const T* vbase = static_cast<const T*>(p.v_cache) + (static_cast<int64_t>(b) * p.n_kv + kvh) * p.smax * HD + sl * 8;
+  const int kd = MASKED ? p.dim : HD, vd = MASKED ? p.vdim : HD;
+  const bool k_live = !MASKED || sl * 8 < kd, v_live = !MASKED || sl * 8 < vd;
+  const T* kbase = static_cast<const T*>(p.k_cache) + (static_cast<int64_t>(b) * p.n_kv + kvh) * p.smax * kd + sl * 8;
+  const T* vbase = static_cast<const T*>(p.v_cache) + (static_cast<int64_t>(b) * p.n_kv + kvh) * p.smax * vd + sl * 8;
   {
     // While the preceding kernel (the QKV projection) still runs: ask the L2 for this CTA's share of the
     // cache, so that the loads below cost an L2 round trip instead of a DRAM one.  All rows but the newest
@@ -84,13 +95,14 @@ __global__ void __launch_bounds__(kClThreads) attn_decode_cluster_kernel(const C
     int64_t hint = (p.pos_is_i64 ? *reinterpret_cast<const volatile int64_t*>(p.input_pos)
                                  : static_cast<int64_t>(*reinterpret_cast<const volatile int32_t*>(p.input_pos))) + 2;
     hint = hint < 0 ? 0 : (hint > p.smax ? p.smax : hint);
-    const int64_t hchunk = (hint + ns - 1) / ns;
-    const int64_t h0 = split * hchunk;
+    const int64_t hlo = MASKED && hint > 1 ? first_visible(hint - 1, p.window, p.chunk) : 0;
+    const int64_t hchunk = (hint - hlo + ns - 1) / ns;
+    const int64_t h0 = hlo + split * hchunk;
     const int64_t h1 = (h0 + hchunk < hint) ? h0 + hchunk : hint;
     if ((sl & 7) == 0) {  // one request per 128-byte line
       for (int64_t j = h0 + rg; j < h1; j += NRG) {
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(kbase + j * HD));
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(vbase + j * HD));
+        if (k_live) asm volatile("prefetch.global.L2 [%0];" ::"l"(kbase + j * kd));
+        if (v_live) asm volatile("prefetch.global.L2 [%0];" ::"l"(vbase + j * vd));
       }
     }
   }
@@ -100,14 +112,15 @@ __global__ void __launch_bounds__(kClThreads) attn_decode_cluster_kernel(const C
   float qf[GT][8];
 #pragma unroll
   for (int h = 0; h < GT; ++h) {
-    const T* qp = static_cast<const T*>(p.q) + (static_cast<int64_t>(b) * p.n_head + head0 + h) * HD + sl * 8;
-    unpack8<T>(*reinterpret_cast<const uint4*>(qp), qf[h]);
+    const T* qp = static_cast<const T*>(p.q) + (static_cast<int64_t>(b) * p.n_head + head0 + h) * kd + sl * 8;
+    unpack8<T>(k_live ? *reinterpret_cast<const uint4*>(qp) : make_uint4(0, 0, 0, 0), qf[h]);
 #pragma unroll
     for (int e = 0; e < 8; ++e) qf[h][e] *= p.scale_log2;
   }
   ctx = ctx < 0 ? 0 : (ctx > p.smax ? p.smax : ctx);
-  const int64_t chunk = (ctx + ns - 1) / ns;
-  const int64_t p0 = split * chunk;
+  const int64_t lo = MASKED && ctx > 0 ? first_visible(ctx - 1, p.window, p.chunk) : 0;
+  const int64_t chunk = (ctx - lo + ns - 1) / ns;
+  const int64_t p0 = lo + split * chunk;
   const int64_t p1 = (p0 + chunk < ctx) ? p0 + chunk : ctx;
 
   float m[GT], l[GT], acc[GT][8];
@@ -129,8 +142,8 @@ __global__ void __launch_bounds__(kClThreads) attn_decode_cluster_kernel(const C
       const int64_t j = jb + lane / LPR + static_cast<int64_t>(t) * NRG;
       valid[t] = j < p1;
       const int64_t jc = valid[t] ? j : p1 - 1;
-      kv[t] = ld_stream16(kbase + jc * HD);
-      vv[t] = ld_stream16(vbase + jc * HD);
+      kv[t] = k_live ? ld_stream16(kbase + jc * kd) : make_uint4(0, 0, 0, 0);
+      vv[t] = v_live ? ld_stream16(vbase + jc * vd) : make_uint4(0, 0, 0, 0);
     }
     float s[U][GT];
 #pragma unroll
@@ -218,6 +231,11 @@ __global__ void __launch_bounds__(kClThreads) attn_decode_cluster_kernel(const C
     float mm = -INFINITY;
     for (int r = 0; r < ns; ++r) mm = fmaxf(mm, g_m[r * GT + h]);
     float ll = 0.f, oo = 0.f;
+    if (MASKED && p.sink) {
+      const float s = Num<T>::to_f(static_cast<const T*>(p.sink)[head0 + h]) * 1.4426950408889634f;
+      mm = fmaxf(mm, s);
+      ll = exp2f(s - mm);
+    }
     if (mm > -INFINITY) {
       for (int r = 0; r < ns; ++r) {
         const float w = exp2f(g_m[r * GT + h] - mm);
@@ -226,14 +244,18 @@ __global__ void __launch_bounds__(kClThreads) attn_decode_cluster_kernel(const C
       }
     }
     const float res = ll > 0.f ? oo / ll : 0.f;
-    static_cast<T*>(p.out)[(static_cast<int64_t>(b) * p.n_head + head0 + h) * HD + e] = Num<T>::from_f(res);
+    if (MASKED) {
+      if (e < vd) static_cast<T*>(p.out)[b * p.out_ld + static_cast<int64_t>(head0 + h) * vd + e] = Num<T>::from_f(res * p.out_scale);
+    } else {
+      static_cast<T*>(p.out)[(static_cast<int64_t>(b) * p.n_head + head0 + h) * HD + e] = Num<T>::from_f(res);
+    }
   }
 }
 
-template <typename T, int HD, int GT, int U>
+template <typename T, int HD, int GT, int U, bool MASKED>
 int launch_one(const ClusterDecodeParams& p, int B, int ns, int tiles, cudaStream_t st) {
   constexpr int smem = cluster_smem_bytes<HD, GT>();
-  auto kern = attn_decode_cluster_kernel<T, HD, GT, U>;
+  auto kern = attn_decode_cluster_kernel<T, HD, GT, U, MASKED>;
   static std::atomic<unsigned long long> attr_set{0};  // per template instantiation, one bit per device
   if (device_setup_needed(attr_set)) {
     LRI_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
@@ -261,26 +283,29 @@ int launch_one(const ClusterDecodeParams& p, int B, int ns, int tiles, cudaStrea
 
 // U = positions per row group kept in flight: enough to cover the longest range a CTA can get
 // (ceil(smax / ns) positions over NRG row groups) in one pass when that takes at most 12, else 4 per pass.
-template <typename T, int HD, int GT>
+template <typename T, int HD, int GT, bool MASKED>
 int launch_u(const ClusterDecodeParams& p, int B, int ns, int tiles, cudaStream_t st) {
   constexpr int NRG = (32 / (HD / 8)) * kClWarps;
-  const int64_t longest = (p.smax + ns - 1) / ns;
+  int64_t visible = p.smax;
+  if (MASKED && p.window < visible) visible = p.window;
+  if (MASKED && p.chunk > 0 && p.chunk < visible) visible = p.chunk;
+  const int64_t longest = (visible + ns - 1) / ns;
   const int64_t need = (longest + NRG - 1) / NRG;
-  if (need <= 2) return launch_one<T, HD, GT, 2>(p, B, ns, tiles, st);
-  if (need <= 4) return launch_one<T, HD, GT, 4>(p, B, ns, tiles, st);
-  if (need <= 6) return launch_one<T, HD, GT, 6>(p, B, ns, tiles, st);
-  if (need <= 8 && GT <= 2) return launch_one<T, HD, GT, 8>(p, B, ns, tiles, st);
-  return launch_one<T, HD, GT, 4>(p, B, ns, tiles, st);
+  if (need <= 2) return launch_one<T, HD, GT, 2, MASKED>(p, B, ns, tiles, st);
+  if (need <= 4) return launch_one<T, HD, GT, 4, MASKED>(p, B, ns, tiles, st);
+  if (need <= 6) return launch_one<T, HD, GT, 6, MASKED>(p, B, ns, tiles, st);
+  if (need <= 8 && GT <= 2) return launch_one<T, HD, GT, 8, MASKED>(p, B, ns, tiles, st);
+  return launch_one<T, HD, GT, 4, MASKED>(p, B, ns, tiles, st);
 }
 
-template <typename T, int HD>
+template <typename T, int HD, bool MASKED = false>
 int launch_hd(const ClusterDecodeParams& p, int B, int ns, cudaStream_t st) {
   const int g = p.n_head / p.n_kv;
   const int gt = attn_decode_cluster_head_tile(B, p.n_kv, g);
   const int tiles = p.n_kv * (g / gt);
-  if (gt == 4) return launch_u<T, HD, 4>(p, B, ns, tiles, st);
-  if (gt == 2) return launch_u<T, HD, 2>(p, B, ns, tiles, st);
-  return launch_u<T, HD, 1>(p, B, ns, tiles, st);
+  if (gt == 4) return launch_u<T, HD, 4, MASKED>(p, B, ns, tiles, st);
+  if (gt == 2) return launch_u<T, HD, 2, MASKED>(p, B, ns, tiles, st);
+  return launch_u<T, HD, 1, MASKED>(p, B, ns, tiles, st);
 }
 
 }  // namespace
@@ -314,6 +339,35 @@ int attn_decode_cluster_launch(int dtype, const void* q, const void* k_cache, co
     return head_dim == 128 ? launch_hd<__nv_bfloat16, 128>(p, B, num_splits, st)
                            : launch_hd<__nv_bfloat16, 64>(p, B, num_splits, st);
   return head_dim == 128 ? launch_hd<__half, 128>(p, B, num_splits, st) : launch_hd<__half, 64>(p, B, num_splits, st);
+}
+
+bool attn_decode_masked_supports(int dtype, const WindowParams& w) {
+  if (dtype != LRI_BF16 && dtype != LRI_FP16) return false;
+  if (w.S != 1 || w.history >= 0 || w.d2 != 0 || !attn_decode_cluster_supports(1)) return false;
+  if (w.d1 % 8 || w.d1 > 128 || w.dv % 8 || w.dv > 128 || w.H % w.group) return false;
+  const int64_t kv_heads = w.H / w.group;
+  return w.q_head == w.d1 && w.q_row == static_cast<int64_t>(w.H) * w.d1 && w.k_row == w.d1 && w.v_row == w.dv &&
+         w.k_head == w.k_rows * w.d1 && w.v_head == w.k_rows * w.dv && w.k_batch == kv_heads * w.k_head &&
+         w.v_batch == kv_heads * w.v_head && kv_heads <= 65535 / w.group && aligned16(w.q) && aligned16(w.k) && aligned16(w.v);
+}
+
+int attn_decode_masked_launch(int dtype, const WindowParams& w, int B, cudaStream_t st) {
+  ClusterDecodeParams p{};
+  const int n_kv = w.H / w.group;
+  p.q = w.q, p.k_cache = w.k, p.v_cache = w.v, p.input_pos = w.input_pos, p.pos_is_i64 = w.pos_is_i64, p.out = w.out;
+  p.n_head = w.H, p.n_kv = n_kv, p.smax = w.k_rows, p.scale_log2 = w.scale * 1.4426950408889634f;
+  p.dim = w.d1, p.vdim = w.dv, p.window = w.window, p.chunk = w.chunk, p.sink = w.sink, p.out_ld = w.out_ld, p.out_scale = w.out_scale;
+  int64_t visible = w.k_rows < w.window ? w.k_rows : w.window;
+  if (w.chunk > 0 && w.chunk < visible) visible = w.chunk;
+  const int gt = attn_decode_cluster_head_tile(B, n_kv, w.group);
+  const int64_t base = static_cast<int64_t>(B) * n_kv * (w.group / gt), want = (2 * device_sm_count() + base - 1) / base;
+  const int64_t lim = want < 8 ? want : (base <= 4 ? 16 : 8);
+  int ns = 1;
+  while (ns * 2 <= lim && visible / (ns * 2) >= 32) ns *= 2;
+  const bool narrow = w.d1 <= 64 && w.dv <= 64;
+  if (dtype == LRI_BF16)
+    return narrow ? launch_hd<__nv_bfloat16, 64, true>(p, B, ns, st) : launch_hd<__nv_bfloat16, 128, true>(p, B, ns, st);
+  return narrow ? launch_hd<__half, 64, true>(p, B, ns, st) : launch_hd<__half, 128, true>(p, B, ns, st);
 }
 
 }  // namespace lri

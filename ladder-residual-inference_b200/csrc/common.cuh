@@ -66,6 +66,7 @@ enum Option {
   OPT_MOE_STREAM_PAIRS, // LRI_MOE_STREAM_PAIRS  (token, expert) pairs up to which experts run as streaming projections
   OPT_WINDOW_TC,        // LRI_WINDOW_TC      0: sliding-window attention always on the plain kernel
   OPT_HGRN2_BLOCKS,     // LRI_HGRN2_BLOCKS   0: the HGRN2 recurrence always runs token by token
+  OPT_SCAN_COLUMNS,     // LRI_SCAN_COLUMNS   state columns per lane of the recurrence kernel: 1, 2, 4 (0 = choose)
   OPT_COUNT
 };
 int option(int which);

@@ -58,7 +58,7 @@ __device__ __forceinline__ void tile_segments(int tile, const StreamKParams& p, 
 
 template <int EPI>
 struct Acc {
-  static constexpr int kCount = EPI == EPI_SWIGLU ? 2 : 1;  // accumulators per tile (up, gate)
+  static constexpr int kCount = EPI == EPI_SWIGLU || EPI == EPI_GLU ? 2 : 1;  // accumulators per tile (up, gate)
 };
 
 template <typename T, int BN, int EPI>
@@ -244,6 +244,12 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
           if (e < m)
             y[static_cast<int64_t>(e) * p.lin.n] =
                 swiglu_rounded<T>(rnd<T>(__uint_as_float(acc[0][e])), rnd<T>(__uint_as_float(acc[kAcc - 1][e])));
+      } else if (EPI == EPI_GLU) {
+#pragma unroll
+        for (int e = 0; e < BN; ++e)
+          if (e < m)
+            y[static_cast<int64_t>(e) * p.lin.n] =
+                Num<T>::from_f(clamped_glu(__uint_as_float(acc[kAcc - 1][e]), __uint_as_float(acc[0][e]), p.lin.ex.glu));
       }
     }
   }
@@ -266,7 +272,7 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
 // epilogue is applied.
 template <int EPI>
 struct FinishShape {
-  static constexpr int kTokens = EPI == EPI_SWIGLU ? 2 : 4;
+  static constexpr int kTokens = EPI == EPI_SWIGLU || EPI == EPI_GLU ? 2 : 4;
 };
 
 template <typename T, int BN, int EPI>
@@ -280,7 +286,7 @@ __global__ void __launch_bounds__(256) streamk_finish_kernel(const StreamKParams
   pdl_launch_dependents();
   if (nseg == 1 && EPI != EPI_QKV) return;
   const float* tile_partial = p.partial + static_cast<int64_t>(tile) * p.max_seg * kSlot;
-  if (EPI == EPI_SWIGLU) {
+  if (EPI == EPI_SWIGLU || EPI == EPI_GLU) {
     const int tok = blockIdx.y * FinishShape<EPI>::kTokens + (threadIdx.x >> 7);
     const int c = threadIdx.x & 127;
     const int64_t j = static_cast<int64_t>(tile) * kBM + c;
@@ -290,7 +296,8 @@ __global__ void __launch_bounds__(256) streamk_finish_kernel(const StreamKParams
       up += tile_partial[z * kSlot + tok * kBM + c];
       gate += tile_partial[z * kSlot + (BN + tok) * kBM + c];
     }
-    static_cast<T*>(p.lin.y)[static_cast<int64_t>(tok) * p.lin.n + j] = swiglu_rounded<T>(rnd<T>(up), rnd<T>(gate));
+    static_cast<T*>(p.lin.y)[static_cast<int64_t>(tok) * p.lin.n + j] =
+        EPI == EPI_GLU ? Num<T>::from_f(clamped_glu(gate, up, p.lin.ex.glu)) : swiglu_rounded<T>(rnd<T>(up), rnd<T>(gate));
     return;
   }
   const int tok = blockIdx.y * FinishShape<EPI>::kTokens + (threadIdx.x >> 6);
@@ -351,7 +358,7 @@ int launch(int dtype, const LinearParams& lin, float* partial, cudaStream_t st) 
   p.tiles = tiles_of(lin.n);
   p.total_kt = (lin.k + kBK - 1) / kBK;
   p.max_seg = max_segments(p.tiles);
-  const int64_t w_rows = EPI == EPI_SWIGLU ? 2 * static_cast<int64_t>(lin.n) : lin.n;
+  const int64_t w_rows = kAcc == 2 ? 2 * static_cast<int64_t>(lin.n) : lin.n;
   CUtensorMap tw, tx;
   int rc = make_tmap(&tw, dtype, lin.w, w_rows, lin.k, kBM);
   if (rc != LRI_OK) return rc;
@@ -380,6 +387,7 @@ template <typename T, int BN>
 int launch_epi(int dtype, int epi, const LinearParams& lin, float* partial, cudaStream_t st) {
   if (epi == EPI_PLAIN) return launch<T, BN, EPI_PLAIN>(dtype, lin, partial, st);
   if (epi == EPI_SWIGLU) return launch<T, BN, EPI_SWIGLU>(dtype, lin, partial, st);
+  if (epi == EPI_GLU) return launch<T, BN, EPI_GLU>(dtype, lin, partial, st);
   if (epi == EPI_F32) return launch<T, BN, EPI_F32>(dtype, lin, partial, st);
   return launch<T, BN, EPI_QKV>(dtype, lin, partial, st);
 }
@@ -396,7 +404,7 @@ int launch_bn(int dtype, int epi, const LinearParams& lin, float* partial, cudaS
 size_t gemm_streamk_workspace_bytes(int epi, int64_t m, int n) {
   if (m < 1 || m > kSplitKMaxRows || n < 1) return 0;
   const int tiles = tiles_of(n);
-  return static_cast<size_t>(tiles) * max_segments(tiles) * (epi == EPI_SWIGLU ? 2 : 1) * token_tile(m) * kBM *
+  return static_cast<size_t>(tiles) * max_segments(tiles) * (epi == EPI_SWIGLU || epi == EPI_GLU ? 2 : 1) * token_tile(m) * kBM *
          sizeof(float);
 }
 

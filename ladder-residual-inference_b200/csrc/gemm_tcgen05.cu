@@ -71,7 +71,7 @@ __device__ __forceinline__ WorkItem work_item(int item, const GemmGrid& g) {
 //   EPI_SWIGLU  the Q tile is BN/2 up rows followed by the BN/2 matching gate rows of w1, so that a
 //               thread finds up_j and gate_j of its token in the same accumulator row; it stores
 //               silu(gate) * up to h [m, I] (lin.y, lin.n = I)
-//   EPI_GLU     as SWIGLU with the clamped unit, on fp32 accumulators scaled per row (experts)
+//   EPI_GLU     as SWIGLU with the clamped unit, on fp32 accumulators (scaled per row for experts)
 //   EPI_F32     stores the fp32 accumulators
 //   EPI_QKV     a thread rotates the 16 adjacent pairs of each 32-column chunk of its token with the
 //               table row of the token's position and stores them to q_out / k-cache / v-cache
@@ -211,7 +211,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_p, const __grid_con
       const uint32_t tacc = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + a * kAccCols;
       if (!SWAP && kGlu) {
         const int64_t row = static_cast<int64_t>(w.tile_p) * kBM + i;
-        const float sc = EPI == EPI_GLU && row < shape.m ? lin.ex.row_scale[row] : 0.f;
+        const float sc = EPI == EPI_GLU && lin.ex.row_scale && row < shape.m ? lin.ex.row_scale[row] : 1.f;
 #pragma unroll 1
         for (int cc = 0; cc < BN / 2; cc += 32) {
           uint32_t up[32], gate[32];
@@ -505,9 +505,10 @@ int launch_experts(int dtype, const LinearParams& p, int max_tiles, cudaStream_t
 // prefill with the epilogue fused: the same tile choice, counted in output tiles
 template <typename T, int EPI>
 int launch_fused(int dtype, const LinearParams& p, int64_t m, cudaStream_t st) {
-  const int n_rows = EPI == EPI_SWIGLU ? 2 * p.n : p.n;       // rows of the weight
+  constexpr bool kGlu = EPI == EPI_SWIGLU || EPI == EPI_GLU;
+  const int n_rows = kGlu ? 2 * p.n : p.n;       // rows of the weight
   const int64_t mt = (m + kBM - 1) / kBM;
-  const int w256 = EPI == EPI_SWIGLU ? 128 : 256, w128 = EPI == EPI_SWIGLU ? 64 : 128;  // outputs per Q tile
+  const int w256 = kGlu ? 128 : 256, w128 = kGlu ? 64 : 128;  // outputs per Q tile
   const int64_t t256 = mt * ((p.n + w256 - 1) / w256), t128 = mt * ((p.n + w128 - 1) / w128);
   const int sms = sm_count();
   const int64_t cost256 = ((t256 + sms - 1) / sms) * 110, cost128 = ((t128 + sms - 1) / sms) * 100;
@@ -522,8 +523,9 @@ bool gemm_tcgen05_supports(int64_t m, int n, int k);
 // Prefill-sized projections (more than 64 token rows) with the SwiGLU or the RoPE + KV-cache
 // epilogue applied from the accumulator: p.m token rows, p.n outputs (SWIGLU: I), all epilogue fields set.
 bool gemm_tcgen05_fused_supports(int epi, const LinearParams& p, int64_t m) {
-  if (m <= 64 || !gemm_tcgen05_supports(m, epi == EPI_SWIGLU ? 2 * p.n : p.n, p.k)) return false;
-  if (epi == EPI_SWIGLU) return aligned16(p.y);
+  const bool glu = epi == EPI_SWIGLU || epi == EPI_GLU;
+  if (m <= 64 || !gemm_tcgen05_supports(m, glu ? 2 * p.n : p.n, p.k)) return false;
+  if (glu) return aligned16(p.y);
   if (epi == EPI_QKV) return p.head_dim % 32 == 0 && aligned16(p.rope_table);
   return false;
 }
@@ -533,6 +535,9 @@ int gemm_tcgen05_fused_launch(int dtype, int epi, const LinearParams& p, int64_t
   if (epi == EPI_SWIGLU)
     return dtype == LRI_BF16 ? launch_fused<__nv_bfloat16, EPI_SWIGLU>(dtype, p, m, st)
                              : launch_fused<__half, EPI_SWIGLU>(dtype, p, m, st);
+  if (epi == EPI_GLU)
+    return dtype == LRI_BF16 ? launch_fused<__nv_bfloat16, EPI_GLU>(dtype, p, m, st)
+                             : launch_fused<__half, EPI_GLU>(dtype, p, m, st);
   return dtype == LRI_BF16 ? launch_fused<__nv_bfloat16, EPI_QKV>(dtype, p, m, st)
                            : launch_fused<__half, EPI_QKV>(dtype, p, m, st);
 }

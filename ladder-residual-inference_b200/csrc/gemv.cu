@@ -8,7 +8,7 @@
 //   PLAIN   store (optionally + addend)                       wo / w2 / LM head
 //   SWIGLU  rows (j, I + j) -> silu(gate) * up                 w1
 //   F32     store the fp32 sums                                 projections that feed fp32 arithmetic
-//   GLU     as SWIGLU with the clamped unit of an expert         one (token, expert) pair per grid.x slice
+//   GLU     as SWIGLU with the clamped unit                       one row, or one (token, expert) pair per grid.x slice
 //   QKV     rotate adjacent pairs, scatter q / k-cache / v-cache   wqkv
 //   ARGMAX  no logits stored: arg-max over rows and ranks           LM head, greedy decoding (argmax.cuh)
 #include <cstdlib>
@@ -172,7 +172,7 @@ __global__ void __launch_bounds__(kGemvMaxWarps * 32) gemv_kernel(const LinearPa
   }
   if (EPI == EPI_GLU) {
     const int64_t jj = tile * (R / 2) + j;
-    const float sc = p.ex.row_scale[pair];
+    const float sc = p.ex.row_scale ? p.ex.row_scale[pair] : 1.0f;
     if (jj < p.n) static_cast<T*>(p.y)[pair * p.n + jj] = Num<T>::from_f(clamped_glu(sc * s1, sc * s0, p.ex.glu));
     return;
   }
@@ -266,7 +266,7 @@ int dispatch_epi(int epi, const LinearParams& p, cudaStream_t st) {
     case EPI_SWIGLU: return dispatch_m<T, EPI_SWIGLU>(p, st);
     case EPI_ARGMAX: return dispatch_m<T, EPI_ARGMAX>(p, st);
     case EPI_F32: return dispatch_m<T, EPI_F32>(p, st);
-    case EPI_GLU: {  // one row per expert pair
+    case EPI_GLU: {  // one row (per expert pair)
       if (rows_per_cta(p) == 8) return launch_gemv<T, 1, 8, 2, EPI_GLU>(p, st);
       return launch_gemv<T, 1, 4, 4, EPI_GLU>(p, st);
     }

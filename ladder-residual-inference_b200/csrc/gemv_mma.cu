@@ -27,6 +27,7 @@ constexpr int kMmaMaxWarps = 8;
 // projections use MT = 4, narrow ones keep MT = 1 so that there are enough CTAs.
 template <typename T, int NT, int MT, int EPI>
 __global__ void __launch_bounds__(kMmaMaxWarps * 32) gemv_mma_kernel(const LinearParams p) {
+  constexpr bool kGlu = EPI == EPI_SWIGLU || EPI == EPI_GLU;
   constexpr int BLK = 4 / MT;  // 32-element k blocks per warp iteration: 8 weight loads in flight per thread
   constexpr int kChunk = 32 * BLK;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, W = blockDim.x >> 5;
@@ -42,7 +43,7 @@ __global__ void __launch_bounds__(kMmaMaxWarps * 32) gemv_mma_kernel(const Linea
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
     int64_t row0, row1;
-    if (EPI == EPI_SWIGLU) {
+    if (kGlu) {
       int64_t j = (static_cast<int64_t>(blockIdx.x) * MT + mt) * 8 + a;
       j = j < p.n ? j : p.n - 1;
       row0 = j;        // up
@@ -154,6 +155,12 @@ __global__ void __launch_bounds__(kMmaMaxWarps * 32) gemv_mma_kernel(const Linea
           if (n + 1 < p.n) y[n + 1] = fin[t][2 + q];
           continue;
         }
+        if (EPI == EPI_GLU) {
+          const int64_t j = (static_cast<int64_t>(blockIdx.x) * MT + mt) * 8 + a;
+          if (j < p.n)
+            static_cast<T*>(p.y)[static_cast<int64_t>(tok) * p.n + j] = Num<T>::from_f(clamped_glu(fin[t][2 + q], fin[t][q], p.ex.glu));
+          continue;
+        }
         const float v0 = rnd<T>(fin[t][q]);      // row0 of this thread
         const float v1 = rnd<T>(fin[t][2 + q]);  // row1
         if (EPI == EPI_SWIGLU) {
@@ -182,7 +189,7 @@ int launch_mma(const LinearParams& p, cudaStream_t st) {
   const int nchunks = (p.k + kChunk - 1) / kChunk;
   int W = nchunks < kMmaMaxWarps ? nchunks : kMmaMaxWarps;
   W = W < 1 ? 1 : W;
-  const int64_t per_cta = (EPI == EPI_SWIGLU ? 8 : 16) * MT;
+  const int64_t per_cta = (EPI == EPI_SWIGLU || EPI == EPI_GLU ? 8 : 16) * MT;
   const int64_t grid = (p.n + per_cta - 1) / per_cta;
   LRI_CUDA(launch_pdl(gemv_mma_kernel<T, NT, MT, EPI>, dim3(static_cast<unsigned>(grid)), dim3(W * 32), 0, st, p));
   LRI_LAUNCH_CHECK("gemv_mma_kernel");
@@ -193,7 +200,8 @@ int launch_mma(const LinearParams& p, cudaStream_t st) {
 template <typename T, int NT, int EPI>
 int launch_tiles(const LinearParams& p, cudaStream_t st) {
   const int forced = option(OPT_GEMV_MT);
-  const int64_t tiles = (p.n + (EPI == EPI_SWIGLU ? 8 : 16) - 1) / (EPI == EPI_SWIGLU ? 8 : 16);
+  constexpr int kPer = EPI == EPI_SWIGLU || EPI == EPI_GLU ? 8 : 16;
+  const int64_t tiles = (p.n + kPer - 1) / kPer;
   int mt = tiles >= 4 * 296 ? 4 : (tiles >= 2 * 296 ? 2 : 1);
   if (forced) mt = forced;
   if (mt == 4) return launch_mma<T, NT, 4, EPI>(p, st);
@@ -207,6 +215,7 @@ int dispatch(int epi, const LinearParams& p, cudaStream_t st) {
   switch (epi) {
     case EPI_PLAIN: return one ? launch_tiles<T, 1, EPI_PLAIN>(p, st) : launch_tiles<T, 2, EPI_PLAIN>(p, st);
     case EPI_F32: return one ? launch_tiles<T, 1, EPI_F32>(p, st) : launch_tiles<T, 2, EPI_F32>(p, st);
+    case EPI_GLU: return one ? launch_tiles<T, 1, EPI_GLU>(p, st) : launch_tiles<T, 2, EPI_GLU>(p, st);
     case EPI_SWIGLU: return one ? launch_tiles<T, 1, EPI_SWIGLU>(p, st) : launch_tiles<T, 2, EPI_SWIGLU>(p, st);
     default: return one ? launch_tiles<T, 1, EPI_QKV>(p, st) : launch_tiles<T, 2, EPI_QKV>(p, st);
   }

@@ -325,15 +325,15 @@ __global__ void __launch_bounds__(128) window_attention_kernel(const WindowParam
   __syncwarp();
   const int64_t qpos = load_pos(p.input_pos, p.pos_is_i64, s);
   const int64_t kpos0 = p.history < 0 ? 0 : load_pos(p.input_pos, p.pos_is_i64, 0) - p.history;
-  int64_t lo = qpos - p.window + 1;
-  lo = lo < 0 ? 0 : lo;
+  const int64_t lo = first_visible(qpos, p.window, p.chunk);
   int64_t j0 = lo - kpos0, j1 = qpos - kpos0;  // visible key rows j0 .. j1
   j0 = j0 < 0 ? 0 : j0;
   j1 = j1 >= p.k_rows ? p.k_rows - 1 : j1;
-  const T* k = static_cast<const T*>(p.k) + b * p.k_batch + h * p.k_head;
+  const T* k = static_cast<const T*>(p.k) + b * p.k_batch + (h / p.group) * p.k_head;
   const T* k2 = static_cast<const T*>(p.k2) + b * p.k2_batch;
-  const T* v = static_cast<const T*>(p.v) + b * p.v_batch + h * p.v_head;
-  float m = -INFINITY, l = 0.f, o[NV];
+  const T* v = static_cast<const T*>(p.v) + b * p.v_batch + (h / p.group) * p.v_head;
+  float m = p.sink ? Num<T>::to_f(static_cast<const T*>(p.sink)[h]) : -INFINITY;
+  float l = p.sink ? 1.f : 0.f, o[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) o[i] = 0.f;
   for (int64_t jb = j0; jb <= j1; jb += 32) {
@@ -363,8 +363,8 @@ __global__ void __launch_bounds__(128) window_attention_kernel(const WindowParam
         if (lane + 32 * i < p.dv) o[i] = fmaf(w, Num<T>::to_f(vj[lane + 32 * i]), o[i]);
     }
   }
-  const float inv = l > 0.f ? 1.0f / l : 0.f;
-  T* out = static_cast<T*>(p.out) + (row * p.H + h) * p.dv;
+  const float inv = l > 0.f ? p.out_scale / l : 0.f;
+  T* out = static_cast<T*>(p.out) + row * p.out_ld + static_cast<int64_t>(h) * p.dv;
 #pragma unroll
   for (int i = 0; i < NV; ++i)
     if (lane + 32 * i < p.dv) out[lane + 32 * i] = Num<T>::from_f(o[i] * inv);
@@ -391,6 +391,13 @@ int window(const WindowParams& p, int64_t rows, cudaStream_t st) {
 bool dtype_ok(int dtype) { return dtype >= LRI_BF16 && dtype <= LRI_FP32; }
 
 }  // namespace
+
+int window_attention_plain_launch(int dtype, const WindowParams& p, int64_t rows, cudaStream_t st) {
+  if (dtype == LRI_BF16) return window<__nv_bfloat16>(p, rows, st);
+  if (dtype == LRI_FP16) return window<__half>(p, rows, st);
+  return window<float>(p, rows, st);
+}
+
 }  // namespace lri
 
 using namespace lri;
@@ -495,12 +502,11 @@ extern "C" int lri_window_attention(int dtype, const void* q, int64_t q_row, int
   p.k2 = k2, p.k2_batch = k2_batch, p.k2_row = k2_row, p.v = v, p.v_batch = v_batch, p.v_row = v_row, p.v_head = v_head;
   p.out = out, p.input_pos = input_pos, p.pos_is_i64 = pos_is_i64, p.history = history, p.k_rows = k_rows;
   p.window = window_size, p.scale = scale, p.S = S, p.H = heads, p.d1 = d1, p.d2 = d2, p.dv = dv;
+  p.group = 1, p.out_ld = static_cast<int64_t>(heads) * dv, p.out_scale = 1.0f;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (option(OPT_WINDOW_TC)) {
     if (latent_decode_supports(dtype, p)) return latent_decode_launch(dtype, p, B, scratch, scratch_bytes, st);
     if (window_attention_tc_supports(dtype, p, B)) return window_attention_tc_launch(dtype, p, B, st);
   }
-  if (dtype == LRI_BF16) return window<__nv_bfloat16>(p, rows, st);
-  if (dtype == LRI_FP16) return window<__half>(p, rows, st);
-  return window<float>(p, rows, st);
+  return window_attention_plain_launch(dtype, p, rows, st);
 }

@@ -1,4 +1,5 @@
-// Sliding-window prompt attention with keys in two parts (per head, and one shared by the heads) on tcgen05.
+// Masked prompt attention (sliding window, chunks) with keys in two parts (per key head, and one shared by the heads) on
+// tcgen05.
 //
 // A CTA owns 256 consecutive queries of one (sequence, head) as two groups of 128, and walks the key tiles of 64 that
 // any of them sees; both groups use a tile while it is in shared memory.  Per group and tile:
@@ -10,6 +11,8 @@
 // O is rescaled only when a row's maximum grows by more than 2^8.  Widths are cut in chunks of 64 elements; a tail
 // chunk is filled with zeros by the tensor maps, which view every operand as [rows, heads, width].  A row of a group
 // may see nothing of the group's first tiles (short windows): its maximum is then still -inf and P is zero.
+// Keys are rows gathered for the call (row j = position pos0 - history + j) or rows of a cache (row = position; C2 = 0,
+// key heads shared by groups of query heads).  A sink adds exp(sink) to a row's sum at the end.
 // Every mbarrier wait is bounded; on expiry a status word is set, TMEM is freed and the kernel returns.
 #include "latent_attention.cuh"
 #include "tcgen05.cuh"
@@ -31,22 +34,33 @@ struct TcParams {
   void* out;
   const void* input_pos;
   int pos_is_i64;
-  int S, H, dv;
-  int history, k_rows, window;
-  float scale_log2;
+  int S, H, dv, group;
+  int history, k_rows, window, chunk;
+  int64_t batch_rows, batch_heads;  // offsets of a sequence's keys in rows and in heads of the tensor maps
+  const void* sink;
+  int64_t out_ld;
+  float scale_log2, out_scale;
 };
 
 struct Tiles {
   int lo, n;  // first key tile and number of tiles
 };
 
-// Tiles seen by queries q0 .. q_end - 1 (key row of query i is history + i; rows below j_min do not exist)
-__device__ __forceinline__ Tiles tiles_of_queries(const TcParams& p, int q0, int q_end, int j_min) {
-  int first = p.history + q0 - p.window + 1;
-  first = first > j_min ? first : j_min;
+// First key row seen from key row j (rows below j_min do not exist; chunks need row = position)
+__device__ __forceinline__ int first_row(const TcParams& p, int j, int j_min) {
+  int lo = j - p.window + 1;
+  lo = lo > j_min ? lo : j_min;
+  if (p.chunk > 0) {
+    const int c = j / p.chunk * p.chunk;
+    lo = lo > c ? lo : c;
+  }
+  return lo;
+}
+// Tiles seen by queries q0 .. q_end - 1 (key row of query i is history + i)
+__device__ __forceinline__ Tiles tiles_of_queries(const TcParams& p, int history, int q0, int q_end, int j_min) {
   Tiles t;
-  t.lo = first / kKeys;
-  t.n = (p.history + q_end - 1) / kKeys - t.lo + 1;
+  t.lo = first_row(p, history + q0, j_min) / kKeys;
+  t.n = (history + q_end - 1) / kKeys - t.lo + 1;
   return t;
 }
 
@@ -123,7 +137,8 @@ window_attention_tc_kernel(const __grid_constant__ CUtensorMap tq1, const __grid
 
   int64_t pos0 = load_pos(p.input_pos, p.pos_is_i64, 0);
   pos0 = pos0 < 0 ? 0 : pos0;
-  const int j_min = pos0 < p.history ? p.history - static_cast<int>(pos0) : 0;  // key row of position 0
+  const int history = p.history < 0 ? static_cast<int>(pos0) : p.history;  // key row of the first query
+  const int j_min = pos0 < history ? history - static_cast<int>(pos0) : 0;  // key row of position 0
   Tiles gt[kGroups], all;
   int groups = 0;
 #pragma unroll
@@ -132,7 +147,7 @@ window_attention_tc_kernel(const __grid_constant__ CUtensorMap tq1, const __grid
     const int e = a + kRows < p.S ? a + kRows : p.S;
     gt[g] = Tiles{0, 0};
     if (a < p.S) {
-      gt[g] = tiles_of_queries(p, a, e, j_min);
+      gt[g] = tiles_of_queries(p, history, a, e, j_min);
       groups = g + 1;
     }
   }
@@ -158,13 +173,14 @@ window_attention_tc_kernel(const __grid_constant__ CUtensorMap tq1, const __grid
         if (!mbar_wait(kv_empty0 + 8 * s, (round & 1u) ^ 1u, &abort_flag, 1, &g_window_tc_status)) break;
         mbar_expect_tx(kv_full0 + 8 * s, Z::kStage);
         const uint32_t dst = kv_smem + s * Z::kStage;
-        const int row = b * p.k_rows + (all.lo + j) * kKeys;
+        const int row = static_cast<int>(b * p.batch_rows) + (all.lo + j) * kKeys;
+        const int kv_head = static_cast<int>(b * p.batch_heads) + head / p.group;
 #pragma unroll
-        for (int c = 0; c < C1; ++c) tma_load_3d(dst + c * kKvChunk, &tk1, kv_full0 + 8 * s, c * 64, head, row);
+        for (int c = 0; c < C1; ++c) tma_load_3d(dst + c * kKvChunk, &tk1, kv_full0 + 8 * s, c * 64, kv_head, row);
 #pragma unroll
         for (int c = 0; c < C2; ++c) tma_load_3d(dst + (C1 + c) * kKvChunk, &tk2, kv_full0 + 8 * s, c * 64, 0, row);
 #pragma unroll
-        for (int c = 0; c < CV; ++c) tma_load_3d(dst + (kQk + c) * kKvChunk, &tv, kv_full0 + 8 * s, c * 64, head, row);
+        for (int c = 0; c < CV; ++c) tma_load_3d(dst + (kQk + c) * kKvChunk, &tv, kv_full0 + 8 * s, c * 64, kv_head, row);
       }
     }
   } else if (warp == 1) {
@@ -225,10 +241,10 @@ window_attention_tc_kernel(const __grid_constant__ CUtensorMap tq1, const __grid
     const uint32_t lane_off = static_cast<uint32_t>(quarter * 32) << 16;
     const uint32_t tm = tmem_base + lane_off + g * kGroupCols;
     const int qa = q0 + g * kRows;
-    const int jq = p.history + qa + i;  // key row of this thread's query
-    const int lo_i = jq - p.window + 1 > j_min ? jq - p.window + 1 : j_min;
-    const int full_lo = p.history + qa + kRows - p.window;  // from this key row on every query's window has begun
-    const int full_hi = p.history + qa;                     // up to here no query is behind its key
+    const int jq = history + qa + i;  // key row of this thread's query
+    const int lo_i = first_row(p, jq, j_min);
+    const int full_lo = first_row(p, history + qa + kRows - 1, j_min);  // from this key row on every query's window has begun
+    const int full_hi = history + qa;                                   // up to here no query is behind its key
     const int lo_tile = g == 0 ? gt[0].lo : gt[1].lo, n_tiles = g == 0 ? gt[0].n : gt[1].n;
     float m_ref = -INFINITY, l = 0.f;
     bool alive = n_tiles > 0;
@@ -308,9 +324,10 @@ window_attention_tc_kernel(const __grid_constant__ CUtensorMap tq1, const __grid
       const bool done = mbar_wait(o_done(g, ob), (static_cast<uint32_t>(n_tiles - 1) >> 1) & 1u, &abort_flag, 7, &g_window_tc_status);
       if (__all_sync(0xffffffffu, done)) {
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const float inv = l > 0.f ? 1.0f / l : 0.f;
+        if (p.sink) l += exp2f(fmaf(Num<T>::to_f(static_cast<const T*>(p.sink)[head]), 1.4426950408889634f, m_ref == -INFINITY ? 0.f : -m_ref));
+        const float inv = l > 0.f ? p.out_scale / l : 0.f;
         const int s_idx = qa + i;
-        T* dst = static_cast<T*>(p.out) + ((static_cast<int64_t>(b) * p.S + s_idx) * p.H + head) * p.dv;
+        T* dst = static_cast<T*>(p.out) + (static_cast<int64_t>(b) * p.S + s_idx) * p.out_ld + static_cast<int64_t>(head) * p.dv;
 #pragma unroll 1
         for (int cc = 0; cc < CV * 64; cc += 32) {
           uint32_t o[32];
@@ -348,16 +365,26 @@ int launch(int dtype, const WindowParams& w, int B, cudaStream_t st) {
   using Z = Sizes<T, C1, C2, CV>;
   CUtensorMap tq1, tq2, tk1, tk2, tv;
   const T* q = static_cast<const T*>(w.q);
-  const int64_t q_rows = static_cast<int64_t>(B) * w.S, k_rows = static_cast<int64_t>(B) * w.k_rows;
+  const bool cached = w.history < 0;
+  const int kv_heads = w.H / w.group;
+  const int64_t q_rows = static_cast<int64_t>(B) * w.S, k_rows = cached ? w.k_rows : B * w.k_rows;
+  const int64_t all_heads = cached ? static_cast<int64_t>(B) * kv_heads : kv_heads;
   int rc = make_tmap_heads(&tq1, dtype, q, q_rows, w.q_row, w.H, w.q_head, w.d1, kRows);
-  if (rc == LRI_OK) rc = make_tmap_heads(&tq2, dtype, q + w.d1, q_rows, w.q_row, w.H, w.q_head, w.d2, kRows);
-  if (rc == LRI_OK) rc = make_tmap_heads(&tk1, dtype, w.k, k_rows, w.k_row, w.H, w.k_head, w.d1, kKeys);
-  if (rc == LRI_OK) rc = make_tmap_heads(&tk2, dtype, w.k2, k_rows, w.k2_row, 1, w.k2_row, w.d2, kKeys);
-  if (rc == LRI_OK) rc = make_tmap_heads(&tv, dtype, w.v, k_rows, w.v_row, w.H, w.v_head, w.dv, kKeys);
+  if (rc == LRI_OK) rc = make_tmap_heads(&tk1, dtype, w.k, k_rows, w.k_row, all_heads, w.k_head, w.d1, kKeys);
+  if (rc == LRI_OK) rc = make_tmap_heads(&tv, dtype, w.v, k_rows, w.v_row, all_heads, w.v_head, w.dv, kKeys);
+  if (C2 > 0) {
+    if (rc == LRI_OK) rc = make_tmap_heads(&tq2, dtype, q + w.d1, q_rows, w.q_row, w.H, w.q_head, w.d2, kRows);
+    if (rc == LRI_OK) rc = make_tmap_heads(&tk2, dtype, w.k2, k_rows, w.k2_row, 1, w.k2_row, w.d2, kKeys);
+  } else {
+    tq2 = tq1, tk2 = tk1;  // not read
+  }
   if (rc != LRI_OK) return rc;
   TcParams p{};
   p.out = w.out, p.input_pos = w.input_pos, p.pos_is_i64 = w.pos_is_i64;
   p.S = w.S, p.H = w.H, p.dv = w.dv, p.history = w.history, p.k_rows = static_cast<int>(w.k_rows);
+  p.group = w.group, p.batch_rows = cached ? 0 : w.k_rows, p.batch_heads = cached ? kv_heads : 0;
+  p.chunk = static_cast<int>(w.chunk < (1 << 30) ? w.chunk : 0);
+  p.sink = w.sink, p.out_ld = w.out_ld, p.out_scale = w.out_scale;
   p.window = static_cast<int>(w.window < (1 << 30) ? w.window : (1 << 30));
   p.scale_log2 = w.scale * 1.4426950408889634f;
   auto kern = window_attention_tc_kernel<T, C1, C2, CV>;
@@ -372,6 +399,10 @@ int launch(int dtype, const WindowParams& w, int B, cudaStream_t st) {
 
 template <typename T>
 int dispatch(int dtype, const WindowParams& w, int B, cudaStream_t st) {
+  if (w.d2 == 0) {
+    if (w.d1 <= 64) return w.dv <= 64 ? launch<T, 1, 0, 1>(dtype, w, B, st) : launch<T, 1, 0, 2>(dtype, w, B, st);
+    return w.dv <= 64 ? launch<T, 2, 0, 1>(dtype, w, B, st) : launch<T, 2, 0, 2>(dtype, w, B, st);
+  }
   if (w.d1 <= 64) return w.dv <= 64 ? launch<T, 1, 1, 1>(dtype, w, B, st) : launch<T, 1, 1, 2>(dtype, w, B, st);
   return w.dv <= 64 ? launch<T, 2, 1, 1>(dtype, w, B, st) : launch<T, 2, 1, 2>(dtype, w, B, st);
 }
@@ -380,10 +411,19 @@ int dispatch(int dtype, const WindowParams& w, int B, cudaStream_t st) {
 
 bool window_attention_tc_supports(int dtype, const WindowParams& w, int B) {
   if (dtype != LRI_BF16 && dtype != LRI_FP16) return false;
-  if (w.history < 0 || w.S < 16 || !(w.scale > 0.f)) return false;
-  if (w.d1 < 8 || w.d1 > 128 || w.d1 % 8 || w.d2 < 8 || w.d2 > 64 || w.d2 % 8 || w.dv < 8 || w.dv > 128 || w.dv % 8) return false;
-  if (w.q_row % 8 || w.q_head % 8 || w.k_row % 8 || w.k_head % 8 || w.k2_row % 8 || w.v_row % 8 || w.v_head % 8) return false;
+  if (w.S < 16 || !(w.scale > 0.f)) return false;
+  if (w.d1 < 8 || w.d1 > 128 || w.d1 % 8 || w.d2 > 64 || w.d2 % 8 || w.dv < 8 || w.dv > 128 || w.dv % 8) return false;
+  if (w.q_row % 8 || w.q_head % 8 || w.k_row % 8 || w.k_head % 8 || w.v_row % 8 || w.v_head % 8 || w.out_ld % 8) return false;
   if (w.q_head < 8 || w.k_head < 8 || w.v_head < 8) return false;
+  if (w.history < 0) {
+    // rows of a cache [sequence, key head, position]: the sequences' heads follow one another
+    const int64_t g = w.H / w.group;
+    if (w.d2 != 0 || w.k_batch != g * w.k_head || w.v_batch != g * w.v_head) return false;
+    if (!aligned16(w.q) || !aligned16(w.k) || !aligned16(w.v) || !aligned16(w.out)) return false;
+    return B <= 65535 && w.H <= 65535 && w.k_rows < (1ll << 30) && B * g < (1ll << 31) &&
+           static_cast<int64_t>(B) * w.S + 2 * kRows < (1ll << 31);
+  }
+  if (w.d2 < 8 || w.k2_row % 8 || w.group != 1 || w.chunk > 0) return false;
   // the rows of the sequences follow one another
   if (w.k_batch != w.k_rows * w.k_row || w.k2_batch != w.k_rows * w.k2_row || w.v_batch != w.k_rows * w.v_row) return false;
   if (w.k_rows < w.history + w.S) return false;

@@ -7,7 +7,7 @@
 namespace lri {
 
 // EPI_F32: like PLAIN with an fp32 output (no rounding, no addend).  EPI_GLU: like SWIGLU (weight rows [up | gate])
-// with the clamped gated linear unit in fp32 and a scale per input row (mixture-of-experts feed-forward).
+// with the clamped gated linear unit in fp32 and an optional scale per input row (experts).
 enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_QKV = 2, EPI_ARGMAX = 3, EPI_F32 = 4, EPI_GLU = 5 };
 constexpr int kGemvMaxRows = 8;
 
@@ -32,7 +32,7 @@ struct ExpertArgs {
   int pairs, rows_per_input;
   const int* tiles;
   int64_t matrix_rows;     // weight rows of one expert
-  const float* row_scale;  // GLU epilogue: factor on the input of a pair (or of a row of the tiled input)
+  const float* row_scale;  // GLU epilogue: factor on the input of a pair (or of a row of the tiled input), or NULL
   GluParams glu;
 };
 
@@ -138,6 +138,8 @@ void gemm_streamk_plan(int epi, int64_t m, int n, int k, int* tiles, int* k_tile
                        int* token_tile_out);
 
 // elementwise epilogues used after the GEMM on the prefill path
+// h[r, j] = clamped unit of ug[r, n + j] (gate) and ug[r, j] (up), fp32 in
+int glu_rows_launch(int dtype, const float* ug /*[m, 2n]*/, void* h /*[m, n]*/, int64_t m, int n, const GluParams& glu, cudaStream_t st);
 int swiglu_rows_launch(int dtype, const void* ug /*[m, 2n]*/, void* h /*[m, n]*/, int64_t m, int n, cudaStream_t st);
 int qkv_scatter_launch(int dtype, const void* qkv /*[m, (nh+2nkv)*hd]*/, const LinearParams& p, cudaStream_t st);
 int add_rows_launch(int dtype, void* y, const void* addend, int64_t count, cudaStream_t st);

@@ -49,6 +49,7 @@ const OptionSpec kOptionSpecs[OPT_COUNT] = {
     {"moe_stream_pairs", "LRI_MOE_STREAM_PAIRS", 10, 0, 65535},
     {"window_tc", "LRI_WINDOW_TC", 1, 0, 1},
     {"hgrn2_blocks", "LRI_HGRN2_BLOCKS", 1, 0, 1},
+    {"scan_columns", "LRI_SCAN_COLUMNS", 0, 0, 4},
 };
 
 bool option_value_ok(int which, int v) {
@@ -57,7 +58,7 @@ bool option_value_ok(int which, int v) {
   if (which == OPT_GEMV_R) return v == 0 || v == 2 || v == 4 || v == 8;
   if (which == OPT_GEMV_U) return v == 0 || v == 2;
   if (which == OPT_GEMV_MT) return v == 0 || v == 1 || v == 2 || v == 4;
-  if (which == OPT_ATTN_HEAD_TILE) return v == 0 || v == 1 || v == 2 || v == 4;
+  if (which == OPT_ATTN_HEAD_TILE || which == OPT_SCAN_COLUMNS) return v == 0 || v == 1 || v == 2 || v == 4;
   return true;
 }
 
@@ -455,6 +456,47 @@ extern "C" int lri_gateup_swiglu(int dtype, const void* x, const void* w1, void*
   rc = gemm_launch(dtype, x, w1, workspace, M, 2 * I, K, st);
   if (rc != LRI_OK) return rc;
   return swiglu_rows_launch(dtype, workspace, h, M, I, st);
+}
+
+// The fused forms need K in 16-byte steps; everything else goes through fp32 products and an elementwise kernel.
+static bool glu_fused(int dtype, int64_t M, int I, int K) {
+  if (dtype == LRI_FP32 || K % 8 != 0) return false;
+  return M <= kGemvMmaMaxRows || (I % 8 == 0 && M > kSplitKMaxRows && current_gemm_backend() != LRI_GEMM_SIMT);
+}
+static size_t glu_raw_bytes(int dtype, int64_t M, int I, int K) {
+  return glu_fused(dtype, M, I, K) ? 0 : static_cast<size_t>(M) * 2 * static_cast<size_t>(I) * sizeof(float);
+}
+extern "C" size_t lri_gateup_glu_workspace_bytes(int dtype, int64_t M, int I, int K) {
+  if (M < 0 || I <= 0 || K <= 0) return 0;
+  const size_t sk = dtype != LRI_FP32 && K % 8 == 0 ? streamk_bytes(EPI_GLU, M, I) : 0;
+  return max_size(glu_raw_bytes(dtype, M, I, K), sk);
+}
+
+extern "C" int lri_gateup_glu(int dtype, const void* x, const void* w1, void* h, int64_t M, int I, int K, float alpha,
+                              float limit, float offset, void* workspace, size_t workspace_bytes, lri_stream_t stream) {
+  LRI_REQUIRE(dtype >= LRI_BF16 && dtype <= LRI_FP32, LRI_ERR_UNSUPPORTED, "gateup_glu: dtype %d", dtype);
+  LRI_REQUIRE(x && w1 && h, LRI_ERR_ARG, "gateup_glu: NULL pointer");
+  LRI_REQUIRE(M >= 0 && M < (1ll << 31) && I > 0 && K > 0, LRI_ERR_ARG, "gateup_glu: M=%lld I=%d K=%d", (long long)M, I, K);
+  if (M == 0) return LRI_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  LinearParams p{};
+  p.x = x, p.w = w1, p.y = h, p.m = static_cast<int>(M), p.n = I, p.k = K;
+  p.ex.glu = GluParams{alpha, limit, offset};
+  if (dtype != LRI_FP32 && K % 8 == 0 && aligned16(x) && aligned16(w1)) {
+    if (M == 1) return gemv_launch(dtype, EPI_GLU, p, st);
+    if (M <= streaming_rows()) return gemv_mma_launch(dtype, EPI_GLU, p, st);
+    if (streamk_rows(M) && gemm_streamk_supports(EPI_GLU, p, workspace, workspace_bytes))
+      return gemm_streamk_launch(dtype, EPI_GLU, p, workspace, workspace_bytes, st);
+    if (M <= kGemvMmaMaxRows) return gemv_mma_launch(dtype, EPI_GLU, p, st);
+    if (current_gemm_backend() != LRI_GEMM_SIMT && gemm_tcgen05_fused_supports(EPI_GLU, p, M))
+      return gemm_tcgen05_fused_launch(dtype, EPI_GLU, p, M, st);
+  }
+  const size_t need = static_cast<size_t>(M) * 2 * static_cast<size_t>(I) * sizeof(float);
+  LRI_REQUIRE(workspace && workspace_bytes >= need && aligned16(workspace), LRI_ERR_WORKSPACE,
+              "gateup_glu: workspace of %zu bytes (16-byte aligned) required", need);
+  int rc = lri_linear_f32(dtype, x, w1, static_cast<float*>(workspace), M, 2 * I, K, nullptr, 0, stream);
+  if (rc != LRI_OK) return rc;
+  return glu_rows_launch(dtype, static_cast<const float*>(workspace), h, M, I, p.ex.glu, st);
 }
 
 static size_t qkv_raw_bytes(int64_t M, int n_head, int n_kv, int head_dim) {

@@ -97,7 +97,27 @@ int launch(const void* x, const void* w, const void* addend, void* y, int64_t m,
   return LRI_OK;
 }
 
+template <typename T>
+__global__ void __launch_bounds__(256) glu_rows_kernel(const float* ug, T* h, int64_t m, int n, GluParams glu) {
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
+  if (i >= m * n) return;
+  const int64_t r = i / n, j = i - r * n;
+  h[i] = Num<T>::from_f(clamped_glu(ug[r * 2 * n + n + j], ug[r * 2 * n + j], glu));
+}
+
 }  // namespace
+
+int glu_rows_launch(int dtype, const float* ug, void* h, int64_t m, int n, const GluParams& glu, cudaStream_t st) {
+  const unsigned grid = static_cast<unsigned>((m * n + 255) / 256);
+  if (dtype == LRI_FP32)
+    glu_rows_kernel<float><<<grid, 256, 0, st>>>(ug, static_cast<float*>(h), m, n, glu);
+  else if (dtype == LRI_BF16)
+    glu_rows_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(ug, static_cast<__nv_bfloat16*>(h), m, n, glu);
+  else
+    glu_rows_kernel<__half><<<grid, 256, 0, st>>>(ug, static_cast<__half*>(h), m, n, glu);
+  LRI_LAUNCH_CHECK("glu_rows_kernel");
+  return LRI_OK;
+}
 
 int gemm_generic_launch(int dtype, const void* x, const void* w, const void* addend, void* y, bool out_f32, int64_t m,
                         int n, int k, cudaStream_t st) {

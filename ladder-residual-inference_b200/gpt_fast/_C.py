@@ -100,6 +100,29 @@ _SIGNATURES = {
                                c_int64, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p]),
     "lri_moe_down": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int,
                              c_void_p]),
+    "lri_join_streams": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
+                                 c_void_p, c_int64, c_int, c_int, c_void_p]),
+    "lri_embed_streams": (c_int, [c_int, c_void_p, c_void_p, c_int, c_int64, c_float, c_void_p, c_void_p, c_void_p, c_float,
+                                  c_void_p, c_int64, c_int, c_int, c_void_p]),
+    "lri_gateup_glu_workspace_bytes": (c_size_t, [c_int, c_int64, c_int, c_int]),
+    "lri_gateup_glu": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_float, c_float, c_float,
+                               c_void_p, c_size_t, c_void_p]),
+    "lri_grouped_prepare": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_int,
+                                    c_int, c_float, c_void_p, c_int64, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                    c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_row_squares": (c_int, [c_void_p, c_int64, c_int64, c_int, c_int64, c_int, c_void_p, c_int64, c_void_p]),
+    "lri_grouped_attention": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_float, c_void_p,
+                                      c_int, c_int64, c_int64, c_int64, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
+                                      c_void_p]),
+    "lri_state_scan": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
+                               c_void_p, c_int, c_void_p, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_delta_prepare": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_void_p,
+                                  c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                  c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_logistic_decay": (c_int, [c_int, c_void_p, c_void_p, c_float, c_int64, c_int, c_void_p]),
+    "lri_head_norm_gate": (c_int, [c_int, c_void_p, c_void_p, c_float, c_void_p, c_int64, c_int, c_float, c_void_p, c_int64,
+                                   c_int64, c_int, c_int, c_void_p]),
+    "lri_round_columns": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int, c_void_p, c_int64, c_void_p]),
     "lri_comm_status": (c_int, [c_void_p, c_void_p]),
     "lri_comm_destroy": (c_int, [c_void_p]),
 }
@@ -112,6 +135,7 @@ for _name, (_res, _args) in _SIGNATURES.items():
 EXPORTED_SYMBOLS = tuple(_SIGNATURES)
 
 BF16, FP16, FP32 = 0, 1, 2
+GATE_SIGMOID, GATE_SILU = 0, 1
 GEMM_AUTO, GEMM_TCGEN05, GEMM_SIMT = 0, 1, 2
 
 

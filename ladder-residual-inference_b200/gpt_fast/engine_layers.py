@@ -1,21 +1,24 @@
-"""Whole-model forward of designs given as a list of layers (token mixer + feed-forward, each in a gated, doubly
-normed residual branch) on preallocated buffers.
+"""Whole-model forward of designs given as a list of layers (token mixer + feed-forward) on preallocated buffers.
 
 The heads (logits, last position, greedy, sampling), the tensor-parallel plumbing and the calling conventions are
-`engine.Engine`'s; what differs is the body between embedding and final norm:
+`engine.Engine`'s; what differs is the body between embedding and final norm.  Every sublayer is
 
-    h        = norm(x)                                             first one fused with the embedding
-    gate|in  = in_proj(h)                                          fp32, one projection per sublayer
-    y        = mixer(in)  or  experts(h, router logits in `in`)
-    x, h     = x + post_norm(sigmoid(gate + bias) * y), next norm  one fused pass over the fp32 residual
+    h      = norm(residual)                           prepared by the step before it
+    in     = in_proj(h)                               fp32, one projection per sublayer (none for a dense gated unit)
+    y      = sublayer(in or h)
+    join   the result enters the fp32 residual and the next sublayer's norm is taken, in one fused pass
+
+and there are two kinds of residual: one stream with a gate and a post norm on the result (`GatedResidual`), or several
+streams that a sublayer mixes (`StreamBranch`).
 
 A forward reads positions from the device and can be captured in a CUDA graph.  A batch row's first position decides
 whether a recurrence starts anew (0) or continues, so a row is reused by feeding position 0 again.
 """
 import torch
+import torch.distributed as dist
 
 from .engine import Engine
-from .mixers import LatentAttention
+from .mixers import LatentAttention, StreamBranch, _offsets
 
 
 class LayerEngine(Engine):
@@ -29,26 +32,36 @@ class LayerEngine(Engine):
         def buf(n, cols, dt=dtype):
             return torch.empty(n, cols, dtype=dt, device=device)
 
+        branches = self.branches = [br for b in self.model.layers for br in (b.mixer, b.mlp) if br is not None]
+        subs = [m for br in branches for m in ((br.sublayer.left, br.sublayer.right) if br.sublayer.kind == "parallel" else (br.sublayer,))]
         mixers = [b.mixer.sublayer for b in self.model.layers]
-        latent = [m for m in mixers if m.kind == "latent_attention"]
-        hgrn = [m for m in mixers if m.kind == "hgrn2"]
-        moes = [b.mlp.sublayer for b in self.model.layers if b.mlp is not None]
-        branches = [b.mixer for b in self.model.layers] + [b.mlp for b in self.model.layers if b.mlp is not None]
 
-        self.resid = buf(rows, self.d, torch.float32)
+        def of(kind):
+            return [m for m in subs if m.kind == kind]
+
+        def most(ms, f):
+            return max((f(m) for m in ms), default=0)
+
+        streams = getattr(cfg, "streams", None)
+        self.resid = torch.empty(rows, self.d, dtype=torch.float32, device=device) if streams is None else \
+            torch.empty(rows, streams, self.d, dtype=torch.float32, device=device)
         self.normed, self.part = buf(rows, self.d), buf(rows, self.d)
-        self.proj = buf(rows, max(br.in_proj.weight.shape[0] for br in branches), torch.float32)
+        in_rows = [br.in_proj.weight.shape[0] for br in branches if br.in_proj is not None]
+        self.proj = buf(rows, max(in_rows, default=1), torch.float32)
         self.y = buf(rows, max(m.out_width for m in mixers))
 
-        def workspace(size_fn, n):
-            size = max(size_fn(rows, n), size_fn(min(rows, 64), n))
+        def workspace(size_fn, *ns):
+            size = max((max(size_fn(rows, n), size_fn(min(rows, 64), n)) for n in ns), default=0)
             return torch.empty(size, dtype=torch.uint8, device=device) if size else None
 
-        self.ws_in = workspace(ops.linear_f32_workspace_bytes, self.proj.shape[1])
+        self.ws_in = workspace(ops.linear_f32_workspace_bytes, *in_rows)
         self.ws_out = workspace(ops.linear_workspace_bytes, self.d)
 
+        latent, hgrn, moes, glus = of("latent_attention"), of("hgrn2"), of("moe"), of("glu")
+        grouped, delta, gla = of("chunked_attention"), of("gated_delta"), of("gla")
+        if latent or grouped:
+            self.q = buf(rows, max(most(latent, lambda m: m.q_rows), most(grouped, lambda m: m.heads * m.dim)))
         if latent:
-            self.q = buf(rows, max(m.q_rows for m in latent))
             self.q_latent = buf(max_batch, max(m.heads * (m.rank + m.rot_dim) for m in latent))
             self.o_latent = buf(max_batch, max(m.heads * m.rank for m in latent))
             # what a prompt portion sees (history + its own tokens) never exceeds the cache
@@ -60,26 +73,41 @@ class LayerEngine(Engine):
                        for m in latent for b in range(1, max_batch + 1))
             self.attn_scratch = torch.empty(max(size, 16), dtype=torch.uint8, device=device)
             self.ws_expand = workspace(ops.linear_workspace_bytes, self.win_kv.shape[1])
+        if grouped and self.comm.world > 1:
+            self.qk_sums = buf(rows, 2, torch.float32)
         if hgrn:
             size = max(ops.hgrn2_workspace_bytes(dtype, b, max_seq, m.heads, m.dim, m.vdim)
                        for m in hgrn for b in range(1, max_batch + 1))
             self.ws_hgrn = torch.empty(max(size, 16), dtype=torch.uint8, device=device)
+        if delta or gla:
+            scans = delta + gla
+            self.low = buf(rows, max(most(scans, lambda m: m.a2.shape[1]), most(delta, lambda m: m.g2.shape[1])))
+            self.decay = buf(rows, most(scans, lambda m: m.heads * m.dim), torch.float32)
+            self.scan_o = buf(rows, most(scans, lambda m: m.out_width), torch.float32)
+            self.ws_low = workspace(ops.linear_f32_workspace_bytes, *[m.a2.shape[0] for m in scans], *[m.g2.shape[0] for m in delta])
+        if delta:
+            qk = most(delta, lambda m: m.kv_heads * m.dim)
+            self.scan_q, self.scan_k = buf(rows, qk, torch.float32), buf(rows, qk, torch.float32)
+            self.scan_v = buf(rows, most(delta, lambda m: m.out_width), torch.float32)
+            self.scan_gate = buf(rows, most(delta, lambda m: m.out_width), torch.float32)
+            self.scan_beta, self.scan_kq = buf(rows, most(delta, lambda m: m.heads), torch.float32), \
+                buf(rows, most(delta, lambda m: m.kv_heads), torch.float32)
+        if glus:
+            self.glu_hidden = buf(rows, most(glus, lambda m: m.ff))
+            self.ws_glu = workspace(lambda n, m: ops.gateup_glu_workspace_bytes(dtype, n, m.ff, self.d), *glus)
         if moes:
-            def most(f):
-                return max(f(m) for m in moes)
-
             def ints(n):
                 return torch.zeros(n, dtype=torch.int32, device=device)
 
-            pairs = rows * most(lambda m: m.top)
-            tiles = most(lambda m: ops.moe_max_tiles(rows, m.top, m.experts))
+            pairs = rows * most(moes, lambda m: m.top)
+            tiles = most(moes, lambda m: ops.moe_max_tiles(rows, m.top, m.experts))
             packed = any(ops.moe_packs(dtype, rows, m.top, self.d, m.ff) for m in moes)
             out_rows = max(pairs, 128 * tiles) if packed else pairs
             self.moe_ids, self.moe_rank, self.moe_slots = ints(pairs), ints(pairs), ints(pairs)
             self.moe_scores = torch.empty(pairs, dtype=torch.float32, device=device)
-            self.moe_counts, self.moe_first = ints(most(lambda m: m.experts)), ints(most(lambda m: m.experts))
+            self.moe_counts, self.moe_first = ints(most(moes, lambda m: m.experts)), ints(most(moes, lambda m: m.experts))
             self.moe_tiles = ints(1 + tiles)
-            self.moe_hidden = buf(out_rows, most(lambda m: m.ff))
+            self.moe_hidden = buf(out_rows, most(moes, lambda m: m.ff))
             self.moe_out = buf(out_rows, self.d)
             if packed:
                 self.moe_packed = buf(128 * tiles, self.d)
@@ -88,10 +116,11 @@ class LayerEngine(Engine):
         self.ready = True
 
     # ------------------------------------------------------------------------------------------
+    # Mixers leave the rows that their output projection reads in self.y.
     def _latent_attention(self, m: LatentAttention, rows, B, S, pos, eps):
         ops, cache = self.ops, m.kv_cache.rows
         H, dn, dr, dv, r, ld = m.heads, m.dim, m.rot_dim, m.vdim, m.rank, self.ld
-        q_off = self.d
+        q_off = self.off
         kv_off = q_off + m.q_rows
         smax, row_len = cache.shape[1], r + dr
         w_k, w_v = m.expand.weight[: H * dn], m.expand.weight[H * dn:]
@@ -120,15 +149,59 @@ class LayerEngine(Engine):
                              kv[H * dn:], (n * ld_kv, ld_kv, dv), self.y, pos, history, n, m.window, m.scale, B, S, H, dn, dr, dv)
 
     def _hgrn2(self, m, rows, B, S, pos, eps):
-        q_off = self.d
+        q_off = self.off
         f_off = q_off + m.heads * m.dim
         self.ops.hgrn2(self.proj, self.ld, q_off, f_off, f_off + m.heads * m.dim, m.f_bias, m.lower, m.norm, eps,
                        m.kv_cache.state, pos, self.y, B, S, m.heads, m.dim, m.vdim, self.ws_hgrn)
 
+    def _low_rank(self, off, w, out, rows):
+        """out (fp32) = w x, x the columns of the input projection from `off` on, in the storage type."""
+        self.ops.round_columns(self.proj, self.ld, off, w.shape[1], self.low, rows)
+        self.ops.linear_f32(self.low, w, out, rows, workspace=self.ws_low)
+
+    def _gla(self, m, rows, B, S, pos, eps):
+        ops, at, proj = self.ops, _offsets(m.parts(), self.off), self.proj.view(-1)
+        self._low_rank(at["a1"], m.a2, self.decay, rows)
+        ops.logistic_decay(self.decay, m.a2_bias, m.tau, rows)
+        ops.state_scan(proj[at["q"]:], self.ld, proj[at["k"]:], self.ld, proj[at["v"]:], self.ld, self.decay, None, None,
+                       m.kv_cache.state, pos, self.scan_o, m.dim ** -0.5, B, S, m.heads)
+        ops.head_norm_gate(self.scan_o, m.norm, eps, proj[at["g"]:], self.ld, "silu", 1.0, self.y, m.out_width, rows, m.heads)
+
+    def _grouped(self, m, at, y, y_ld, factor, rows, B, S, pos, eps):
+        ops, sums = self.ops, None
+        if self.comm.world > 1:  # the norms run over the heads of all ranks
+            sums = self.qk_sums
+            ops.row_squares(self.proj, self.ld, at["q"], m.heads * m.dim, at["k"], m.kv_heads * m.dim, sums, rows)
+            dist.all_reduce(sums[:rows])
+        kc, vc = m.kv_cache.k_cache, m.kv_cache.v_cache
+        ops.grouped_prepare(self.proj, self.ld, (at["q"], at["k"], at["v"]), m.q_norm, m.k_norm, sums, m.norm_widths, eps,
+                            m.rope_table, m.rot_dims, pos, self.q, kc, vc, B, S, m.heads)
+        ops.grouped_attention(self.q, kc, vc, m.sink, y, y_ld, factor, pos, m.window, m.chunk, m.scale, B, S, m.heads)
+
+    def _gated_delta(self, m, at, y, y_ld, factor, rows, B, S, pos, eps):
+        ops = self.ops
+        self._low_rank(at["a1"], m.a2, self.decay, rows)
+        self._low_rank(at["g1"], m.g2, self.scan_gate, rows)
+        ops.delta_prepare(self.proj, self.ld, (at["q"], at["k"], at["v"], at["b"]), (m.conv_q, m.conv_k, m.conv_v), m.conv_state.ring,
+                          self.decay, m.a_log, m.dt_bias, pos, self.scan_q, self.scan_k, self.scan_v, self.scan_beta, self.scan_kq,
+                          B, S, m.heads, m.kv_heads, m.dim, m.vdim)
+        qk, v = m.kv_heads * m.dim, m.out_width
+        ops.state_scan(self.scan_q, qk, self.scan_k, qk, self.scan_v, v, self.decay, self.scan_beta, self.scan_kq, m.kv_cache.state,
+                       pos, self.scan_o, m.dim ** -0.5, B, S, m.kv_heads)
+        ops.head_norm_gate(self.scan_o, m.norm, eps, self.scan_gate, v, "sigmoid", factor, y, y_ld, rows, m.heads)
+
+    def _parallel(self, m, rows, B, S, pos, eps):
+        at, ld = _offsets(m.parts(), self.off), m.out_width
+        y = self.y.view(-1)
+        for side, run, first in (("left", self._grouped, 0), ("right", self._gated_delta, m.left.out_width)):
+            sub = getattr(m, side)
+            offs = {k[len(side) + 1:]: v for k, v in at.items() if k.startswith(side + ".")}
+            run(sub, offs, y[first:], ld, m.scales[side == "right"], rows, B, S, pos, eps)
+
     def _experts(self, m, rows):
         """Returns (result rows, slots, number of result rows): the row of each (token, choice) pair in self.moe_out."""
         ops, pairs = self.ops, rows * m.top
-        logits = self.proj.view(-1)[self.d:]
+        logits = self.proj.view(-1)[self.off:]
         if not ops.moe_packs(self.dtype, rows, m.top, self.d, m.ff):
             ops.moe_route(logits, self.ld, m.experts, m.top, rows, self.moe_ids, self.moe_scores)
             ops.moe_gateup(self.normed, m.w1, self.moe_hidden, self.moe_ids, self.moe_scores, pairs, m.top, m.glu)
@@ -143,39 +216,53 @@ class LayerEngine(Engine):
         ops.moe_down(self.moe_hidden, m.w2, self.moe_out, None, pairs, tiles=self.moe_tiles, max_tiles=tiles)
         return self.moe_slots, 128 * tiles
 
-    def _join(self, branch, y, rows, next_norm, n_slots=1, slots=None, y_rows=None):
-        """x += post_norm(gate * sum of y's slots); normed = norm of x for the next sublayer (or the head)."""
-        if self.comm.world > 1:
-            # ranks hold partial sums of y: add the slots, then the ranks
-            if n_slots > 1 or slots is not None:
-                self.ops.sum_slots(y, rows, n_slots, slots, y_rows, self.part)
-                y, n_slots, slots, y_rows = self.part, 1, None, None
+    def _start(self, idx, first):
+        m, eps = self.model, self.cfg.norm_eps
+        if isinstance(first, StreamBranch):
+            self.ops.embed_streams(m.tok_embeddings.weight, idx, self.cfg.embed_scale, self.resid, first.w_in, first.pre_norm, eps,
+                                   self.normed)
+        else:
+            self.ops.embed_norm(m.tok_embeddings.weight, idx, self.resid, first.pre_norm, eps, self.normed)
+
+    def _join(self, branch, nxt, y, rows, n_slots=1, slots=None, y_rows=None):
+        """The sublayer's result (the sum of y's slots) enters the residual; normed = norm for the next sublayer or the head."""
+        ops, eps = self.ops, self.cfg.norm_eps
+        weight = nxt.pre_norm if nxt is not None else self.model.norm.weight
+        streams = isinstance(branch, StreamBranch)
+        if (self.comm.world > 1 or streams) and (n_slots > 1 or slots is not None):
+            ops.sum_slots(y, rows, n_slots, slots, y_rows, self.part)
+            y, n_slots, slots, y_rows = self.part, 1, None, None
+        if self.comm.world > 1:  # ranks hold partial sums of y
             self.comm.all_reduce(y, rows)
-        self.ops.gated_norm_add(self.resid, y, self.proj, self.ld, branch.gate_bias, branch.post_norm, self.cfg.norm_eps,
-                                next_norm, self.normed, rows, n_slots=n_slots, slots=slots, y_rows=y_rows)
+        if streams:
+            ops.join_streams(self.resid, y, branch.w_mix, branch.w_out, nxt.w_in if nxt is not None else None, weight, eps,
+                             self.normed, rows, write=nxt is not None)
+        else:
+            ops.gated_norm_add(self.resid, y, self.proj, self.ld, branch.gate_bias, branch.post_norm, eps, weight, self.normed, rows,
+                               n_slots=n_slots, slots=slots, y_rows=y_rows)
 
     def _in_proj(self, branch, rows):
-        self.ld = branch.in_proj.weight.shape[0]
-        self.ops.linear_f32(self.normed, branch.in_proj.weight, self.proj, rows, workspace=self.ws_in)
+        self.off = branch.gate_rows
+        if branch.in_proj is not None:
+            self.ld = branch.in_proj.weight.shape[0]
+            self.ops.linear_f32(self.normed, branch.in_proj.weight, self.proj, rows, workspace=self.ws_in)
 
     def _body(self, idx, rows, B, S, pos):
-        m, eps, ops = self.model, self.cfg.norm_eps, self.ops
-        norms = []  # the norm each sublayer's join prepares
-        for block in m.layers:
-            norms += [block.mixer.pre_norm] + ([block.mlp.pre_norm] if block.mlp is not None else [])
-        norms.append(m.norm.weight)
-        n = 0
-        ops.embed_norm(m.tok_embeddings.weight, idx, self.resid, norms[0], eps, self.normed)
-        for block in m.layers:
-            n += 1
-            mixer = block.mixer.sublayer
-            self._in_proj(block.mixer, rows)
-            (self._latent_attention if mixer.kind == "latent_attention" else self._hgrn2)(mixer, rows, B, S, pos, eps)
-            ops.linear(self.y, mixer.wo.weight, self.part, rows, workspace=self.ws_out)
-            self._join(block.mixer, self.part, rows, norms[n])
-            if block.mlp is not None:
-                n += 1
-                self._in_proj(block.mlp, rows)
-                moe = block.mlp.sublayer
-                slots, y_rows = self._experts(moe, rows)
-                self._join(block.mlp, self.moe_out, rows, norms[n], moe.top, slots, y_rows)
+        eps, ops = self.cfg.norm_eps, self.ops
+        run = {"latent_attention": self._latent_attention, "hgrn2": self._hgrn2, "gla": self._gla, "parallel": self._parallel}
+        self._start(idx, self.branches[0])
+        for i, branch in enumerate(self.branches):
+            nxt = self.branches[i + 1] if i + 1 < len(self.branches) else None
+            self._in_proj(branch, rows)
+            sub = branch.sublayer
+            if sub.kind == "moe":
+                slots, y_rows = self._experts(sub, rows)
+                self._join(branch, nxt, self.moe_out, rows, sub.top, slots, y_rows)
+            elif sub.kind == "glu":
+                ops.gateup_glu(self.normed, sub.w1, self.glu_hidden, rows, sub.glu, workspace=self.ws_glu)
+                ops.linear(self.glu_hidden, sub.w2, self.part, rows, workspace=self.ws_out)
+                self._join(branch, nxt, self.part, rows)
+            else:
+                run[sub.kind](sub, rows, B, S, pos, eps)
+                ops.linear(self.y, sub.wo.weight, self.part, rows, workspace=self.ws_out)
+                self._join(branch, nxt, self.part, rows)

@@ -1,4 +1,4 @@
-"""Checkpoints -> the fused, sharded parameter layout of this package: Hugging Face Llama / LlamaLadder, and Patevik.
+"""Checkpoints -> the fused, sharded parameter layout of this package: Hugging Face Llama / LlamaLadder, Patevik and Migosun.
 `load_model(path)` picks the model class from the folder's config.json.
 
 The reference has no loader (every rank draws its own random shard, benchmark.py:242-243); the only
@@ -22,7 +22,8 @@ unchanged by a permutation applied to both, and v / o_proj are untouched.
 import glob
 import json
 import os
-from typing import Dict, List, Optional
+import struct
+from typing import Dict, List, Optional, Tuple
 
 import torch
 import torch.distributed as dist
@@ -131,6 +132,73 @@ def patevik_to_local(w: Dict[str, Tensor], model, rank: int, world: int) -> Dict
     return out
 
 
+def _pad_to(w: Tensor, dim: int, n: int) -> Tensor:
+    """w with zeros behind it along `dim`, n in all."""
+    if w.shape[dim] == n:
+        return w
+    shape = list(w.shape)
+    shape[dim] = n - w.shape[dim]
+    return torch.cat([w, torch.zeros(shape, dtype=w.dtype)], dim)
+
+
+def migosun_to_local(w: Dict[str, Tensor], model, rank: int, world: int) -> Dict[str, Tensor]:
+    """Migosun checkpoint tensors -> state dict of rank `rank` of `world` for GPTMigosun's module tree:
+
+        in_proj   the mixer's input rows of the rank, low-rank parts padded with zero rows, zero rows at the end
+        a2, g2    rows of the rank's heads, columns padded like the rows they multiply
+        wo        columns of the rank's heads; side by side: [left o | right o]
+        w1        rows [up | gate] of the rank's slice of the feed-forward width
+    """
+    out = {"tok_embeddings.weight": w["embed"], "norm.weight": w["final.norm"]}
+    for i, block in enumerate(model.layers):
+        p = f"l{i}."
+
+        def rows(name):
+            return _rows(w[name], rank, world)
+
+        for branch, mine, norm, hc in ((block.mixer, "mixer", "norm1", "hc1"), (block.mlp, "mlp", "norm2", "hc2")):
+            if branch is not None:
+                dst = f"layers.{i}.{mine}."
+                out[dst + "pre_norm"] = w[p + norm]
+                for t in ("in", "mix", "out"):
+                    out[f"{dst}w_{t}"] = w[f"{p}{hc}.{t}"]
+        mixer, src, dst = block.mixer.sublayer, p + "mix.", f"layers.{i}.mixer."
+        parts = [_pad_to(rows(src + r.name) if r.split == "rows" else w[src + r.name], 0, r.padded) for r in mixer.parts()]
+        out[dst + "in_proj.weight"] = _pad_to(torch.cat(parts), 0, block.mixer.in_proj.weight.shape[0])
+        dst += "sublayer."
+        if mixer.kind == "parallel":
+            left, right = src + "left.", src + "right."
+            out[dst + "wo.weight"] = torch.cat([_cols(w[left + "o"], rank, world), _cols(w[right + "o"], rank, world)], 1)
+            out[dst + "left.q_norm"], out[dst + "left.k_norm"] = rows(left + "q.norm"), rows(left + "k.norm")
+            out[dst + "left.sink"] = rows(left + "sink")
+            for t in ("q", "k", "v"):
+                out[f"{dst}right.conv_{t}"] = rows(f"{right}{t}.conv")
+            out[dst + "right.a2"] = _pad_to(rows(right + "a2"), 1, mixer.right.a2.shape[1])
+            out[dst + "right.g2"] = _pad_to(rows(right + "g2"), 1, mixer.right.g2.shape[1])
+            out[dst + "right.a_log"], out[dst + "right.dt_bias"] = rows(right + "A_log"), rows(right + "dt_bias")
+            out[dst + "right.norm"] = w[right + "norm"]
+        else:
+            out[dst + "wo.weight"] = _cols(w[src + "o"], rank, world)
+            out[dst + "a2"] = _pad_to(rows(src + "a2"), 1, mixer.a2.shape[1])
+            out[dst + "a2_bias"] = rows(src + "a2.b")
+            out[dst + "norm"] = w[src + "norm"]
+        if block.mlp is not None:
+            src, dst = p + "mlp.", f"layers.{i}.mlp.sublayer."
+            out[dst + "w1"] = torch.cat([rows(src + "up"), rows(src + "gate")])
+            out[dst + "w2"] = _cols(w[src + "down"], rank, world)
+    return out
+
+
+def _safetensors_shapes(path: str) -> Dict[str, Tuple[int, ...]]:
+    """Shapes of the tensors in a folder's *.safetensors, from the files' headers."""
+    out: Dict[str, Tuple[int, ...]] = {}
+    for name in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with open(name, "rb") as f:
+            header = json.loads(f.read(struct.unpack("<Q", f.read(8))[0]))
+        out.update({k: tuple(v["shape"]) for k, v in header.items() if k != "__metadata__"})
+    return out
+
+
 def _read_safetensors(path: str) -> Dict[str, Tensor]:
     from safetensors.torch import load_file
     files = sorted(glob.glob(os.path.join(path, "*.safetensors"))) if os.path.isdir(path) else [path]
@@ -155,9 +223,18 @@ def _copy_parameters(model, local: Dict[str, Tensor]) -> None:
             p.copy_(src.to(device=p.device, dtype=p.dtype))
 
 
-def _patevik_class(config: dict):
+def _patevik_class(config: dict, path: str):
     from .gpt_patevik_TP import GPTPatevik, ModelArgs
     return GPTPatevik, ModelArgs.from_config(config)
+
+
+def _migosun_class(config: dict, path: str):
+    from .gpt_migosun_TP import GPTMigosun, ModelArgs
+    return GPTMigosun, ModelArgs.from_config(config, _safetensors_shapes(path))
+
+
+# designs with a checkpoint format of their own: state dict of a rank from the checkpoint's tensors
+_LAYOUTS = {"patevik": patevik_to_local, "migosun": migosun_to_local}
 
 
 def _llama_class(path_or_config):
@@ -177,10 +254,10 @@ def model_class(path: str):
     name = config.get("architecture")
     if name is None:
         return _llama_class(path)
-    known = {"Patevik": _patevik_class}
+    known = {"Patevik": _patevik_class, "Migosun": _migosun_class}
     if name not in known:
         raise ValueError(f"unknown architecture {name!r}; known: {sorted(known)}")
-    return known[name](config)
+    return known[name](config, path)
 
 
 def load_model(path: str, dtype=torch.bfloat16, device="cuda", max_batch_size: Optional[int] = None,
@@ -195,8 +272,8 @@ def load_model(path: str, dtype=torch.bfloat16, device="cuda", max_batch_size: O
     model = model.to(dtype=dtype).to_empty(device=device).eval()
     rank, world = dist.get_rank(), dist.get_world_size()
     tensors = _read_safetensors(path)
-    if cls.family == "patevik":
-        _copy_parameters(model, patevik_to_local(tensors, model, rank, world))
+    if cls.family in _LAYOUTS:
+        _copy_parameters(model, _LAYOUTS[cls.family](tensors, model, rank, world))
     else:
         load_hf_state_dict(model, tensors, rank, world)
     if max_batch_size is not None and max_seq_length is not None:

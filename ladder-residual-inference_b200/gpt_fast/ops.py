@@ -258,6 +258,112 @@ class CudaOps:
         _C.check(_C.lib.lri_moe_down(_C.dtype_code_any(hidden.dtype), hidden.data_ptr(), w2.data_ptr(), y.data_ptr(),
                                      _C.ptr(ids), pairs, _C.ptr(tiles), max_tiles, experts, dim, ff, _C.stream_handle()))
 
+    # ---- residual held as several streams ------------------------------------------------------------------
+    @staticmethod
+    def embed_streams(table, idx, scale, streams, in_next, weight, eps, normed):
+        """Every stream of `streams` [rows, n, dim] = scale * table row; normed = norm of their sum weighted by in_next."""
+        _C.require_cuda(table, idx, streams, in_next, weight, normed)
+        if idx.dtype not in (torch.int32, torch.int64):
+            idx = idx.to(torch.int64)
+        idx = idx.contiguous()
+        _C.check(_C.lib.lri_embed_streams(_C.dtype_code_any(table.dtype), table.data_ptr(), idx.data_ptr(),
+                                          int(idx.dtype == torch.int64), table.shape[0], float(scale), streams.data_ptr(),
+                                          _C.ptr(in_next), weight.data_ptr(), float(eps), normed.data_ptr(), idx.numel(),
+                                          streams.shape[1], table.shape[1], _C.stream_handle()))
+
+    @staticmethod
+    def join_streams(streams, y, mix, out, in_next, weight, eps, normed, rows, write=True):
+        """streams [.., n, dim] <- mix of the old ones + out * y (write=False: not stored); normed = norm of the sum weighted
+        by in_next (None: plain sum)."""
+        _C.require_cuda(streams, y, mix, out, in_next, weight, normed)
+        _C.check(_C.lib.lri_join_streams(_C.dtype_code_any(y.dtype), streams.data_ptr(), y.data_ptr(), mix.data_ptr(),
+                                         out.data_ptr(), streams.data_ptr() if write else None, _C.ptr(in_next), weight.data_ptr(),
+                                         float(eps), normed.data_ptr(), rows, streams.shape[1], streams.shape[2],
+                                         _C.stream_handle()))
+
+    # ---- gate/up with the clamped unit -----------------------------------------------------------------------
+    @staticmethod
+    def gateup_glu_workspace_bytes(dtype, rows, inter, k):
+        return _C.lib.lri_gateup_glu_workspace_bytes(_C.dtype_code_any(dtype), rows, inter, k)
+
+    @staticmethod
+    def gateup_glu(x, w1, h, rows, glu, workspace=None):
+        """w1 [2 ff, dim] = [up | gate]; glu = (alpha, limit, offset)."""
+        _C.require_cuda(x, w1, h)
+        two_i, k = w1.shape
+        ws_ptr, ws_bytes = (workspace.data_ptr(), workspace.numel() * workspace.element_size()) if workspace is not None else (None, 0)
+        _C.check(_C.lib.lri_gateup_glu(_C.dtype_code_any(x.dtype), x.data_ptr(), w1.data_ptr(), h.data_ptr(), rows, two_i // 2, k,
+                                       *[float(g) for g in glu], ws_ptr, ws_bytes, _C.stream_handle()))
+
+    # ---- grouped attention on a cache ------------------------------------------------------------------------
+    @staticmethod
+    def row_squares(x, ld, off1, n1, off2, n2, sums, rows):
+        _C.require_cuda(x, sums)
+        _C.check(_C.lib.lri_row_squares(x.data_ptr(), ld, off1, n1, off2, n2, sums.data_ptr(), rows, _C.stream_handle()))
+
+    @staticmethod
+    def grouped_prepare(proj, ld, offs, q_norm, k_norm, sums, widths, eps, table, rot_dims, input_pos, q, k_cache, v_cache, B, S,
+                        n_head):
+        """offs: columns of q, k, v in proj; widths: elements that the norms of q and k run over; sums: their sums of
+        squares where other ranks hold a part."""
+        _C.require_cuda(proj, q_norm, k_norm, sums, table, input_pos, q, k_cache, v_cache)
+        _, n_kv, smax, dim = k_cache.shape
+        _C.check(_C.lib.lri_grouped_prepare(
+            _C.dtype_code_any(k_cache.dtype), proj.data_ptr(), ld, *offs, q_norm.data_ptr(), k_norm.data_ptr(), _C.ptr(sums), *widths,
+            float(eps), table.data_ptr(), table.shape[0], rot_dims, input_pos.data_ptr(), int(input_pos.dtype == torch.int64),
+            q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), smax, B, S, n_head, n_kv, dim, v_cache.shape[3],
+            _C.stream_handle()))
+
+    @staticmethod
+    def grouped_attention(q, k_cache, v_cache, sink, out, out_ld, out_scale, input_pos, window, chunk, scale, B, S, n_head):
+        """window, chunk: 0 for none; sink: a logit per head or None; out starts at the first column to write."""
+        _C.require_cuda(q, k_cache, v_cache, sink, out, input_pos)
+        _, n_kv, smax, dim = k_cache.shape
+        _C.check(_C.lib.lri_grouped_attention(
+            _C.dtype_code_any(q.dtype), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _C.ptr(sink), out.data_ptr(), out_ld,
+            float(out_scale), input_pos.data_ptr(), int(input_pos.dtype == torch.int64), smax, window, chunk, float(scale), B, S,
+            n_head, n_kv, dim, v_cache.shape[3], _C.stream_handle()))
+
+    # ---- matrix-state recurrences ------------------------------------------------------------------------------
+    @staticmethod
+    def delta_prepare(proj, ld, offs, convs, ring, z, a_log, dt_bias, input_pos, q, k, v, beta, kq, B, S, heads, kv_heads, dim, vdim):
+        """offs: columns of q, k, v, b; convs: [channels, taps] of q, k, v; z becomes the decays."""
+        _C.require_cuda(proj, *convs, ring, z, a_log, dt_bias, input_pos, q, k, v, beta, kq)
+        _C.check(_C.lib.lri_delta_prepare(
+            _C.dtype_code_any(a_log.dtype), proj.data_ptr(), ld, *offs, *[c.data_ptr() for c in convs], convs[0].shape[1],
+            ring.data_ptr(), z.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), input_pos.data_ptr(),
+            int(input_pos.dtype == torch.int64), q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), kq.data_ptr(), B, S, heads,
+            kv_heads, dim, vdim, _C.stream_handle()))
+
+    @staticmethod
+    def logistic_decay(z, bias, tau, rows):
+        _C.require_cuda(z, bias)
+        _C.check(_C.lib.lri_logistic_decay(_C.dtype_code_any(bias.dtype), z.data_ptr(), bias.data_ptr(), float(tau), rows,
+                                           bias.numel(), _C.stream_handle()))
+
+    @staticmethod
+    def state_scan(q, q_row, k, k_row, v, v_row, decay, beta, kq, state, input_pos, o, o_scale, B, S, kv_heads):
+        """fp32 throughout; beta, kq: None for plain gated linear attention.  q, k, v start at their first column."""
+        _C.require_cuda(q, k, v, decay, beta, kq, state, input_pos, o)
+        _, heads, dim, vdim = state.shape
+        _C.check(_C.lib.lri_state_scan(q.data_ptr(), q_row, k.data_ptr(), k_row, v.data_ptr(), v_row, decay.data_ptr(), _C.ptr(beta),
+                                       _C.ptr(kq), state.data_ptr(), input_pos.data_ptr(), int(input_pos.dtype == torch.int64),
+                                       o.data_ptr(), float(o_scale), B, S, heads, kv_heads, dim, vdim, _C.stream_handle()))
+
+    @staticmethod
+    def head_norm_gate(o, norm_weight, eps, gate, gate_ld, activation, scale, out, out_ld, rows, heads):
+        """activation: "sigmoid" or "silu" of the gate; gate and out start at their first column."""
+        _C.require_cuda(o, norm_weight, gate, out)
+        act = {"sigmoid": _C.GATE_SIGMOID, "silu": _C.GATE_SILU}[activation]
+        _C.check(_C.lib.lri_head_norm_gate(_C.dtype_code_any(out.dtype), o.data_ptr(), norm_weight.data_ptr(), float(eps),
+                                           gate.data_ptr(), gate_ld, act, float(scale), out.data_ptr(), out_ld, rows, heads,
+                                           norm_weight.numel(), _C.stream_handle()))
+
+    @staticmethod
+    def round_columns(x, ld, off, n, y, rows):
+        _C.require_cuda(x, y)
+        _C.check(_C.lib.lri_round_columns(_C.dtype_code_any(y.dtype), x.data_ptr(), ld, off, n, y.data_ptr(), rows, _C.stream_handle()))
+
 
 def decode_splits(B, n_head, n_kv, smax, head_dim=128):
     """Number of sequence ranges for decode attention, fixed per cache geometry so that the launch

@@ -80,6 +80,31 @@ LAYER_LISTS = {
     "patevik-8b": _layer_list(32, 4096, 32, 128, 128, 512, 64, 4096, 8, 2, 7168, 128256),
 }
 
+
+
+def _stream_list(n_layer, width, streams, left, right, gla, ff, vocab, every=3):
+    """Layers with two mixers side by side, every `every`-th one gated linear attention; a dense unit behind each.
+    left (heads, kv_heads, dim, chunk), right (heads, kv_heads, dim, rank), gla (heads, dim, vdim, rank)."""
+    mlp = dict(kind="dense", ff=ff, limit=7.0)
+    lh, lk, ld, chunk = left
+    rh, rk, rd, rank = right
+    gh, gd, gv, grank = gla
+    side_by_side = dict(type="parallel", mlp=mlp, mixer=dict(
+        left_scale=1.0, right_scale=1.0,
+        left=dict(heads=lh, kv_heads=lk, dim=ld, vdim=ld, scale=ld ** -0.5, mask=dict(size=chunk), rot=dict(base=500000.0, dims=ld // 2)),
+        right=dict(heads=rh, kv_heads=rk, dim=rd, vdim=rd, conv=4, decay_rank=rank, gate_rank=rank)))
+    linear = dict(type="gla", mlp=mlp, mixer=dict(heads=gh, dim=gd, vdim=gv, tau=16.0, decay_rank=grank))
+    return dict(vocab_size=vocab, dim=width, streams=streams, embed_scale=1.0,
+                layers=[deepcopy(linear if i % every == every - 1 else side_by_side) for i in range(n_layer)])
+
+
+# Residual streams with dense feed-forwards: width, depth, vocabulary and feed-forward of the Llama shape of the same name.
+STREAM_LISTS = {
+    "migosun-tiny": _stream_list(4, 192, 3, (6, 2, 32, 48), (4, 2, 32, 16), (3, 32, 64, 8), 320, 512),
+    "migosun-1b": _stream_list(16, 2048, 4, (32, 8, 64, 2048), (16, 16, 64, 64), (16, 64, 128, 16), 8192, 128256),
+    "migosun-8b": _stream_list(32, 4096, 4, (32, 8, 128, 8192), (16, 16, 128, 128), (16, 128, 256, 16), 14336, 128256),
+}
+
 _COMMON = ["CodeLlama-7b-Python-hf", "1b", "3b", "7B", "13B", "30B", "34B", "70B", "Mistral-7B", "stories15M",
            "stories110M", "llama-3.2-1b", "llama-3.2-3b", "llama-3-8b", "llama-3-70b", "llama-3.1-405b",
            "ladder-llama-1b", "ladder-llama-405b-kv8"]
@@ -95,7 +120,9 @@ def _every_other_mlp(n_layer):
 
 
 def family_presets(family):
-    """Returns {preset name: ModelArgs kwargs} for 'ladder', 'dense', 'parallel', 'desync' or 'patevik'."""
+    """Returns {preset name: ModelArgs kwargs} for 'ladder', 'dense', 'parallel', 'desync', 'patevik' or 'migosun'."""
+    if family == "migosun":
+        return deepcopy(STREAM_LISTS)
     if family == "patevik":
         return deepcopy(LAYER_LISTS)
     out = {}
