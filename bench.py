@@ -1,7 +1,7 @@
 """Decode-throughput bench of the tensor-parallel Ladder-Llama step on B200.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--batch B] [--preset llama-3-8b]
-                    [--family ladder|...|patevik] [--impl ours|reference] [--mode decode|prefill|kernels]
+                    [--family ladder|...|patevik|migosun] [--impl ours|reference] [--mode decode|prefill|kernels]
     python -m torch.distributed.run --nnodes=1 --nproc-per-node N --master-addr 127.0.0.1 \
         --master-port P bench.py --gpus N ...
 
@@ -50,6 +50,7 @@ for _p in (ROOT, PKG):
         sys.path.insert(0, _p)
 
 METRIC = "decode_tokens_per_s"
+LAYER_FAMILIES = ("patevik", "migosun")
 UNIT = "tokens/s"
 FALLBACK_HBM_GBS = 6650.0
 
@@ -67,11 +68,11 @@ def parse_args(argv=None):
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--repeats", type=int, default=5, help="repeats of the K-step timed region (median reported)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--family", default="ladder", choices=["ladder", "dense", "parallel", "desync", "patevik"],
-                    help="patevik (presets patevik-8b, patevik-1b): decode and prompt throughput of the layer-list design "
-                         "beside the dense Llama model of equal width, depth and active parameters, one line for both; "
+    ap.add_argument("--family", default="ladder", choices=["ladder", "dense", "parallel", "desync", "patevik", "migosun"],
+                    help="patevik, migosun (presets <family>-8b, <family>-1b): decode and prompt throughput of a layer-list "
+                         "design beside the models of equal width, depth and active parameters, one line for all; "
                          "with --mode kernels a table of every op of a decode step and of a prompt pass against its roofline")
-    ap.add_argument("--preset", default=None, help="default: llama-3-8b (patevik-8b for --family patevik)")
+    ap.add_argument("--preset", default=None, help="default: llama-3-8b (patevik-8b, migosun-8b for those families)")
     ap.add_argument("--batch", type=int, default=1)
     ap.add_argument("--prompt", type=int, default=1024)
     ap.add_argument("--dtype", default="bf16", choices=["bf16", "fp16"])
@@ -105,7 +106,7 @@ def parse_args(argv=None):
     ap.add_argument("--eager", action="store_true", help="kernels mode: launch from Python instead of replaying a graph")
     args = ap.parse_args(argv)
     if args.preset is None:
-        args.preset = "patevik-8b" if args.family == "patevik" else "llama-3-8b"
+        args.preset = args.family + "-8b" if args.family in LAYER_FAMILIES else "llama-3-8b"
     return args
 
 
@@ -370,9 +371,11 @@ def workload_config(args, a, note=None):
 # ---------------------------------------------------------------------------------------------
 
 FAMILY_CLASS = {"ladder": "GPTLadder", "dense": "GPTDense", "parallel": "GPTParallel", "desync": "GPTDesync",
-                "patevik": "GPTPatevik"}
-# dense Llama shape of equal width, depth, vocabulary and active feed-forward parameters
-EQUAL_SIZE = {"patevik-8b": "llama-3-8b", "patevik-1b": "ladder-llama-1b"}
+                "patevik": "GPTPatevik", "migosun": "GPTMigosun"}
+# models of equal width, depth, vocabulary and active feed-forward parameters
+EQUAL_SIZE = {"patevik-8b": [("dense", "llama-3-8b")], "patevik-1b": [("dense", "ladder-llama-1b")],
+              "migosun-8b": [("dense", "llama-3-8b"), ("patevik", "patevik-8b")],
+              "migosun-1b": [("dense", "ladder-llama-1b"), ("patevik", "patevik-1b")]}
 
 
 class DecodeLoop:
@@ -658,21 +661,21 @@ def run_ours(args):
 
 
 def run_layer_family(args):
-    """Decode and prompt throughput of a layer-list model and of the dense Llama model of equal size, same batch, prompt
-    and kernels' conventions; or (--mode kernels) every op of both against its roofline."""
+    """Decode and prompt throughput of a layer-list model and of the models of equal size, same batch, prompt and
+    kernels' conventions; or (--mode kernels) every op of both against its roofline."""
     import torch
     import gpt_fast
     from gpt_fast import _C, op_bench
     assert args.gpus == 1, "the layer-list comparison runs on one GPU"
     if args.preset not in EQUAL_SIZE:
-        raise SystemExit(f"--family patevik takes --preset {' or '.join(EQUAL_SIZE)}")
+        raise SystemExit(f"--family {args.family} takes --preset {' or '.join(p for p in EQUAL_SIZE if p.startswith(args.family))}")
     dev = torch.device("cuda", torch.cuda.current_device())
     dtype = torch.bfloat16 if args.dtype == "bf16" else torch.float16
     B, T, K, W, R = args.batch, args.prompt, args.steps, args.warmup, max(1, args.repeats)
     hbm, _ = measured_hbm_peak()
     tensor, _ = measured_tensor_peak()
     g = torch.Generator().manual_seed(1234)
-    arms = [("patevik", args.preset)] + ([] if args.no_compare else [("dense", EQUAL_SIZE[args.preset])])
+    arms = [(args.family, args.preset)] + ([] if args.no_compare else EQUAL_SIZE[args.preset])
     out = {}
     sampler = ClockSampler(torch.cuda.current_device())
     for family, preset in arms:
@@ -739,14 +742,15 @@ def run_layer_family(args):
         torch.cuda.empty_cache()
     if args.mode == "kernels":
         return
-    line = {"metric": METRIC, "value": out["patevik"]["decode_tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": K, "warmup": W,
-            "ms_per_step": out["patevik"]["decode_ms_per_step"], "higher_is_better": True, "vs_baseline": None, "dtype": args.dtype,
+    line = {"metric": METRIC, "value": out[args.family]["decode_tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": K, "warmup": W,
+            "ms_per_step": out[args.family]["decode_ms_per_step"], "higher_is_better": True, "vs_baseline": None, "dtype": args.dtype,
             "data": "synthetic", "models": out,
-            "config": {"workload": f"patevik:{args.preset}, batch {B}, prompt {T} random ids (logits of the last position), greedy "
+            "config": {"workload": f"{args.family}:{args.preset}, batch {B}, prompt {T} random ids (logits of the last position), greedy "
                                    f"decode from there, random weights", "batch": B, "context": T,
                        "l2": "inputs larger than L2: every step streams GBs of weights, no flush"}}
-    if "dense" in out:
-        line["vs_dense"] = {k: out["patevik"][k] / out["dense"][k] for k in ("decode_tokens_per_s", "prompt_tokens_per_s")}
+    for other in out:
+        if other != args.family:
+            line["vs_" + other] = {k: out[args.family][k] / out[other][k] for k in ("decode_tokens_per_s", "prompt_tokens_per_s")}
     print(json.dumps(line), flush=True)
 
 
@@ -1145,7 +1149,7 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         run_reference_arm(args)
-    elif args.family == "patevik":
+    elif args.family in LAYER_FAMILIES:
         run_layer_family(args)
     elif args.mode == "comm":
         run_comm(args)

@@ -68,7 +68,8 @@ int lri_set_gemm_backend(int backend);
  * moe_stream_pairs (LRI_MOE_STREAM_PAIRS: (token, expert) pairs up to which experts run as streaming projections),
  * window_tc (LRI_WINDOW_TC: 0 keeps sliding-window attention on the plain kernel), hgrn2_blocks
  * (LRI_HGRN2_BLOCKS: 0 keeps the HGRN2 recurrence token by token), scan_columns (LRI_SCAN_COLUMNS: state columns per
- * lane of the matrix-state recurrences, 0 choose, 1, 2, 4).  Unknown
+ * lane of the matrix-state recurrences, 0 choose, 1, 2, 4), scan_warps (LRI_SCAN_WARPS: their warps per CTA, 0 choose, 1, 2, 4),
+ * scan_lanes (LRI_SCAN_LANES: lanes per state column, 0 choose, 8, 16).  Unknown
  * names and values an option does not take return LRI_ERR_ARG.  No counterpart in the reference
  * (its only switches are benchmark.py's command-line flags). */
 int lri_set_option(const char* name, int value);
@@ -414,27 +415,46 @@ int lri_grouped_attention(int dtype, const void* q, const void* k_cache, const v
                           int vdim, lri_stream_t stream);
 
 /* ---- matrix-state recurrences with a decay per key channel ----------------------------------------------------
- * lri_state_scan: per sequence and head, over the tokens of the call, S <- decay * S (rows); beta != NULL (delta rule):
- * u = beta (v - S^T k), else u = v; S <- S + k u^T; o = o_scale S^T q.  q, k [rows, kv_heads, dim] with row pitches (head h
- * reads h / (heads / kv_heads)), v [rows, heads, vdim] with row pitch, decay [rows, heads, dim], beta [rows, heads],
- * kq [rows, kv_heads] = k . q, o [rows, heads, vdim]; all fp32.  state [B, heads, dim, vdim] is read and written; a call that
- * starts at position 0 starts from zero. */
-int lri_state_scan(const float* q, int64_t q_row, const float* k, int64_t k_row, const float* v, int64_t v_row,
-                   const float* decay, const float* beta, const float* kq, float* state, const void* input_pos,
-                   int pos_is_i64, float* o, float o_scale, int B, int S, int heads, int kv_heads, int dim, int vdim,
+ * Per sequence and head, token by token: S <- g * S (g per row of S [dim, vdim]); u = v (gated linear attention) or
+ * u = beta (v - S^T k) (gated delta rule); S <- S + k u^T; o = S^T q.  All fp32.  Several tokens run in blocks of four:
+ * lri_delta_blocks / lri_gla_blocks prepare a call's block vectors, lri_state_scan runs it.
+ * lri_state_blocks: blocks of a sequence of S tokens; the arrays hold B times as many, blocks [.., heads, dim] for decay and
+ * [.., heads, 32] for coef, four rows [heads, dim] a block for qd, kd and ku. */
+int64_t lri_state_blocks(int64_t S);
+/* proj [B*S, ld] holds q, k (kv_heads of dim), v (heads of vdim) and b (heads).  q, k, v pass a causal convolution over time
+ * per channel (conv_* [channels, taps], last column = current token) and silu; q and k become unit vectors
+ * x / sqrt(sum x^2 + 1e-6), q also times dim^(-1/2); beta = sigmoid(b); g = exp(-exp(a_log) softplus(z + dt_bias)),
+ * z [B*S, heads, dim].  ring [B, taps, 2 kv_heads dim + heads vdim] keeps the last inputs of each channel (position p in slot
+ * p % taps); it is read for tokens before the call and updated.  v [B*S, heads, vdim] receives the values. */
+int lri_delta_blocks(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, int64_t b_off,
+                     const void* conv_q, const void* conv_k, const void* conv_v, int taps, float* ring, const float* z,
+                     const void* a_log, const void* dt_bias, const void* input_pos, int pos_is_i64, float* qd, float* kd,
+                     float* ku, float* decay, float* coef, float* v, int B, int S, int heads, int kv_heads, int dim,
+                     int vdim, lri_stream_t stream);
+/* q (times dim^(-1/2)) and k from proj, g = sigmoid(z + bias)^(1 / tau). */
+int lri_gla_blocks(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, const float* z, const void* bias,
+                   float tau, float* qd, float* ku, float* decay, float* coef, int B, int S, int heads, int dim,
                    lri_stream_t stream);
-/* Inputs of the gated delta rule.  proj [B*S, ld] holds q, k (kv_heads of dim), v (heads of vdim) and b (heads).  q, k, v
- * pass a causal convolution over time per channel (conv_* [channels, taps], last column = current token) and silu, q and k
- * become unit vectors x / sqrt(sum x^2 + 1e-6); beta = sigmoid(b); kq = k . q; z [rows, heads, dim] becomes
- * exp(-exp(a_log) softplus(z + dt_bias)).  ring [B, taps, 2 kv_heads dim + heads vdim] keeps the last inputs of each
- * channel (position p in slot p % taps); it is read for tokens before the call and updated. */
-int lri_delta_prepare(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, int64_t b_off,
-                      const void* conv_q, const void* conv_k, const void* conv_v, int taps, float* ring, float* z,
-                      const void* a_log, const void* dt_bias, const void* input_pos, int pos_is_i64, float* q, float* k,
-                      float* v, float* beta, float* kq, int B, int S, int heads, int kv_heads, int dim, int vdim,
-                      lri_stream_t stream);
-/* z [rows, width] <- sigmoid(z + bias)^(1 / tau). */
-int lri_logistic_decay(int dtype, float* z, const void* bias, float tau, int64_t rows, int width, lri_stream_t stream);
+/* The recurrence over a call's tokens; kd NULL: gated linear attention.  v [.., heads, vdim] with row pitch v_row; o [B*S,
+ * heads, vdim]; state [B, heads, dim, vdim] is read and written, a call that starts at position 0 starts from zero. */
+int lri_state_scan(const float* qd, const float* kd, const float* ku, const float* decay, const float* coef, const float* v,
+                   int64_t v_row, float* state, const void* input_pos, int pos_is_i64, float* o, int B, int S, int heads,
+                   int dim, int vdim, lri_stream_t stream);
+/* One token per sequence, everything between the input projections and the output projection's rows in one kernel; inputs
+ * as above, the low-rank second projections included: a2 [heads dim, a_rank] and g2 [heads vdim, g_rank] in `dtype` multiply
+ * the columns at a_off and g_off rounded to `dtype` (ranks multiples of 8, zero padded).  out (pitch out_ld) = factor *
+ * RMSNorm over vdim * norm_weight * gate; gate = sigmoid(g2 ..) or, gla, silu of the columns at g_off. */
+int lri_state_step_supports(int dim, int vdim, int decay_rank, int gate_rank);
+int lri_delta_step(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, int64_t a_off,
+                   int64_t g_off, int64_t b_off, const void* conv_q, const void* conv_k, const void* conv_v, int taps,
+                   float* ring, const void* a2, int a_rank, const void* g2, int g_rank, const void* a_log,
+                   const void* dt_bias, const void* norm_weight, float eps, float factor, float* state,
+                   const void* input_pos, int pos_is_i64, void* out, int64_t out_ld, int B, int heads, int kv_heads,
+                   int dim, int vdim, lri_stream_t stream);
+int lri_gla_step(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, int64_t a_off,
+                 int64_t g_off, const void* a2, int a_rank, const void* bias, float tau, const void* norm_weight, float eps,
+                 float factor, float* state, const void* input_pos, int pos_is_i64, void* out, int64_t out_ld, int B,
+                 int heads, int dim, int vdim, lri_stream_t stream);
 /* out[row, head] = scale * RMSNorm(o[row, head]) * norm_weight * act(gate[row, head]), gate fp32 with row pitch gate_ld. */
 enum lri_gate { LRI_GATE_SIGMOID = 0, LRI_GATE_SILU = 1 };
 int lri_head_norm_gate(int dtype, const float* o, const void* norm_weight, float eps, const float* gate, int64_t gate_ld,

@@ -67,6 +67,8 @@ enum Option {
   OPT_WINDOW_TC,        // LRI_WINDOW_TC      0: sliding-window attention always on the plain kernel
   OPT_HGRN2_BLOCKS,     // LRI_HGRN2_BLOCKS   0: the HGRN2 recurrence always runs token by token
   OPT_SCAN_COLUMNS,     // LRI_SCAN_COLUMNS   state columns per lane of the recurrence kernel: 1, 2, 4 (0 = choose)
+  OPT_SCAN_WARPS,       // LRI_SCAN_WARPS     warps per CTA of that kernel: 1, 2, 4 (0 = choose)
+  OPT_SCAN_LANES,       // LRI_SCAN_LANES     lanes per state column of that kernel: 8, 16 (0 = choose)
   OPT_COUNT
 };
 int option(int which);

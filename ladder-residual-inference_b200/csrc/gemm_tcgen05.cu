@@ -409,6 +409,21 @@ int make_tmap_heads(CUtensorMap* map, int dtype, const void* ptr, int64_t rows, 
   return LRI_OK;
 }
 
+int make_tmap_f32(CUtensorMap* map, const float* ptr, int64_t rows, int64_t row_pitch, int64_t heads, int64_t head_pitch, int64_t width,
+                  int box_width, int box_rows) {
+  EncodeTiledFn enc = encode_fn();
+  if (!enc) return fail(LRI_ERR_CUDA, "tensor map: cuTensorMapEncodeTiled is not available from the driver");
+  cuuint64_t dims[3] = {static_cast<cuuint64_t>(width), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(rows)};
+  cuuint64_t strides[2] = {static_cast<cuuint64_t>(head_pitch) * 4, static_cast<cuuint64_t>(row_pitch) * 4};
+  cuuint32_t box[3] = {static_cast<cuuint32_t>(box_width), 1, static_cast<cuuint32_t>(box_rows)};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT32, 3, const_cast<float*>(ptr), dims, strides, box, estr,
+                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return fail(LRI_ERR_CUDA, "tensor map: cuTensorMapEncodeTiled failed with CUresult %d", (int)r);
+  return LRI_OK;
+}
+
 int sm_count() { return device_sm_count(); }
 
 namespace {

@@ -36,11 +36,39 @@ constexpr int kThreads = 256;
 template <typename T, int VEC, typename Store>
 __device__ __forceinline__ void norm_rotate(const float* x, const T* w, float inv, const float* cs, int heads, int d, int rot, Store store) {
   const int half = rot >> 1, per = d / VEC;
-  for (int i = threadIdx.x; i < heads * per; i += kThreads) {
+  const bool whole = VEC == 8 && half % 8 == 0;  // 8 elements lie in one half, or behind the rotated part
+  for (int i = blockIdx.y * kThreads + threadIdx.x; i < heads * per; i += kThreads * gridDim.y) {
     const int h = i / per, e0 = (i - h * per) * VEC;
     const float* xh = x + h * d;
     const T* wh = w + h * d;
     float f[VEC];
+    if constexpr (VEC == 8) {
+      if (whole) {
+        float a[8], wa[8];
+        load8<float>(xh + e0, a);
+        load8<T>(wh + e0, wa);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = a[j] * inv * wa[j];
+        if (e0 < rot) {
+          const bool lower = e0 < half;
+          const int other = lower ? e0 + half : e0 - half;
+          const float* c = cs + 2 * (lower ? e0 : other);
+          float b[8], wb[8], t0[8], t1[8];
+          load8<float>(xh + other, b);
+          load8<T>(wh + other, wb);
+          load8<float>(c, t0);
+          load8<float>(c + 8, t1);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            const float co = j < 4 ? t0[2 * j] : t1[2 * j - 8], si = j < 4 ? t0[2 * j + 1] : t1[2 * j - 7];
+            const float y = b[j] * inv * wb[j];
+            f[j] = lower ? f[j] * co - y * si : f[j] * co + y * si;
+          }
+        }
+        store(h, e0, f);
+        continue;
+      }
+    }
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
       const int e = e0 + j;
@@ -65,7 +93,8 @@ __device__ __forceinline__ void put(T* dst, const float (&f)[VEC]) {
     dst[0] = Num<T>::from_f(f[0]);
 }
 
-// One CTA per row; q and k of the row are staged in shared memory, since a rotation needs both halves.
+// Grid (rows, slices): q and k of the row are staged in shared memory, since a norm needs all of them and a rotation both
+// halves; with few rows several CTAs stage the same row and store a share of it each.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kThreads) grouped_prepare_kernel(const PrepareParams p) {
   extern __shared__ __align__(16) float gp_smem[];
@@ -117,7 +146,7 @@ __global__ void __launch_bounds__(kThreads) grouped_prepare_kernel(const Prepare
                       [&](int h, int e, const float(&f)[VEC]) { put<T, VEC>(qo + h * p.d + e, f); });
   norm_rotate<T, VEC>(k, static_cast<const T*>(p.k_norm), 1.0f / sqrtf(sk / static_cast<float>(p.k_width) + p.eps), cs, p.G, p.d, p.rot,
                       [&](int h, int e, const float(&f)[VEC]) { put<T, VEC>(kc + h * p.smax * p.d + e, f); });
-  for (int i = threadIdx.x * VEC; i < nv; i += kThreads * VEC) {
+  for (int i = (blockIdx.y * kThreads + threadIdx.x) * VEC; i < nv; i += kThreads * VEC * gridDim.y) {
     const int h = i / p.dv, e = i - h * p.dv;
     float f[VEC];
     if constexpr (VEC == 8)
@@ -154,7 +183,9 @@ int prepare(const PrepareParams& p, int64_t rows, bool vec, cudaStream_t st) {
     LRI_ONCE_PER_DEVICE(set8, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxStaged * 4));
   else
     LRI_ONCE_PER_DEVICE(set1, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxStaged * 4));
-  LRI_CUDA(launch_pdl(kern, dim3(static_cast<unsigned>(rows)), dim3(kThreads), smem, st, p));
+  const int items = p.H * p.d / (vec ? 8 : 1);
+  const unsigned slices = rows > 64 ? 1 : (items + kThreads - 1) / kThreads;
+  LRI_CUDA(launch_pdl(kern, dim3(static_cast<unsigned>(rows), slices < 8 ? slices : 8), dim3(kThreads), smem, st, p));
   LRI_LAUNCH_CHECK("grouped_prepare_kernel");
   return LRI_OK;
 }
@@ -196,7 +227,8 @@ extern "C" int lri_grouped_prepare(int dtype, const float* proj, int64_t ld, int
   p.input_pos = input_pos, p.pos_is_i64 = pos_is_i64, p.q = q, p.k_cache = k_cache, p.v_cache = v_cache, p.smax = smax;
   p.S = S, p.H = n_head, p.G = n_kv, p.d = dim, p.dv = vdim, p.rot = rot_dims;
   const bool vec = dim % 8 == 0 && vdim % 8 == 0 && ld % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 &&
-                   aligned16(proj) && aligned16(q) && aligned16(k_cache) && aligned16(v_cache);
+                   aligned16(proj) && aligned16(q) && aligned16(k_cache) && aligned16(v_cache) && aligned16(q_norm) && aligned16(k_norm) &&
+                   aligned16(rope_table);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (dtype == LRI_BF16) return prepare<__nv_bfloat16>(p, rows, vec, st);
   if (dtype == LRI_FP16) return prepare<__half>(p, rows, vec, st);

@@ -17,6 +17,7 @@ int gemm_tcgen05_launch(int dtype, const void* a, const void* w, void* c, int64_
 int gemm_tcgen05_status_read_and_clear(int* status_out);
 int attn_prefill_tc_status_read_and_clear(int* status_out);
 int window_attention_tc_status_read_and_clear(int* status_out);
+int state_scan_status_read_and_clear(int* status_out);
 bool gemm_tcgen05_fused_supports(int epi, const LinearParams& p, int64_t m);
 int gemm_tcgen05_fused_launch(int dtype, int epi, const LinearParams& p, int64_t m, cudaStream_t st);
 
@@ -50,6 +51,8 @@ const OptionSpec kOptionSpecs[OPT_COUNT] = {
     {"window_tc", "LRI_WINDOW_TC", 1, 0, 1},
     {"hgrn2_blocks", "LRI_HGRN2_BLOCKS", 1, 0, 1},
     {"scan_columns", "LRI_SCAN_COLUMNS", 0, 0, 4},
+    {"scan_warps", "LRI_SCAN_WARPS", 0, 0, 4},
+    {"scan_lanes", "LRI_SCAN_LANES", 0, 0, 16},
 };
 
 bool option_value_ok(int which, int v) {
@@ -58,7 +61,8 @@ bool option_value_ok(int which, int v) {
   if (which == OPT_GEMV_R) return v == 0 || v == 2 || v == 4 || v == 8;
   if (which == OPT_GEMV_U) return v == 0 || v == 2;
   if (which == OPT_GEMV_MT) return v == 0 || v == 1 || v == 2 || v == 4;
-  if (which == OPT_ATTN_HEAD_TILE || which == OPT_SCAN_COLUMNS) return v == 0 || v == 1 || v == 2 || v == 4;
+  if (which == OPT_ATTN_HEAD_TILE || which == OPT_SCAN_COLUMNS || which == OPT_SCAN_WARPS) return v == 0 || v == 1 || v == 2 || v == 4;
+  if (which == OPT_SCAN_LANES) return v == 0 || v == 8 || v == 16;
   return true;
 }
 
@@ -340,6 +344,10 @@ extern "C" int lri_gemm_status(void) {
     rc = window_attention_tc_status_read_and_clear(&v3);
     if (rc != LRI_OK) return rc;
   }
+  int v4 = 0;
+  rc = state_scan_status_read_and_clear(&v4);
+  if (rc != LRI_OK) return rc;
+  if (v4 != 0) return fail(LRI_ERR_TIMEOUT, "matrix-state recurrence: a bounded mbarrier wait gave up (site %d)", v4);
   if (v3 != 0) return fail(LRI_ERR_TIMEOUT, "tcgen05 prefill attention: a bounded mbarrier wait gave up (site %d)", v3);
   return LRI_OK;
 }

@@ -1,0 +1,314 @@
+// One token of a matrix-state recurrence (linear_state.cuh) with everything around it in one kernel: from the fp32 input
+// projections to the rows that the output projection reads.
+//
+//   gated delta rule          convolutions with the ring, silu, unit vectors, both low-rank second projections, decay, step
+//                             size, state update, readout, RMSNorm over the value channels, sigmoid gate
+//   gated linear attention    low-rank decay, state update, readout, RMSNorm, silu gate
+//
+// A cluster serves one (sequence, head), each CTA 32 value channels.  A warp owns four of them, 8 lanes a column of the
+// state.  What all columns need (queries, keys, decays) every CTA computes for itself; only the sums of squares of the
+// results cross the cluster.  Weights are fetched, and the state is asked into the L2, before the preceding kernel is awaited.
+#include <cooperative_groups.h>
+
+#include "linear_state.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace lri {
+namespace {
+
+constexpr int kThreads = 256, kCols = 32, kMaxCluster = 8;
+constexpr int kStageBytes = 96 * 1024;  // second projections up to this size are staged in shared memory
+
+struct StepParams {
+  const float* proj;  // [B, ld]
+  int64_t ld, q_off, k_off, v_off, b_off, a_off, gate_off;  // a: input of the decay's projection; gate: of the gate's, or the gate
+  const void *conv_q, *conv_k, *conv_v;
+  int taps;
+  float* ring;
+  const void *a2, *g2;  // [H * C, a_rank], [H * E, g_rank]; ranks are multiples of 8
+  int a_rank, g_rank;
+  const void *a_log, *bias;  // bias: dt_bias, or the decay projection's
+  float inv_tau;
+  const void* norm_w;
+  float eps;
+  float* state;
+  const void* input_pos;
+  int pos_is_i64;
+  void* out;  // out + b * out_ld + h * E
+  int64_t out_ld;
+  float factor;
+  int H, G, C, E;
+  int staged;
+};
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src) : "memory");
+}
+
+// w[row] . x for the rows first, first + 32, ... below n: 8 lanes a row, 4 rows a warp; fn(row, sum) on one lane
+template <typename T, typename Fn>
+__device__ __forceinline__ void rows_dot(const T* w, int rank, const float* x, int n, Fn fn) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = (lane & 7) * 8;
+  for (int r0 = warp * 4; r0 < n; r0 += kThreads / 8) {
+    const int r = r0 + (lane >> 3);
+    float acc = 0.f;
+    if (r < n)
+      for (int i = part; i < rank; i += 64) {
+        float f[8];
+        load8<T>(w + static_cast<int64_t>(r) * rank + i, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc = fmaf(f[e], x[i + e], acc);
+      }
+#pragma unroll
+    for (int o = 1; o < 8; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+    if ((lane & 7) == 0 && r < n) fn(r, acc);
+  }
+}
+
+template <typename T, bool DELTA, int RV>
+__global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p) {
+  constexpr int CP = 32 * RV;
+  extern __shared__ __align__(16) uint8_t step_smem[];
+  __shared__ __align__(16) float sq[CP], sk[CP], sg[CP];
+  __shared__ float sv[kCols], sgate[kCols], part[8], cluster_part[kMaxCluster];
+  cg::cluster_group cluster = cg::this_cluster();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rg = lane & 7, cl = lane >> 3;
+  const int h = blockIdx.y, H = p.H, G = p.G, C = p.C, E = p.E, hk = h / (H / G);
+  const int64_t b = blockIdx.z;
+  const int col0 = blockIdx.x * kCols, my = warp * 4 + cl, e0 = col0 + my;
+  const int cols = E - col0 < kCols ? E - col0 : kCols;
+  float* x_a = reinterpret_cast<float*>(step_smem);  // input of the decay's second projection
+  float* x_g = x_a + p.a_rank;
+  T* w_smem = reinterpret_cast<T*>(x_g + (DELTA ? p.g_rank : 0));
+  const T* a2 = static_cast<const T*>(p.a2) + static_cast<int64_t>(h) * C * p.a_rank;
+  const T* g2 = DELTA ? static_cast<const T*>(p.g2) + (static_cast<int64_t>(h) * E + col0) * p.g_rank : nullptr;
+  float* st_base = p.state + (b * H + h) * static_cast<int64_t>(C) * E;
+  if (p.staged) {  // constants of the model
+    constexpr int kPer = 16 / sizeof(T);
+    const int na = C * p.a_rank / kPer, ng = DELTA ? cols * p.g_rank / kPer : 0;
+    for (int i = tid; i < na; i += kThreads) cp_async16(w_smem + i * kPer, a2 + i * kPer);
+    for (int i = tid; i < ng; i += kThreads) cp_async16(w_smem + (na + i) * kPer, g2 + i * kPer);
+    a2 = w_smem;
+    if (DELTA) g2 = w_smem + na * kPer;
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  for (int c = tid; c < C; c += kThreads) asm volatile("prefetch.global.L2 [%0];" ::"l"(st_base + static_cast<int64_t>(c) * E + col0));
+  pdl_launch_dependents();
+  pdl_wait();
+
+  // ---- state, and what the columns share -------------------------------------------------------------------
+  const int64_t pos = load_pos(p.input_pos, p.pos_is_i64, 0);
+  float st[RV][4];
+#pragma unroll
+  for (int i = 0; i < RV; ++i)
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+      const int c = 32 * i + 4 * rg + r;
+      st[i][r] = pos > 0 && c < C && e0 < E ? st_base[static_cast<int64_t>(c) * E + e0] : 0.f;
+    }
+  const float* in = p.proj + b * p.ld;
+  const int64_t channels = 2ll * G * C + static_cast<int64_t>(H) * E;
+  float* ring = DELTA ? p.ring + b * p.taps * channels : nullptr;
+  // convolution of one channel at this position; its input enters the ring (slots that are read here are other ones)
+  auto conv = [&](int64_t off, int64_t ch, const void* w, int64_t ch_w, bool keep) {
+    const T* tw = static_cast<const T*>(w) + ch_w * p.taps;
+    const float x = in[off];
+    float y = 0.f;
+    for (int j = p.taps - 1; j > 0; --j)
+      if (pos - j >= 0) y = fmaf(Num<T>::to_f(tw[p.taps - 1 - j]), ring[(pos - j) % p.taps * channels + ch], y);
+    y = fmaf(Num<T>::to_f(tw[p.taps - 1]), x, y);
+    if (keep && pos >= 0) ring[pos % p.taps * channels + ch] = x;
+    return silu_f(y);
+  };
+  const bool first = blockIdx.x == 0 && h % (H / G) == 0;  // keeps the shared channels of its group
+  for (int c = tid; c < CP; c += kThreads) {
+    float q = 0.f, k = 0.f;
+    if (c < C) {
+      const int64_t ch = static_cast<int64_t>(hk) * C + c;
+      if constexpr (DELTA) {
+        q = conv(p.q_off + ch, ch, p.conv_q, ch, first);
+        k = conv(p.k_off + ch, static_cast<int64_t>(G) * C + ch, p.conv_k, ch, first);
+      } else {
+        q = in[p.q_off + ch], k = in[p.k_off + ch];
+      }
+    }
+    sq[c] = q, sk[c] = k, sg[c] = 1.f;
+  }
+  if (tid >= kThreads - kCols) {
+    const int e = tid - (kThreads - kCols);
+    const int64_t ch = static_cast<int64_t>(h) * E + col0 + e;
+    float v = 0.f;
+    if (e < cols) v = DELTA ? conv(p.v_off + ch, 2ll * G * C + ch, p.conv_v, ch, true) : in[p.v_off + ch];
+    sv[e] = v;
+    if (!DELTA) sgate[e] = e < cols ? silu_f(in[p.gate_off + ch]) : 0.f;
+  }
+  for (int i = tid; i < p.a_rank; i += kThreads) x_a[i] = rnd<T>(in[p.a_off + i]);
+  if (DELTA)
+    for (int i = tid; i < p.g_rank; i += kThreads) x_g[i] = rnd<T>(in[p.gate_off + i]);
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+
+  const float a = DELTA ? expf(Num<T>::to_f(static_cast<const T*>(p.a_log)[h])) : 0.f;
+  rows_dot<T>(a2, p.a_rank, x_a, C, [&](int c, float z) {
+    z += Num<T>::to_f(static_cast<const T*>(p.bias)[h * C + c]);
+    sg[c] = DELTA ? delta_decay_f(z, a) : logistic_decay_f(z, p.inv_tau);
+  });
+  if constexpr (DELTA) rows_dot<T>(g2, p.g_rank, x_g, cols, [&](int e, float z) { sgate[e] = sigmoid_f(z); });
+  float qs = 1.0f / sqrtf(static_cast<float>(C)), ks = 1.f, kq = 0.f, beta = 0.f;
+  if constexpr (DELTA) {
+    float qq = 0.f, kk = 0.f;
+    for (int c = lane; c < C; c += 32) qq = fmaf(sq[c], sq[c], qq), kk = fmaf(sk[c], sk[c], kk), kq = fmaf(sq[c], sk[c], kq);
+    qs /= sqrtf(warp_sum(qq) + kUnitEps);
+    ks = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
+    kq = warp_sum(kq) * ks * qs;
+    beta = sigmoid_f(in[p.b_off + h]);
+  }
+  __syncthreads();
+
+  // ---- the recurrence ------------------------------------------------------------------------------------------
+  float dk = 0.f, dq = 0.f, u = sv[my];
+#pragma unroll
+  for (int i = 0; i < RV; ++i) {
+    const float4 g = *reinterpret_cast<const float4*>(&sg[32 * i + 4 * rg]);
+    const float4 q = *reinterpret_cast<const float4*>(&sq[32 * i + 4 * rg]), k = *reinterpret_cast<const float4*>(&sk[32 * i + 4 * rg]);
+    st[i][0] *= g.x, st[i][1] *= g.y, st[i][2] *= g.z, st[i][3] *= g.w;
+    if constexpr (!DELTA) {
+      st[i][0] = fmaf(k.x, u, st[i][0]), st[i][1] = fmaf(k.y, u, st[i][1]), st[i][2] = fmaf(k.z, u, st[i][2]), st[i][3] = fmaf(k.w, u, st[i][3]);
+    } else {
+      dk = fmaf(st[i][0], k.x, dk), dk = fmaf(st[i][1], k.y, dk), dk = fmaf(st[i][2], k.z, dk), dk = fmaf(st[i][3], k.w, dk);
+    }
+    dq = fmaf(st[i][0], q.x, dq), dq = fmaf(st[i][1], q.y, dq), dq = fmaf(st[i][2], q.z, dq), dq = fmaf(st[i][3], q.w, dq);
+  }
+#pragma unroll
+  for (int o = 1; o < 8; o <<= 1) {
+    if (DELTA) dk += __shfl_xor_sync(0xffffffffu, dk, o);
+    dq += __shfl_xor_sync(0xffffffffu, dq, o);
+  }
+  float o = dq * qs;
+  if constexpr (DELTA) {
+    u = beta * (u - dk * ks);
+    o = fmaf(u, kq, o);
+    const float uk = u * ks;
+#pragma unroll
+    for (int i = 0; i < RV; ++i) {
+      const float4 k = *reinterpret_cast<const float4*>(&sk[32 * i + 4 * rg]);
+      st[i][0] = fmaf(k.x, uk, st[i][0]), st[i][1] = fmaf(k.y, uk, st[i][1]), st[i][2] = fmaf(k.z, uk, st[i][2]), st[i][3] = fmaf(k.w, uk, st[i][3]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < RV; ++i)
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+      const int c = 32 * i + 4 * rg + r;
+      if (c < C && e0 < E) st_base[static_cast<int64_t>(c) * E + e0] = st[i][r];
+    }
+
+  // ---- norm over the head's value channels, gate -----------------------------------------------------------------
+  const float ss = warp_sum(rg == 0 && e0 < E ? o * o : 0.f);
+  if (lane == 0) part[warp] = ss;
+  __syncthreads();
+  const int ranks = static_cast<int>(cluster.num_blocks());
+  if (tid < ranks) {
+    float s = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) s += part[w];
+    *cluster.map_shared_rank(&cluster_part[cluster.block_rank()], tid) = s;
+  }
+  cluster.sync();
+  float total = 0.f;
+  for (int r = 0; r < ranks; ++r) total += cluster_part[r];
+  if (rg == 0 && e0 < E) {
+    const float inv = p.factor / sqrtf(total / static_cast<float>(E) + p.eps);
+    static_cast<T*>(p.out)[b * p.out_ld + static_cast<int64_t>(h) * E + e0] =
+        Num<T>::from_f(o * inv * Num<T>::to_f(static_cast<const T*>(p.norm_w)[e0]) * sgate[my]);
+  }
+}
+
+template <typename T, bool DELTA, int RV>
+int launch(const StepParams& p, int B, cudaStream_t st) {
+  const size_t x_bytes = (static_cast<size_t>(p.a_rank) + (DELTA ? p.g_rank : 0)) * 4;
+  const size_t w_bytes = (static_cast<size_t>(p.C) * p.a_rank + (DELTA ? static_cast<size_t>(kCols) * p.g_rank : 0)) * sizeof(T);
+  StepParams q = p;
+  q.staged = w_bytes <= kStageBytes;
+  auto kern = state_step_kernel<T, DELTA, RV>;
+  static std::atomic<unsigned long long> attr_set{0};
+  LRI_ONCE_PER_DEVICE(attr_set, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * kStageBytes));
+  const unsigned cs = (p.E + kCols - 1) / kCols;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(cs, p.H, B);
+  cfg.blockDim = dim3(kThreads);
+  cfg.dynamicSmemBytes = x_bytes + (q.staged ? w_bytes : 0);
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = cs;
+  attr[0].val.clusterDim.y = 1;
+  attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = pdl_enabled() ? 2 : 1;
+  LRI_CUDA(cudaLaunchKernelEx(&cfg, kern, q));
+  LRI_LAUNCH_CHECK("state_step_kernel");
+  return LRI_OK;
+}
+template <typename T, bool DELTA>
+int by_channels(const StepParams& p, int B, cudaStream_t st) {
+  if (p.C <= 32) return launch<T, DELTA, 1>(p, B, st);
+  if (p.C <= 64) return launch<T, DELTA, 2>(p, B, st);
+  if (p.C <= 128) return launch<T, DELTA, 4>(p, B, st);
+  return launch<T, DELTA, 8>(p, B, st);
+}
+template <bool DELTA>
+int run(const char* who, int dtype, const StepParams& p, int B, cudaStream_t st) {
+  LRI_REQUIRE(dtype >= LRI_BF16 && dtype <= LRI_FP32, LRI_ERR_UNSUPPORTED, "%s: dtype %d", who, dtype);
+  LRI_REQUIRE(p.proj && p.a2 && p.bias && p.norm_w && p.state && p.input_pos && p.out, LRI_ERR_ARG, "%s: NULL pointer", who);
+  LRI_REQUIRE(B >= 0 && B <= 65535 && p.H > 0 && p.H <= 65535 && p.G > 0 && p.H % p.G == 0, LRI_ERR_ARG, "%s: B=%d heads=%d kv_heads=%d", who,
+              B, p.H, p.G);
+  LRI_REQUIRE(lri_state_step_supports(p.C, p.E, p.a_rank, p.g_rank), LRI_ERR_UNSUPPORTED, "%s: dim=%d vdim=%d ranks %d, %d", who, p.C, p.E,
+              p.a_rank, p.g_rank);
+  LRI_REQUIRE(aligned16(p.a2) && aligned16(p.g2), LRI_ERR_ALIGN, "%s: second projections must be 16-byte aligned", who);
+  if (B == 0) return LRI_OK;
+  if (dtype == LRI_BF16) return by_channels<__nv_bfloat16, DELTA>(p, B, st);
+  if (dtype == LRI_FP16) return by_channels<__half, DELTA>(p, B, st);
+  return by_channels<float, DELTA>(p, B, st);
+}
+
+}  // namespace
+}  // namespace lri
+
+using namespace lri;
+
+extern "C" int lri_state_step_supports(int dim, int vdim, int decay_rank, int gate_rank) {
+  return dim >= 1 && dim <= 256 && vdim >= 1 && vdim <= kCols * kMaxCluster && decay_rank >= 8 && decay_rank % 8 == 0 && decay_rank <= 4096 &&
+         gate_rank >= 0 && gate_rank % 8 == 0 && gate_rank <= 4096;
+}
+
+extern "C" int lri_delta_step(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, int64_t a_off,
+                              int64_t g_off, int64_t b_off, const void* conv_q, const void* conv_k, const void* conv_v, int taps,
+                              float* ring, const void* a2, int a_rank, const void* g2, int g_rank, const void* a_log,
+                              const void* dt_bias, const void* norm_weight, float eps, float factor, float* state,
+                              const void* input_pos, int pos_is_i64, void* out, int64_t out_ld, int B, int heads, int kv_heads, int dim,
+                              int vdim, lri_stream_t stream) {
+  LRI_REQUIRE(conv_q && conv_k && conv_v && ring && g2 && a_log && taps >= 1 && taps <= kMaxTaps && g_rank >= 8, LRI_ERR_ARG,
+              "delta_step: NULL pointer, taps=%d or gate rank %d", taps, g_rank);
+  StepParams p{};
+  p.proj = proj, p.ld = ld, p.q_off = q_off, p.k_off = k_off, p.v_off = v_off, p.a_off = a_off, p.gate_off = g_off, p.b_off = b_off;
+  p.conv_q = conv_q, p.conv_k = conv_k, p.conv_v = conv_v, p.taps = taps, p.ring = ring, p.a2 = a2, p.g2 = g2, p.a_rank = a_rank, p.g_rank = g_rank;
+  p.a_log = a_log, p.bias = dt_bias, p.norm_w = norm_weight, p.eps = eps, p.factor = factor, p.state = state;
+  p.input_pos = input_pos, p.pos_is_i64 = pos_is_i64, p.out = out, p.out_ld = out_ld, p.H = heads, p.G = kv_heads, p.C = dim, p.E = vdim;
+  return run<true>("delta_step", dtype, p, B, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" int lri_gla_step(int dtype, const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, int64_t a_off,
+                            int64_t g_off, const void* a2, int a_rank, const void* bias, float tau, const void* norm_weight, float eps,
+                            float factor, float* state, const void* input_pos, int pos_is_i64, void* out, int64_t out_ld, int B, int heads,
+                            int dim, int vdim, lri_stream_t stream) {
+  LRI_REQUIRE(tau > 0.f, LRI_ERR_ARG, "gla_step: tau=%g", tau);
+  StepParams p{};
+  p.proj = proj, p.ld = ld, p.q_off = q_off, p.k_off = k_off, p.v_off = v_off, p.a_off = a_off, p.gate_off = g_off;
+  p.a2 = a2, p.a_rank = a_rank, p.bias = bias, p.inv_tau = 1.0f / tau, p.norm_w = norm_weight, p.eps = eps, p.factor = factor, p.state = state;
+  p.input_pos = input_pos, p.pos_is_i64 = pos_is_i64, p.out = out, p.out_ld = out_ld, p.H = heads, p.G = heads, p.C = dim, p.E = vdim;
+  return run<false>("gla_step", dtype, p, B, static_cast<cudaStream_t>(stream));
+}

@@ -169,6 +169,10 @@ int make_tmap(CUtensorMap* map, int dtype, const void* ptr, int64_t rows, int64_
 // box_rows rows, 128-byte swizzle; elements past `width` read as zero
 int make_tmap_heads(CUtensorMap* map, int dtype, const void* ptr, int64_t rows, int64_t row_pitch, int64_t heads,
                     int64_t head_pitch, int64_t width, int box_rows);
+// 3-D view [rows, heads, width] of fp32 elements, pitches in elements (multiples of 4), box = box_width elements of one head x
+// box_rows rows, not swizzled; elements past `width` read as zero
+int make_tmap_f32(CUtensorMap* map, const float* ptr, int64_t rows, int64_t row_pitch, int64_t heads, int64_t head_pitch, int64_t width,
+                  int box_width, int box_rows);
 int sm_count();
 
 }  // namespace lri

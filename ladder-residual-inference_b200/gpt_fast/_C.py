@@ -114,12 +114,21 @@ _SIGNATURES = {
     "lri_grouped_attention": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_float, c_void_p,
                                       c_int, c_int64, c_int64, c_int64, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
                                       c_void_p]),
-    "lri_state_scan": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
-                               c_void_p, c_int, c_void_p, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
-    "lri_delta_prepare": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_void_p,
-                                  c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                                  c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
-    "lri_logistic_decay": (c_int, [c_int, c_void_p, c_void_p, c_float, c_int64, c_int, c_void_p]),
+    "lri_state_blocks": (c_int64, [c_int64]),
+    "lri_delta_blocks": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_void_p,
+                                 c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_gla_blocks": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
+                               c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_state_scan": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int,
+                               c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_state_step_supports": (c_int, [c_int, c_int, c_int, c_int]),
+    "lri_delta_step": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_int64, c_int64, c_int64, c_int64, c_void_p, c_void_p,
+                               c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float,
+                               c_float, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "lri_gla_step": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int64, c_int64, c_int64, c_int64, c_void_p, c_int, c_void_p,
+                             c_float, c_void_p, c_float, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_int, c_int, c_int,
+                             c_int, c_void_p]),
     "lri_head_norm_gate": (c_int, [c_int, c_void_p, c_void_p, c_float, c_void_p, c_int64, c_int, c_float, c_void_p, c_int64,
                                    c_int64, c_int, c_int, c_void_p]),
     "lri_round_columns": (c_int, [c_int, c_void_p, c_int64, c_int64, c_int, c_void_p, c_int64, c_void_p]),

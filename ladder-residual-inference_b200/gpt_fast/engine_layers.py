@@ -82,16 +82,16 @@ class LayerEngine(Engine):
         if delta or gla:
             scans = delta + gla
             self.low = buf(rows, max(most(scans, lambda m: m.a2.shape[1]), most(delta, lambda m: m.g2.shape[1])))
-            self.decay = buf(rows, most(scans, lambda m: m.heads * m.dim), torch.float32)
-            self.scan_o = buf(rows, most(scans, lambda m: m.out_width), torch.float32)
+            hc = most(scans, lambda m: m.heads * m.dim)
+            self.scan_z, self.scan_o = buf(rows, hc, torch.float32), buf(rows, most(scans, lambda m: m.out_width), torch.float32)
+            # every sequence's tokens are cut in blocks from the call's first on
+            blocks = max(b * ops.state_blocks(max_seq) for b in (1, max_batch))
+            vectors = buf(4 * blocks, hc, torch.float32), buf(4 * blocks if delta else 0, hc, torch.float32), buf(4 * blocks, hc, torch.float32)
+            self.scan_blocks = vectors + (buf(blocks, hc, torch.float32), buf(blocks, 32 * most(scans, lambda m: m.heads), torch.float32))
             self.ws_low = workspace(ops.linear_f32_workspace_bytes, *[m.a2.shape[0] for m in scans], *[m.g2.shape[0] for m in delta])
         if delta:
-            qk = most(delta, lambda m: m.kv_heads * m.dim)
-            self.scan_q, self.scan_k = buf(rows, qk, torch.float32), buf(rows, qk, torch.float32)
             self.scan_v = buf(rows, most(delta, lambda m: m.out_width), torch.float32)
             self.scan_gate = buf(rows, most(delta, lambda m: m.out_width), torch.float32)
-            self.scan_beta, self.scan_kq = buf(rows, most(delta, lambda m: m.heads), torch.float32), \
-                buf(rows, most(delta, lambda m: m.kv_heads), torch.float32)
         if glus:
             self.glu_hidden = buf(rows, most(glus, lambda m: m.ff))
             self.ws_glu = workspace(lambda n, m: ops.gateup_glu_workspace_bytes(dtype, n, m.ff, self.d), *glus)
@@ -161,10 +161,13 @@ class LayerEngine(Engine):
 
     def _gla(self, m, rows, B, S, pos, eps):
         ops, at, proj = self.ops, _offsets(m.parts(), self.off), self.proj.view(-1)
-        self._low_rank(at["a1"], m.a2, self.decay, rows)
-        ops.logistic_decay(self.decay, m.a2_bias, m.tau, rows)
-        ops.state_scan(proj[at["q"]:], self.ld, proj[at["k"]:], self.ld, proj[at["v"]:], self.ld, self.decay, None, None,
-                       m.kv_cache.state, pos, self.scan_o, m.dim ** -0.5, B, S, m.heads)
+        if S == 1 and ops.state_step_supports(m.dim, m.vdim, m.a2.shape[1], 0):
+            ops.gla_step(self.proj, self.ld, [at[k] for k in ("q", "k", "v", "a1", "g")], m.a2, m.a2_bias, m.tau, m.norm, eps, 1.0,
+                         m.kv_cache.state, pos, self.y, m.out_width, B)
+            return
+        self._low_rank(at["a1"], m.a2, self.scan_z, rows)
+        ops.gla_blocks(self.proj, self.ld, (at["q"], at["k"]), self.scan_z, m.a2_bias, m.tau, self.scan_blocks, B, S, m.heads, m.dim)
+        ops.state_scan(self.scan_blocks, False, proj[at["v"]:], self.ld, m.kv_cache.state, pos, self.scan_o, B, S)
         ops.head_norm_gate(self.scan_o, m.norm, eps, proj[at["g"]:], self.ld, "silu", 1.0, self.y, m.out_width, rows, m.heads)
 
     def _grouped(self, m, at, y, y_ld, factor, rows, B, S, pos, eps):
@@ -179,15 +182,17 @@ class LayerEngine(Engine):
         ops.grouped_attention(self.q, kc, vc, m.sink, y, y_ld, factor, pos, m.window, m.chunk, m.scale, B, S, m.heads)
 
     def _gated_delta(self, m, at, y, y_ld, factor, rows, B, S, pos, eps):
-        ops = self.ops
-        self._low_rank(at["a1"], m.a2, self.decay, rows)
+        ops, convs, ring = self.ops, (m.conv_q, m.conv_k, m.conv_v), m.conv_state.ring
+        if S == 1 and ops.state_step_supports(m.dim, m.vdim, m.a2.shape[1], m.g2.shape[1]):
+            ops.delta_step(self.proj, self.ld, [at[k] for k in ("q", "k", "v", "a1", "g1", "b")], convs, ring, m.a2, m.g2, m.a_log,
+                           m.dt_bias, m.norm, eps, factor, m.kv_cache.state, pos, y, y_ld, B, m.kv_heads)
+            return
+        self._low_rank(at["a1"], m.a2, self.scan_z, rows)
         self._low_rank(at["g1"], m.g2, self.scan_gate, rows)
-        ops.delta_prepare(self.proj, self.ld, (at["q"], at["k"], at["v"], at["b"]), (m.conv_q, m.conv_k, m.conv_v), m.conv_state.ring,
-                          self.decay, m.a_log, m.dt_bias, pos, self.scan_q, self.scan_k, self.scan_v, self.scan_beta, self.scan_kq,
-                          B, S, m.heads, m.kv_heads, m.dim, m.vdim)
-        qk, v = m.kv_heads * m.dim, m.out_width
-        ops.state_scan(self.scan_q, qk, self.scan_k, qk, self.scan_v, v, self.decay, self.scan_beta, self.scan_kq, m.kv_cache.state,
-                       pos, self.scan_o, m.dim ** -0.5, B, S, m.kv_heads)
+        v = m.out_width
+        ops.delta_blocks(self.proj, self.ld, (at["q"], at["k"], at["v"], at["b"]), convs, ring, self.scan_z, m.a_log, m.dt_bias,
+                         pos, self.scan_blocks, self.scan_v, B, S, m.heads, m.kv_heads, m.dim, m.vdim)
+        ops.state_scan(self.scan_blocks, True, self.scan_v, v, m.kv_cache.state, pos, self.scan_o, B, S)
         ops.head_norm_gate(self.scan_o, m.norm, eps, self.scan_gate, v, "sigmoid", factor, y, y_ld, rows, m.heads)
 
     def _parallel(self, m, rows, B, S, pos, eps):

@@ -9,7 +9,7 @@ import torch
 
 # a call that is only valid right after another one is timed together with it
 _JOINED = {"moe_pack": "moe_route"}
-_HOST_ONLY = ("moe_packs", "moe_max_tiles")
+_HOST_ONLY = ("moe_packs", "moe_max_tiles", "state_step_supports", "state_blocks")
 
 
 class _Recorder:
@@ -43,9 +43,9 @@ def record(engine, step):
     return rec.calls
 
 
-def _visible(S, pos0, window):
+def _visible(S, pos0, window, chunk=0):
     """Visible (query, key) pairs of S queries from position pos0 on."""
-    return sum(min(pos0 + i + 1, window) for i in range(S))
+    return sum(min(pos0 + i + 1, window, (pos0 + i) % chunk + 1 if chunk else window) for i in range(S))
 
 
 def cost(name, a, kw, pos0, experts_used):
@@ -94,6 +94,44 @@ def cost(name, a, kw, pos0, experts_used):
     if name == "hgrn2":
         B, S, H, C, E = a[12:17]
         return B * (S * H * ((2 * C + E) * 4 + E * 2) + 8 * H * C * E), 4 * B * S * H * C * E
+    if name in ("embed_streams", "join_streams"):
+        n, d = (a[1].numel(), a[0].shape[1]) if name == "embed_streams" else (a[8], a[0].shape[2])
+        streams = (a[3] if name == "embed_streams" else a[0]).shape[1]
+        moved = streams * 4 + 4 if name == "embed_streams" else streams * (8 if kw.get("write", True) else 4) + 4
+        return n * d * moved, 0
+    if name == "gateup_glu":
+        (n, k), m = a[1].shape, a[3]
+        return n * k * 2 + m * (k + n // 2) * 2, 2 * m * n * k
+    if name == "grouped_prepare":
+        B, S, H = a[14:17]
+        (_, G, _, d), dv = a[12].shape, a[13].shape[3]
+        return B * S * ((H + G) * d + G * dv) * 6, 0
+    if name == "grouped_attention":
+        window, chunk, (B, S, H) = a[8], a[9], a[11:14]
+        (_, G, _, d), dv = a[1].shape, a[2].shape[3]
+        first = max(0, pos0 - window + 1 if window else 0, pos0 // chunk * chunk if chunk else 0)
+        pairs = _visible(S, pos0, window or 1 << 60, chunk)
+        return 2 * B * (S * H * (d + dv) + (pos0 + S - first) * G * (d + dv)), 2 * B * H * (d + dv) * pairs
+    if name == "delta_blocks":
+        B, S, H, G, C, E = a[11:17]
+        return 4 * B * S * ((2 * G * C + H * E) + H * C + 3 * H * C + H * C // 4 + H * E + 8 * H), 0
+    if name == "gla_blocks":
+        B, S, H, C = a[7:11]
+        return 4 * B * S * (3 * H * C + 2 * H * C + H * C // 4 + 8 * H), 0
+    if name == "state_scan":
+        # the recurrence's own inputs (q, k, decay, v) and results, however the blocks carry them
+        B, S = a[7:9]
+        _, H, C, E = a[4].shape
+        return 4 * B * (S * (3 * H * C + 2 * H * E) + 2 * H * C * E), (8 if a[1] else 6) * B * S * H * C * E
+    if name in ("delta_step", "gla_step"):
+        st, B, a2 = (a[12], a[16], a[5]) if name == "delta_step" else (a[9], a[13], a[3])
+        _, H, C, E = st.shape
+        low = a2.numel() + (a[6].numel() if name == "delta_step" else 0)
+        return B * (8 * H * C * E + 4 * H * (2 * C + 2 * E)) + 2 * low, (8 if name == "delta_step" else 6) * B * H * C * E
+    if name == "head_norm_gate":
+        return a[9] * a[10] * a[1].numel() * 10, 0
+    if name == "round_columns":
+        return a[5] * a[3] * 6, 0
     if name == "moe_route":
         return a[4] * a[2] * 4, 0
     if name == "moe_pack":
@@ -109,9 +147,14 @@ def cost(name, a, kw, pos0, experts_used):
 
 
 def _key(call):
+    def shape(x):
+        if isinstance(x, (tuple, list)):
+            return tuple(shape(y) for y in x)
+        return tuple(x.shape) if torch.is_tensor(x) else x
+
     out = []
     for name, _, a, kw in call:
-        out.append((name, tuple(tuple(x.shape) if torch.is_tensor(x) else x for x in a if not isinstance(x, float)),
+        out.append((name, tuple(shape(x) for x in a if not isinstance(x, float)),
                     tuple(sorted(k for k in kw))))
     return tuple(out)
 

@@ -325,30 +325,66 @@ class CudaOps:
             n_head, n_kv, dim, v_cache.shape[3], _C.stream_handle()))
 
     # ---- matrix-state recurrences ------------------------------------------------------------------------------
+    # blocks = (qd, kd, ku, decay, coef): vectors and coefficients of blocks of four tokens, fp32 (kd unused without the
+    # delta rule)
     @staticmethod
-    def delta_prepare(proj, ld, offs, convs, ring, z, a_log, dt_bias, input_pos, q, k, v, beta, kq, B, S, heads, kv_heads, dim, vdim):
-        """offs: columns of q, k, v, b; convs: [channels, taps] of q, k, v; z becomes the decays."""
-        _C.require_cuda(proj, *convs, ring, z, a_log, dt_bias, input_pos, q, k, v, beta, kq)
-        _C.check(_C.lib.lri_delta_prepare(
+    def state_blocks(S):
+        return _C.lib.lri_state_blocks(S)
+
+    @staticmethod
+    def delta_blocks(proj, ld, offs, convs, ring, z, a_log, dt_bias, input_pos, blocks, v, B, S, heads, kv_heads, dim, vdim):
+        """offs: columns of q, k, v, b; convs: [channels, taps] of q, k, v; z: the decays' projection."""
+        _C.require_cuda(proj, *convs, ring, z, a_log, dt_bias, input_pos, *blocks, v)
+        _C.check(_C.lib.lri_delta_blocks(
             _C.dtype_code_any(a_log.dtype), proj.data_ptr(), ld, *offs, *[c.data_ptr() for c in convs], convs[0].shape[1],
             ring.data_ptr(), z.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), input_pos.data_ptr(),
-            int(input_pos.dtype == torch.int64), q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), kq.data_ptr(), B, S, heads,
-            kv_heads, dim, vdim, _C.stream_handle()))
+            int(input_pos.dtype == torch.int64), *[x.data_ptr() for x in blocks], v.data_ptr(), B, S, heads, kv_heads, dim, vdim,
+            _C.stream_handle()))
 
     @staticmethod
-    def logistic_decay(z, bias, tau, rows):
-        _C.require_cuda(z, bias)
-        _C.check(_C.lib.lri_logistic_decay(_C.dtype_code_any(bias.dtype), z.data_ptr(), bias.data_ptr(), float(tau), rows,
-                                           bias.numel(), _C.stream_handle()))
+    def gla_blocks(proj, ld, offs, z, bias, tau, blocks, B, S, heads, dim):
+        """offs: columns of q, k."""
+        qd, _, ku, decay, coef = blocks
+        _C.require_cuda(proj, z, bias, qd, ku, decay, coef)
+        _C.check(_C.lib.lri_gla_blocks(_C.dtype_code_any(bias.dtype), proj.data_ptr(), ld, *offs, z.data_ptr(), bias.data_ptr(),
+                                       float(tau), qd.data_ptr(), ku.data_ptr(), decay.data_ptr(), coef.data_ptr(), B, S, heads, dim,
+                                       _C.stream_handle()))
 
     @staticmethod
-    def state_scan(q, q_row, k, k_row, v, v_row, decay, beta, kq, state, input_pos, o, o_scale, B, S, kv_heads):
-        """fp32 throughout; beta, kq: None for plain gated linear attention.  q, k, v start at their first column."""
-        _C.require_cuda(q, k, v, decay, beta, kq, state, input_pos, o)
+    def state_scan(blocks, delta, v, v_row, state, input_pos, o, B, S):
+        """v starts at its first column."""
+        _C.require_cuda(*[x for x in blocks if x is not None], v, state, input_pos, o)
+        qd, kd, ku, decay, coef = blocks
         _, heads, dim, vdim = state.shape
-        _C.check(_C.lib.lri_state_scan(q.data_ptr(), q_row, k.data_ptr(), k_row, v.data_ptr(), v_row, decay.data_ptr(), _C.ptr(beta),
-                                       _C.ptr(kq), state.data_ptr(), input_pos.data_ptr(), int(input_pos.dtype == torch.int64),
-                                       o.data_ptr(), float(o_scale), B, S, heads, kv_heads, dim, vdim, _C.stream_handle()))
+        _C.check(_C.lib.lri_state_scan(qd.data_ptr(), kd.data_ptr() if delta else None, ku.data_ptr(), decay.data_ptr(),
+                                       coef.data_ptr(), v.data_ptr(), v_row, state.data_ptr(), input_pos.data_ptr(),
+                                       int(input_pos.dtype == torch.int64), o.data_ptr(), B, S, heads, dim, vdim,
+                                       _C.stream_handle()))
+
+    @staticmethod
+    def state_step_supports(dim, vdim, decay_rank, gate_rank):
+        return bool(_C.lib.lri_state_step_supports(dim, vdim, decay_rank, gate_rank))
+
+    @staticmethod
+    def delta_step(proj, ld, offs, convs, ring, a2, g2, a_log, dt_bias, norm, eps, factor, state, input_pos, out, out_ld, B, kv_heads):
+        """offs: columns of q, k, v, a1, g1, b; out starts at the first column to write."""
+        _C.require_cuda(proj, *convs, ring, a2, g2, a_log, dt_bias, norm, state, input_pos, out)
+        _, heads, dim, vdim = state.shape
+        _C.check(_C.lib.lri_delta_step(
+            _C.dtype_code_any(out.dtype), proj.data_ptr(), ld, *offs, *[c.data_ptr() for c in convs], convs[0].shape[1], ring.data_ptr(),
+            a2.data_ptr(), a2.shape[1], g2.data_ptr(), g2.shape[1], a_log.data_ptr(), dt_bias.data_ptr(), norm.data_ptr(), float(eps),
+            float(factor), state.data_ptr(), input_pos.data_ptr(), int(input_pos.dtype == torch.int64), out.data_ptr(), out_ld, B,
+            heads, kv_heads, dim, vdim, _C.stream_handle()))
+
+    @staticmethod
+    def gla_step(proj, ld, offs, a2, bias, tau, norm, eps, factor, state, input_pos, out, out_ld, B):
+        """offs: columns of q, k, v, a1, g."""
+        _C.require_cuda(proj, a2, bias, norm, state, input_pos, out)
+        _, heads, dim, vdim = state.shape
+        _C.check(_C.lib.lri_gla_step(
+            _C.dtype_code_any(out.dtype), proj.data_ptr(), ld, *offs, a2.data_ptr(), a2.shape[1], bias.data_ptr(), float(tau),
+            norm.data_ptr(), float(eps), float(factor), state.data_ptr(), input_pos.data_ptr(), int(input_pos.dtype == torch.int64),
+            out.data_ptr(), out_ld, B, heads, dim, vdim, _C.stream_handle()))
 
     @staticmethod
     def head_norm_gate(o, norm_weight, eps, gate, gate_ld, activation, scale, out, out_ld, rows, heads):
