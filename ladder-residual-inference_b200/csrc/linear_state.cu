@@ -141,11 +141,13 @@ __global__ void __launch_bounds__(128, 1) state_scan_kernel(const __grid_constan
     f2 a0 = mul2(s[0], x[0]), a1 = mul2(s[1], x[1]);
 #pragma unroll
     for (int i = 2; i < 2 * RV; i += 2) a0 = fma2(s[i], x[i], a0), a1 = fma2(s[i + 1], x[i + 1], a1);
-    return sum_f2(a0) + sum_f2(a1);
+    return sum_f2(add2(a0, a1));
   };
+  // results: lane rg keeps token rg / kPerToken of the block number rg % kPerToken of a pair
+  constexpr int kPerToken = LN / kT;
+  const int my_t = rg / kPerToken, my_block = rg % kPerToken;
   float keep[NC];
-  // one block of four tokens; its results are kept by the lanes rg = lane0 .. lane0 + 3
-  auto block = [&](const float* cur, int sub, int lane0) {
+  auto block = [&](const float* cur, int sub, int nth) {
     const float* cf = cur + L::kCf + sub * kCoef;
     float d[kT][NC], dq[kT][NC], u[kT][NC];
 #pragma unroll
@@ -198,21 +200,19 @@ __global__ void __launch_bounds__(128, 1) state_scan_kernel(const __grid_constan
         for (int i = 0; i < 2 * RV; ++i) st[j][i] = fma2(x[i], u2, st[j][i]);
       }
     }
+    // sums of dq: each of the first two exchanges halves the tokens a lane holds
+    const float4 bt = *reinterpret_cast<const float4*>(cf + kCoefB + kT * my_t);
 #pragma unroll
-    for (int o = 1; o < LN; o <<= 1)
+    for (int j = 0; j < NC; ++j) {
+      const bool up = rg & (LN / 2), up2 = rg & (LN / 4);
+      const float x0 = (up ? dq[2][j] : dq[0][j]) + __shfl_xor_sync(0xffffffffu, up ? dq[0][j] : dq[2][j], LN / 2);
+      const float x1 = (up ? dq[3][j] : dq[1][j]) + __shfl_xor_sync(0xffffffffu, up ? dq[1][j] : dq[3][j], LN / 2);
+      float x = (up2 ? x1 : x0) + __shfl_xor_sync(0xffffffffu, up2 ? x0 : x1, LN / 4);
 #pragma unroll
-      for (int t = 0; t < kT; ++t)
-#pragma unroll
-        for (int j = 0; j < NC; ++j) dq[t][j] += __shfl_xor_sync(0xffffffffu, dq[t][j], o);
-#pragma unroll
-    for (int t = 0; t < kT; ++t)
-#pragma unroll
-      for (int j = 0; j < NC; ++j) {
-        float x = dq[t][j];
-#pragma unroll
-        for (int s = 0; s <= t; ++s) x = fmaf(cf[kCoefB + t * (t + 1) / 2 + s], u[s][j], x);
-        keep[j] = rg == lane0 + t ? x : keep[j];
-      }
+      for (int o = LN / 8; o >= 1; o >>= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+      x = fmaf(bt.x, u[0][j], x), x = fmaf(bt.y, u[1][j], x), x = fmaf(bt.z, u[2][j], x), x = fmaf(bt.w, u[3][j], x);
+      keep[j] = my_block == nth ? x : keep[j];
+    }
   };
 
   bool ok = true;
@@ -232,13 +232,13 @@ __global__ void __launch_bounds__(128, 1) state_scan_kernel(const __grid_constan
       for (int j = 0; j < NC; ++j) keep[j] = 0.f;
       if (n > kT) {  // straight on: the second block's sums start while the first one's results are reduced
         block(cur, t0 / kT, 0);
-        block(cur, t0 / kT + 1, kT);
+        block(cur, t0 / kT + 1, 1);
       } else {
         block(cur, t0 / kT, 0);
       }
-      // lane rg holds the results of token t0 + rg
-      if (rg < n) {
-        float* dst = p.o + ((b * p.S + i * kBlock + t0 + rg) * H + h) * E + e0;
+      const int mine = my_block * kT + my_t;  // token whose results this lane holds
+      if (my_block < 2 && mine < n) {
+        float* dst = p.o + ((b * p.S + i * kBlock + t0 + mine) * H + h) * E + e0;
 #pragma unroll
         for (int j = 0; j < NC; ++j)
           if (e0 + j < E) dst[j] = keep[j];

@@ -20,7 +20,7 @@
 namespace lri {
 
 constexpr int kStateBlock = 4;  // tokens of a block
-// coefficients of a block and head: beta_t, then A[t, s] (s < t), then B[t, s] (s <= t)
+// coefficients of a block and head: beta_t, then A[t, s] (s < t), then B[t, s] as rows of four (zero for s > t)
 constexpr int kCoef = 32, kCoefA = 4, kCoefB = 12;
 
 // ---- packed fp32 pairs ---------------------------------------------------------------------------------
@@ -41,6 +41,11 @@ __device__ __forceinline__ f2 pack_f2(float lo, float hi) {
   return d;
 }
 __device__ __forceinline__ void unpack_f2(f2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ f2 add2(f2 a, f2 b) {
+  f2 d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
 __device__ __forceinline__ float sum_f2(f2 v) {
   float a, b;
   unpack_f2(v, a, b);

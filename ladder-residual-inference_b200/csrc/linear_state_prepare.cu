@@ -63,8 +63,10 @@ __device__ __forceinline__ void block_channel(const float (&q)[kT], const float 
 // the lanes' shares of A (6) and B (10) -> coefficients of the block
 __device__ __forceinline__ void store_coef(float (&coef)[16], float* dst, int lane) {
   const float x = reduce_scatter<16>(coef, lane);
-  const int e = lane >> 1;
-  if ((lane & 1) == 0) dst[e < 6 ? kCoefA + e : kCoefB + e - 6] = x;
+  // element 6 + t (t + 1) / 2 + s of B goes to row t, column s
+  const int e = lane >> 1, i = e - 6, t = i < 1 ? 0 : (i < 3 ? 1 : (i < 6 ? 2 : 3));
+  if ((lane & 1) == 0) dst[e < 6 ? kCoefA + e : kCoefB + kT * t + i - t * (t + 1) / 2] = x;
+  if (lane < kT * kT && lane % kT > lane / kT) dst[kCoefB + lane] = 0.f;
 }
 
 struct DeltaBlocksParams {
@@ -85,6 +87,12 @@ struct DeltaBlocksParams {
   int S, H, G, C, E;
 };
 
+// Activation of a convolution: 16-bit models take it from the special-function unit (a few units in the last place of fp32).
+template <typename T>
+__device__ __forceinline__ float conv_silu(float x) {
+  return sizeof(T) == 4 ? silu_f(x) : x * __fdividef(1.0f, 1.0f + __expf(-x));
+}
+
 // silu of the convolution of one channel at the block's tokens (zero past the n of them).  `in` is the input of the block's
 // first token, s its place in the call, pos its position; inputs before the call come from the ring, those before the
 // sequence are zero.
@@ -95,9 +103,19 @@ __device__ __forceinline__ void conv_block(const float* in, int64_t ld, const T*
 #pragma unroll
   for (int t = 0; t < kT; ++t) x[TAPS - 1 + t] = t < n ? in[t * ld] : 0.f;
   float c[TAPS];  // leading taps that do not exist have weight zero
+  const bool whole = TAPS == 4 && sizeof(T) == 2 && taps == 4 && (reinterpret_cast<uintptr_t>(w) & 7u) == 0;
+  if (whole) {
+    if constexpr (TAPS == 4 && sizeof(T) == 2) {
+      const uint2 v = *reinterpret_cast<const uint2*>(w);
+      Num<T>::unpack2(v.x, c[0], c[1]);
+      Num<T>::unpack2(v.y, c[2], c[3]);
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) c[TAPS - 1 - j] = j < taps ? Num<T>::to_f(w[taps - 1 - j]) : 0.f;
+  }
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) {  // j tokens back
-    c[TAPS - 1 - j] = j < taps ? Num<T>::to_f(w[taps - 1 - j]) : 0.f;
     if (j > 0) {
       float v = 0.f;
       if (j < taps) {
@@ -114,18 +132,20 @@ __device__ __forceinline__ void conv_block(const float* in, int64_t ld, const T*
     float a = 0.f;
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) a = fmaf(c[j], x[t + j], a);
-    y[t] = t < n ? silu_f(a) : 0.f;
+    y[t] = t < n ? conv_silu<T>(a) : 0.f;
   }
 }
 
-// One warp per (block, value head); a lane owns the channels lane, lane + 32, ...  CI > 0: at most 32 CI channels, whose q and
+// One warp per (block, value head) for the vectors over key channels, and one for the values and the step size; a lane owns
+// the channels lane, lane + 32, ...  CI > 0: at most 32 CI channels, whose q and
 // k stay in registers over the unit norms' sums; CI = 0: any number, computed twice.
 template <typename T, int CI, int TAPS>
-__global__ void __launch_bounds__(256) delta_blocks_kernel(const DeltaBlocksParams p) {
+__global__ void __launch_bounds__(256, CI > 0 ? 3 : 1) delta_blocks_kernel(const DeltaBlocksParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int lane = threadIdx.x & 31, h = blockIdx.y * 8 + (threadIdx.x >> 5);
-  if (h >= p.H) return;
+  const int lane = threadIdx.x & 31, unit = blockIdx.y * 8 + (threadIdx.x >> 5);
+  if (unit >= 2 * p.H) return;
+  const int h = unit < p.H ? unit : unit - p.H;
   const int blocks = (p.S + kT - 1) / kT;
   const int64_t blk = blockIdx.x, b = blk / blocks;
   const int s = static_cast<int>(blk - b * blocks) * kT;
@@ -135,6 +155,20 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const DeltaBlocksPara
   const int64_t channels = 2ll * G * C + static_cast<int64_t>(H) * E;
   const float* ring = p.ring + b * p.taps * channels;
   const float* in = p.proj + row * p.ld;
+  if (unit >= p.H) {
+    if (lane < kT) p.coef[(blk * H + h) * kCoef + lane] = lane < n ? sigmoid_f(in[lane * p.ld + p.b_off + h]) : 0.f;
+#pragma unroll 2
+    for (int e = lane; e < E; e += 32) {
+      const int64_t ch = static_cast<int64_t>(h) * E + e;
+      float y[kT];
+      conv_block<T, TAPS>(in + p.v_off + ch, p.ld, static_cast<const T*>(p.conv_v) + ch * p.taps, ring + 2ll * G * C + ch, channels, p.taps, s,
+                          pos, n, y);
+#pragma unroll
+      for (int t = 0; t < kT; ++t)
+        if (t < n) p.v[(row + t) * H * E + ch] = y[t];
+    }
+    return;
+  }
 
   auto conv_qk = [&](int c, float (&q)[kT], float (&k)[kT]) {
     const int64_t ch = static_cast<int64_t>(hk) * C + c;
@@ -153,9 +187,9 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const DeltaBlocksPara
   if constexpr (CI > 0) {
 #pragma unroll
     for (int i = 0; i < CI; ++i) {
-      if (lane + 32 * i >= C) break;
-      conv_qk(lane + 32 * i, qr[i], kr[i]);
-      add_squares(qr[i], kr[i]);
+      // (channels past the end repeat the last one and count nothing)
+      conv_qk(lane + 32 * i < C ? lane + 32 * i : C - 1, qr[i], kr[i]);
+      if (lane + 32 * i < C) add_squares(qr[i], kr[i]);
     }
   } else {
     for (int c = lane; c < C; c += 32) {
@@ -191,8 +225,7 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const DeltaBlocksPara
   if constexpr (CI > 0) {
 #pragma unroll
     for (int i = 0; i < CI; ++i) {
-      if (lane + 32 * i >= C) break;
-      finish(lane + 32 * i, qr[i], kr[i]);
+      if (lane + 32 * i < C) finish(lane + 32 * i, qr[i], kr[i]);
     }
   } else {
     for (int c = lane; c < C; c += 32) {
@@ -201,18 +234,7 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const DeltaBlocksPara
       finish(c, q, k);
     }
   }
-  float* cf = p.coef + (blk * H + h) * kCoef;
-  store_coef(coef, cf, lane);
-  if (lane < kT) cf[lane] = lane < n ? sigmoid_f(in[lane * p.ld + p.b_off + h]) : 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const int64_t ch = static_cast<int64_t>(h) * E + e;
-    float y[kT];
-    conv_block<T, TAPS>(in + p.v_off + ch, p.ld, static_cast<const T*>(p.conv_v) + ch * p.taps, ring + 2ll * G * C + ch, channels, p.taps, s,
-                        pos, n, y);
-#pragma unroll
-    for (int t = 0; t < kT; ++t)
-      if (t < n) p.v[(row + t) * H * E + ch] = y[t];
-  }
+  store_coef(coef, p.coef + (blk * H + h) * kCoef, lane);
 }
 
 struct GlaBlocksParams {
@@ -289,7 +311,7 @@ __global__ void __launch_bounds__(256) round_columns_kernel(const float* x, int6
 template <typename T>
 int delta_blocks(const DeltaBlocksParams& p, int B, cudaStream_t st) {
   auto kern = p.taps > 4 || p.C > 128 ? delta_blocks_kernel<T, 0, kMaxTaps> : (p.C <= 64 ? delta_blocks_kernel<T, 2, 4> : delta_blocks_kernel<T, 4, 4>);
-  LRI_CUDA(launch_pdl(kern, dim3(static_cast<unsigned>(B) * ((p.S + kT - 1) / kT), (p.H + 7) / 8), dim3(256), 0, st, p));
+  LRI_CUDA(launch_pdl(kern, dim3(static_cast<unsigned>(B) * ((p.S + kT - 1) / kT), (2 * p.H + 7) / 8), dim3(256), 0, st, p));
   LRI_LAUNCH_CHECK("delta_blocks_kernel");
   return LRI_OK;
 }

@@ -18,6 +18,7 @@ namespace lri {
 namespace {
 
 constexpr int kThreads = 256, kCols = 32, kMaxCluster = 8;
+constexpr int kRegTaps = 4;  // convolution weights up to this many taps are held in registers
 constexpr int kStageBytes = 96 * 1024;  // second projections up to this size are staged in shared memory
 
 struct StepParams {
@@ -66,11 +67,46 @@ __device__ __forceinline__ void rows_dot(const T* w, int rank, const float* x, i
   }
 }
 
+// Convolution of one channel at this position, silu taken; its input enters the ring.  The slots that are read are other ones
+// than the one that is written.
+template <typename T>
+struct StepConv {
+  float w[kRegTaps];  // w[j]: tap j tokens back
+  const T* taps_w;
+  __device__ __forceinline__ void load(const void* w_all, int64_t ch, int taps, bool live) {
+    taps_w = static_cast<const T*>(w_all) + ch * taps;
+#pragma unroll
+    for (int j = 0; j < kRegTaps; ++j) w[j] = live && taps <= kRegTaps && j < taps ? Num<T>::to_f(taps_w[taps - 1 - j]) : 0.f;
+  }
+  // slot: pos % taps
+  __device__ __forceinline__ float run(float x, float* ring, int64_t channels, int taps, int64_t pos, int slot, bool keep) const {
+    float y = w[0] * x;
+    if (taps <= kRegTaps) {
+      float old[kRegTaps];
+#pragma unroll
+      for (int j = 1; j < kRegTaps; ++j) {
+        const int at = slot >= j ? slot - j : slot - j + taps;
+        old[j] = j < taps && pos >= j ? ring[at * channels] : 0.f;
+      }
+#pragma unroll
+      for (int j = 1; j < kRegTaps; ++j) y = fmaf(w[j], old[j], y);
+    } else {
+      y = Num<T>::to_f(taps_w[taps - 1]) * x;
+      for (int j = 1; j < taps; ++j)
+        if (pos >= j) y = fmaf(Num<T>::to_f(taps_w[taps - 1 - j]), ring[(slot >= j ? slot - j : slot - j + taps) * channels], y);
+    }
+    if (keep && pos >= 0) ring[slot * channels] = x;
+    return silu_f(y);
+  }
+};
+
 template <typename T, bool DELTA, int RV>
 __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p) {
   constexpr int CP = 32 * RV;
   extern __shared__ __align__(16) uint8_t step_smem[];
+  static_assert(CP <= kThreads, "a thread takes one key channel");
   __shared__ __align__(16) float sq[CP], sk[CP], sg[CP];
+  __shared__ float sbias[CP];
   __shared__ float sv[kCols], sgate[kCols], part[8], cluster_part[kMaxCluster];
   cg::cluster_group cluster = cg::this_cluster();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rg = lane & 7, cl = lane >> 3;
@@ -94,6 +130,21 @@ __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
   for (int c = tid; c < C; c += kThreads) asm volatile("prefetch.global.L2 [%0];" ::"l"(st_base + static_cast<int64_t>(c) * E + col0));
+  // a thread takes key channel tid and, the last ones, a value channel
+  const int64_t ch_k = static_cast<int64_t>(hk) * C + tid;
+  const int e_mine = tid - (kThreads - kCols);
+  const bool has_k = tid < C, has_v = e_mine >= 0 && e_mine < cols;
+  const int64_t ch_v = static_cast<int64_t>(h) * E + col0 + e_mine;
+  [[maybe_unused]] StepConv<T> conv_q, conv_k, conv_v;
+  float a = 0.f;
+  if constexpr (DELTA) {
+    conv_q.load(p.conv_q, ch_k, p.taps, has_k);
+    conv_k.load(p.conv_k, ch_k, p.taps, has_k);
+    conv_v.load(p.conv_v, ch_v, p.taps, has_v);
+    a = expf(Num<T>::to_f(static_cast<const T*>(p.a_log)[h]));
+  }
+  if (has_k) sbias[tid] = Num<T>::to_f(static_cast<const T*>(p.bias)[h * C + tid]);
+  const float norm_w = e0 < E ? Num<T>::to_f(static_cast<const T*>(p.norm_w)[e0]) : 0.f;
   pdl_launch_dependents();
   pdl_wait();
 
@@ -110,38 +161,31 @@ __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p
   const float* in = p.proj + b * p.ld;
   const int64_t channels = 2ll * G * C + static_cast<int64_t>(H) * E;
   float* ring = DELTA ? p.ring + b * p.taps * channels : nullptr;
-  // convolution of one channel at this position; its input enters the ring (slots that are read here are other ones)
-  auto conv = [&](int64_t off, int64_t ch, const void* w, int64_t ch_w, bool keep) {
-    const T* tw = static_cast<const T*>(w) + ch_w * p.taps;
-    const float x = in[off];
-    float y = 0.f;
-    for (int j = p.taps - 1; j > 0; --j)
-      if (pos - j >= 0) y = fmaf(Num<T>::to_f(tw[p.taps - 1 - j]), ring[(pos - j) % p.taps * channels + ch], y);
-    y = fmaf(Num<T>::to_f(tw[p.taps - 1]), x, y);
-    if (keep && pos >= 0) ring[pos % p.taps * channels + ch] = x;
-    return silu_f(y);
-  };
-  const bool first = blockIdx.x == 0 && h % (H / G) == 0;  // keeps the shared channels of its group
-  for (int c = tid; c < CP; c += kThreads) {
+  const float beta = DELTA ? sigmoid_f(in[p.b_off + h]) : 0.f;
+  if (tid < CP) {
     float q = 0.f, k = 0.f;
-    if (c < C) {
-      const int64_t ch = static_cast<int64_t>(hk) * C + c;
+    if (has_k) {
+      q = in[p.q_off + ch_k], k = in[p.k_off + ch_k];
       if constexpr (DELTA) {
-        q = conv(p.q_off + ch, ch, p.conv_q, ch, first);
-        k = conv(p.k_off + ch, static_cast<int64_t>(G) * C + ch, p.conv_k, ch, first);
-      } else {
-        q = in[p.q_off + ch], k = in[p.k_off + ch];
+        const int slot = static_cast<int>((pos < 0 ? 0 : pos) % p.taps);
+        const bool keep = blockIdx.x == 0 && h % (H / G) == 0;  // the first CTA of a group keeps the shared channels
+        q = conv_q.run(q, ring + ch_k, channels, p.taps, pos, slot, keep);
+        k = conv_k.run(k, ring + static_cast<int64_t>(G) * C + ch_k, channels, p.taps, pos, slot, keep);
       }
+    } else {
+      sg[tid] = 1.f;
     }
-    sq[c] = q, sk[c] = k, sg[c] = 1.f;
+    sq[tid] = q, sk[tid] = k;
   }
-  if (tid >= kThreads - kCols) {
-    const int e = tid - (kThreads - kCols);
-    const int64_t ch = static_cast<int64_t>(h) * E + col0 + e;
+  if (e_mine >= 0) {
     float v = 0.f;
-    if (e < cols) v = DELTA ? conv(p.v_off + ch, 2ll * G * C + ch, p.conv_v, ch, true) : in[p.v_off + ch];
-    sv[e] = v;
-    if (!DELTA) sgate[e] = e < cols ? silu_f(in[p.gate_off + ch]) : 0.f;
+    if (has_v) {
+      v = in[p.v_off + ch_v];
+      if constexpr (DELTA)
+        v = conv_v.run(v, ring + 2ll * G * C + ch_v, channels, p.taps, pos, static_cast<int>((pos < 0 ? 0 : pos) % p.taps), true);
+    }
+    sv[e_mine] = v;
+    if (!DELTA) sgate[e_mine] = has_v ? silu_f(in[p.gate_off + ch_v]) : 0.f;
   }
   for (int i = tid; i < p.a_rank; i += kThreads) x_a[i] = rnd<T>(in[p.a_off + i]);
   if (DELTA)
@@ -149,20 +193,18 @@ __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
 
-  const float a = DELTA ? expf(Num<T>::to_f(static_cast<const T*>(p.a_log)[h])) : 0.f;
   rows_dot<T>(a2, p.a_rank, x_a, C, [&](int c, float z) {
-    z += Num<T>::to_f(static_cast<const T*>(p.bias)[h * C + c]);
+    z += sbias[c];
     sg[c] = DELTA ? delta_decay_f(z, a) : logistic_decay_f(z, p.inv_tau);
   });
   if constexpr (DELTA) rows_dot<T>(g2, p.g_rank, x_g, cols, [&](int e, float z) { sgate[e] = sigmoid_f(z); });
-  float qs = 1.0f / sqrtf(static_cast<float>(C)), ks = 1.f, kq = 0.f, beta = 0.f;
+  float qs = 1.0f / sqrtf(static_cast<float>(C)), ks = 1.f, kq = 0.f;
   if constexpr (DELTA) {
     float qq = 0.f, kk = 0.f;
     for (int c = lane; c < C; c += 32) qq = fmaf(sq[c], sq[c], qq), kk = fmaf(sk[c], sk[c], kk), kq = fmaf(sq[c], sk[c], kq);
     qs /= sqrtf(warp_sum(qq) + kUnitEps);
     ks = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
     kq = warp_sum(kq) * ks * qs;
-    beta = sigmoid_f(in[p.b_off + h]);
   }
   __syncthreads();
 
@@ -221,7 +263,7 @@ __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p
   if (rg == 0 && e0 < E) {
     const float inv = p.factor / sqrtf(total / static_cast<float>(E) + p.eps);
     static_cast<T*>(p.out)[b * p.out_ld + static_cast<int64_t>(h) * E + e0] =
-        Num<T>::from_f(o * inv * Num<T>::to_f(static_cast<const T*>(p.norm_w)[e0]) * sgate[my]);
+        Num<T>::from_f(o * inv * norm_w * sgate[my]);
   }
 }
 

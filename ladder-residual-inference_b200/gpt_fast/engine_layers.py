@@ -14,6 +14,8 @@ streams that a sublayer mixes (`StreamBranch`).
 A forward reads positions from the device and can be captured in a CUDA graph.  A batch row's first position decides
 whether a recurrence starts anew (0) or continues, so a row is reused by feeding position 0 again.
 """
+import os
+
 import torch
 import torch.distributed as dist
 
@@ -112,6 +114,10 @@ class LayerEngine(Engine):
             if packed:
                 self.moe_packed = buf(128 * tiles, self.d)
                 self.moe_scale = torch.zeros(128 * tiles, dtype=torch.float32, device=device)
+        self.side_stream = None
+        if of("chunked_attention") and self.comm.world == 1 and self.resid.is_cuda and os.environ.get("LRI_SIDE_STREAM", "1") != "0":
+            self.side_stream = torch.cuda.Stream()
+            self._fork, self._join_event = torch.cuda.Event(), torch.cuda.Event()
         self._setup_head(max_batch, device, dtype)
         self.ready = True
 
@@ -196,12 +202,31 @@ class LayerEngine(Engine):
         ops.head_norm_gate(self.scan_o, m.norm, eps, self.scan_gate, v, "sigmoid", factor, y, y_ld, rows, m.heads)
 
     def _parallel(self, m, rows, B, S, pos, eps):
+        """The sides read the same projections and write their own columns of y; on one GPU they run on two streams."""
         at, ld = _offsets(m.parts(), self.off), m.out_width
         y = self.y.view(-1)
-        for side, run, first in (("left", self._grouped, 0), ("right", self._gated_delta, m.left.out_width)):
-            sub = getattr(m, side)
-            offs = {k[len(side) + 1:]: v for k, v in at.items() if k.startswith(side + ".")}
-            run(sub, offs, y[first:], ld, m.scales[side == "right"], rows, B, S, pos, eps)
+
+        def offsets(side):
+            return {k[len(side) + 1:]: v for k, v in at.items() if k.startswith(side + ".")}
+
+        def left():
+            self._grouped(m.left, offsets("left"), y, ld, m.scales[0], rows, B, S, pos, eps)
+
+        def right():
+            self._gated_delta(m.right, offsets("right"), y[m.left.out_width:], ld, m.scales[1], rows, B, S, pos, eps)
+
+        if self.side_stream is None:
+            left()
+            right()
+            return
+        main, side = torch.cuda.current_stream(), self.side_stream
+        self._fork.record(main)
+        side.wait_event(self._fork)
+        with torch.cuda.stream(side):
+            left()
+            self._join_event.record(side)
+        right()
+        main.wait_event(self._join_event)
 
     def _experts(self, m, rows):
         """Returns (result rows, slots, number of result rows): the row of each (token, choice) pair in self.moe_out."""
