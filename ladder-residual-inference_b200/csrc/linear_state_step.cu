@@ -5,9 +5,10 @@
 //                             size, state update, readout, RMSNorm over the value channels, sigmoid gate
 //   gated linear attention    low-rank decay, state update, readout, RMSNorm, silu gate
 //
-// A cluster serves one (sequence, head), each CTA 32 value channels.  A warp owns four of them, 8 lanes a column of the
+// A cluster serves one (sequence, head), each CTA 32 NC value channels.  A warp owns 4 NC of them, 8 lanes a column of the
 // state.  What all columns need (queries, keys, decays) every CTA computes for itself; only the sums of squares of the
-// results cross the cluster.  Weights are fetched, and the state is asked into the L2, before the preceding kernel is awaited.
+// results cross the cluster.  A small grid takes NC = 1 (shortest chain), a large one NC = 4 (least work, mostly no cluster).
+// Weights are fetched, and the state is asked into the L2, before the preceding kernel is awaited.
 #include <cooperative_groups.h>
 
 #include "linear_state.cuh"
@@ -17,7 +18,7 @@ namespace cg = cooperative_groups;
 namespace lri {
 namespace {
 
-constexpr int kThreads = 256, kCols = 32, kMaxCluster = 8;
+constexpr int kThreads = 256, kMaxCluster = 8;
 constexpr int kRegTaps = 4;  // convolution weights up to this many taps are held in registers
 constexpr int kStageBytes = 96 * 1024;  // second projections up to this size are staged in shared memory
 
@@ -47,23 +48,24 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src) : "memory");
 }
 
-// w[row] . x for the rows first, first + 32, ... below n: 8 lanes a row, 4 rows a warp; fn(row, sum) on one lane
-template <typename T, typename Fn>
-__device__ __forceinline__ void rows_dot(const T* w, int rank, const float* x, int n, Fn fn) {
+// y[row] = w[row] . x for n rows: 8 lanes a row, 4 rows a warp
+template <typename T>
+__device__ __forceinline__ void rows_dot(const T* w, int rank, const float* x, int n, float* y) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = (lane & 7) * 8;
   for (int r0 = warp * 4; r0 < n; r0 += kThreads / 8) {
     const int r = r0 + (lane >> 3);
     float acc = 0.f;
     if (r < n)
       for (int i = part; i < rank; i += 64) {
-        float f[8];
-        load8<T>(w + static_cast<int64_t>(r) * rank + i, f);
+        float f[8], xv[8];
+        load8<T>(w + r * rank + i, f);
+        load8<float>(x + i, xv);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc = fmaf(f[e], x[i + e], acc);
+        for (int e = 0; e < 8; ++e) acc = fmaf(f[e], xv[e], acc);
       }
 #pragma unroll
     for (int o = 1; o < 8; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-    if ((lane & 7) == 0 && r < n) fn(r, acc);
+    if ((lane & 7) == 0 && r < n) y[r] = acc;
   }
 }
 
@@ -79,7 +81,7 @@ struct StepConv {
     for (int j = 0; j < kRegTaps; ++j) w[j] = live && taps <= kRegTaps && j < taps ? Num<T>::to_f(taps_w[taps - 1 - j]) : 0.f;
   }
   // slot: pos % taps
-  __device__ __forceinline__ float run(float x, float* ring, int64_t channels, int taps, int64_t pos, int slot, bool keep) const {
+  __device__ __forceinline__ float run(float x, float* ring, int64_t channels, int taps, int pos, int slot, bool keep) const {
     float y = w[0] * x;
     if (taps <= kRegTaps) {
       float old[kRegTaps];
@@ -100,19 +102,21 @@ struct StepConv {
   }
 };
 
-template <typename T, bool DELTA, int RV>
-__global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p) {
-  constexpr int CP = 32 * RV;
+template <typename T, bool DELTA, int RV, int NC>
+__global__ void __launch_bounds__(kThreads, RV <= 4 ? 2 : 1) state_step_kernel(const StepParams p) {
+  constexpr int CP = 32 * RV, kCols = 32 * NC;
   extern __shared__ __align__(16) uint8_t step_smem[];
-  static_assert(CP <= kThreads, "a thread takes one key channel");
+  static_assert(CP <= kThreads && kCols <= kThreads, "a thread takes one key channel and one value channel");
   __shared__ __align__(16) float sq[CP], sk[CP], sg[CP];
   __shared__ float sbias[CP];
-  __shared__ float sv[kCols], sgate[kCols], part[8], cluster_part[kMaxCluster];
+  __shared__ float sv[kCols], sgate[kCols], part[8], part_qk[8][3], cluster_part[kMaxCluster];
   cg::cluster_group cluster = cg::this_cluster();
+  const int ranks = static_cast<int>(cluster.num_blocks());
+  if (ranks > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");  // waited for before the first remote store
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rg = lane & 7, cl = lane >> 3;
   const int h = blockIdx.y, H = p.H, G = p.G, C = p.C, E = p.E, hk = h / (H / G);
   const int64_t b = blockIdx.z;
-  const int col0 = blockIdx.x * kCols, my = warp * 4 + cl, e0 = col0 + my;
+  const int col0 = blockIdx.x * kCols, my = (warp * 4 + cl) * NC, e0 = col0 + my;
   const int cols = E - col0 < kCols ? E - col0 : kCols;
   float* x_a = reinterpret_cast<float*>(step_smem);  // input of the decay's second projection
   float* x_g = x_a + p.a_rank;
@@ -129,7 +133,8 @@ __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p
     if (DELTA) g2 = w_smem + na * kPer;
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
-  for (int c = tid; c < C; c += kThreads) asm volatile("prefetch.global.L2 [%0];" ::"l"(st_base + static_cast<int64_t>(c) * E + col0));
+  for (int i = tid; i < C * NC; i += kThreads)  // one request per 128-byte line
+    if (i % NC * 32 < cols) asm volatile("prefetch.global.L2 [%0];" ::"l"(st_base + i / NC * E + col0 + i % NC * 32));
   // a thread takes key channel tid and, the last ones, a value channel
   const int64_t ch_k = static_cast<int64_t>(hk) * C + tid;
   const int e_mine = tid - (kThreads - kCols);
@@ -144,30 +149,38 @@ __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p
     a = expf(Num<T>::to_f(static_cast<const T*>(p.a_log)[h]));
   }
   if (has_k) sbias[tid] = Num<T>::to_f(static_cast<const T*>(p.bias)[h * C + tid]);
-  const float norm_w = e0 < E ? Num<T>::to_f(static_cast<const T*>(p.norm_w)[e0]) : 0.f;
+  float norm_w[NC];
+#pragma unroll
+  for (int j = 0; j < NC; ++j) norm_w[j] = e0 + j < E ? Num<T>::to_f(static_cast<const T*>(p.norm_w)[e0 + j]) : 0.f;
   pdl_launch_dependents();
   pdl_wait();
 
   // ---- state, and what the columns share -------------------------------------------------------------------
-  const int64_t pos = load_pos(p.input_pos, p.pos_is_i64, 0);
-  float st[RV][4];
+  const int pos = static_cast<int>(load_pos(p.input_pos, p.pos_is_i64, 0));
+  float st[RV][4][NC];
+  float* st_mine = st_base + 4 * rg * E + e0;
 #pragma unroll
   for (int i = 0; i < RV; ++i)
 #pragma unroll
     for (int r = 0; r < 4; ++r) {
-      const int c = 32 * i + 4 * rg + r;
-      st[i][r] = pos > 0 && c < C && e0 < E ? st_base[static_cast<int64_t>(c) * E + e0] : 0.f;
+      const bool live = (C == CP || 32 * i + 4 * rg + r < C) && e0 < E;
+      if constexpr (NC == 4) {  // E is a multiple of 4
+        const float4 v = pos > 0 && live ? *reinterpret_cast<const float4*>(st_mine + (32 * i + r) * E) : make_float4(0.f, 0.f, 0.f, 0.f);
+        st[i][r][0] = v.x, st[i][r][1] = v.y, st[i][r][2] = v.z, st[i][r][3] = v.w;
+      } else {
+        st[i][r][0] = pos > 0 && live ? st_mine[(32 * i + r) * E] : 0.f;
+      }
     }
   const float* in = p.proj + b * p.ld;
   const int64_t channels = 2ll * G * C + static_cast<int64_t>(H) * E;
   float* ring = DELTA ? p.ring + b * p.taps * channels : nullptr;
   const float beta = DELTA ? sigmoid_f(in[p.b_off + h]) : 0.f;
+  const int slot = DELTA ? (pos < 0 ? 0 : pos) % p.taps : 0;
+  float q = 0.f, k = 0.f;
   if (tid < CP) {
-    float q = 0.f, k = 0.f;
     if (has_k) {
       q = in[p.q_off + ch_k], k = in[p.k_off + ch_k];
       if constexpr (DELTA) {
-        const int slot = static_cast<int>((pos < 0 ? 0 : pos) % p.taps);
         const bool keep = blockIdx.x == 0 && h % (H / G) == 0;  // the first CTA of a group keeps the shared channels
         q = conv_q.run(q, ring + ch_k, channels, p.taps, pos, slot, keep);
         k = conv_k.run(k, ring + static_cast<int64_t>(G) * C + ch_k, channels, p.taps, pos, slot, keep);
@@ -182,7 +195,7 @@ __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p
     if (has_v) {
       v = in[p.v_off + ch_v];
       if constexpr (DELTA)
-        v = conv_v.run(v, ring + 2ll * G * C + ch_v, channels, p.taps, pos, static_cast<int>((pos < 0 ? 0 : pos) % p.taps), true);
+        v = conv_v.run(v, ring + 2ll * G * C + ch_v, channels, p.taps, pos, slot, true);
     }
     sv[e_mine] = v;
     if (!DELTA) sgate[e_mine] = has_v ? silu_f(in[p.gate_off + ch_v]) : 0.f;
@@ -190,93 +203,132 @@ __global__ void __launch_bounds__(kThreads) state_step_kernel(const StepParams p
   for (int i = tid; i < p.a_rank; i += kThreads) x_a[i] = rnd<T>(in[p.a_off + i]);
   if (DELTA)
     for (int i = tid; i < p.g_rank; i += kThreads) x_g[i] = rnd<T>(in[p.gate_off + i]);
+  if constexpr (DELTA) {
+    const float qq = warp_sum(q * q), kk = warp_sum(k * k), kq = warp_sum(k * q);
+    if (lane == 0) part_qk[warp][0] = qq, part_qk[warp][1] = kk, part_qk[warp][2] = kq;
+  }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
 
-  rows_dot<T>(a2, p.a_rank, x_a, C, [&](int c, float z) {
-    z += sbias[c];
-    sg[c] = DELTA ? delta_decay_f(z, a) : logistic_decay_f(z, p.inv_tau);
-  });
-  if constexpr (DELTA) rows_dot<T>(g2, p.g_rank, x_g, cols, [&](int e, float z) { sgate[e] = sigmoid_f(z); });
+  rows_dot<T>(a2, p.a_rank, x_a, C, sg);
+  if constexpr (DELTA) rows_dot<T>(g2, p.g_rank, x_g, cols, sgate);
   float qs = 1.0f / sqrtf(static_cast<float>(C)), ks = 1.f, kq = 0.f;
   if constexpr (DELTA) {
     float qq = 0.f, kk = 0.f;
-    for (int c = lane; c < C; c += 32) qq = fmaf(sq[c], sq[c], qq), kk = fmaf(sk[c], sk[c], kk), kq = fmaf(sq[c], sk[c], kq);
-    qs /= sqrtf(warp_sum(qq) + kUnitEps);
-    ks = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
-    kq = warp_sum(kq) * ks * qs;
+#pragma unroll
+    for (int w = 0; w < (CP < kThreads ? CP / 32 : 8); ++w) qq += part_qk[w][0], kk += part_qk[w][1], kq += part_qk[w][2];
+    qs /= sqrtf(qq + kUnitEps);
+    ks = 1.0f / sqrtf(kk + kUnitEps);
+    kq *= ks * qs;
   }
+  __syncthreads();
+  if (has_k) {
+    const float z = sg[tid] + sbias[tid];
+    sg[tid] = DELTA ? delta_decay_f(z, a) : logistic_decay_f(z, p.inv_tau);
+  }
+  if (DELTA && has_v) sgate[e_mine] = sigmoid_f(sgate[e_mine]);
   __syncthreads();
 
   // ---- the recurrence ------------------------------------------------------------------------------------------
-  float dk = 0.f, dq = 0.f, u = sv[my];
+  float dk[NC], dq[NC], u[NC], o[NC];
+#pragma unroll
+  for (int j = 0; j < NC; ++j) dk[j] = dq[j] = 0.f, u[j] = sv[my + j];
 #pragma unroll
   for (int i = 0; i < RV; ++i) {
-    const float4 g = *reinterpret_cast<const float4*>(&sg[32 * i + 4 * rg]);
-    const float4 q = *reinterpret_cast<const float4*>(&sq[32 * i + 4 * rg]), k = *reinterpret_cast<const float4*>(&sk[32 * i + 4 * rg]);
-    st[i][0] *= g.x, st[i][1] *= g.y, st[i][2] *= g.z, st[i][3] *= g.w;
-    if constexpr (!DELTA) {
-      st[i][0] = fmaf(k.x, u, st[i][0]), st[i][1] = fmaf(k.y, u, st[i][1]), st[i][2] = fmaf(k.z, u, st[i][2]), st[i][3] = fmaf(k.w, u, st[i][3]);
-    } else {
-      dk = fmaf(st[i][0], k.x, dk), dk = fmaf(st[i][1], k.y, dk), dk = fmaf(st[i][2], k.z, dk), dk = fmaf(st[i][3], k.w, dk);
-    }
-    dq = fmaf(st[i][0], q.x, dq), dq = fmaf(st[i][1], q.y, dq), dq = fmaf(st[i][2], q.z, dq), dq = fmaf(st[i][3], q.w, dq);
+    float g[4], q4[4], k4[4];
+    *reinterpret_cast<float4*>(g) = *reinterpret_cast<const float4*>(&sg[32 * i + 4 * rg]);
+    *reinterpret_cast<float4*>(q4) = *reinterpret_cast<const float4*>(&sq[32 * i + 4 * rg]);
+    *reinterpret_cast<float4*>(k4) = *reinterpret_cast<const float4*>(&sk[32 * i + 4 * rg]);
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+#pragma unroll
+      for (int j = 0; j < NC; ++j) {
+        float& x = st[i][r][j];
+        x *= g[r];
+        if (DELTA)
+          dk[j] = fmaf(x, k4[r], dk[j]);
+        else
+          x = fmaf(k4[r], u[j], x);
+        dq[j] = fmaf(x, q4[r], dq[j]);
+      }
   }
 #pragma unroll
-  for (int o = 1; o < 8; o <<= 1) {
-    if (DELTA) dk += __shfl_xor_sync(0xffffffffu, dk, o);
-    dq += __shfl_xor_sync(0xffffffffu, dq, o);
-  }
-  float o = dq * qs;
-  if constexpr (DELTA) {
-    u = beta * (u - dk * ks);
-    o = fmaf(u, kq, o);
-    const float uk = u * ks;
+  for (int w = 1; w < 8; w <<= 1)
 #pragma unroll
-    for (int i = 0; i < RV; ++i) {
-      const float4 k = *reinterpret_cast<const float4*>(&sk[32 * i + 4 * rg]);
-      st[i][0] = fmaf(k.x, uk, st[i][0]), st[i][1] = fmaf(k.y, uk, st[i][1]), st[i][2] = fmaf(k.z, uk, st[i][2]), st[i][3] = fmaf(k.w, uk, st[i][3]);
+    for (int j = 0; j < NC; ++j) {
+      if (DELTA) dk[j] += __shfl_xor_sync(0xffffffffu, dk[j], w);
+      dq[j] += __shfl_xor_sync(0xffffffffu, dq[j], w);
     }
-  }
+  float squares = 0.f;
 #pragma unroll
-  for (int i = 0; i < RV; ++i)
-#pragma unroll
-    for (int r = 0; r < 4; ++r) {
-      const int c = 32 * i + 4 * rg + r;
-      if (c < C && e0 < E) st_base[static_cast<int64_t>(c) * E + e0] = st[i][r];
+  for (int j = 0; j < NC; ++j) {
+    o[j] = dq[j] * qs;
+    if constexpr (DELTA) {
+      u[j] = beta * (u[j] - dk[j] * ks);
+      o[j] = fmaf(u[j], kq, o[j]);
+      u[j] *= ks;
     }
+    if (e0 + j < E) squares = fmaf(o[j], o[j], squares);
+  }
 
   // ---- norm over the head's value channels, gate -----------------------------------------------------------------
-  const float ss = warp_sum(rg == 0 && e0 < E ? o * o : 0.f);
+  const float ss = warp_sum(rg == 0 ? squares : 0.f);
   if (lane == 0) part[warp] = ss;
   __syncthreads();
-  const int ranks = static_cast<int>(cluster.num_blocks());
-  if (tid < ranks) {
-    float s = 0.f;
-#pragma unroll
-    for (int w = 0; w < 8; ++w) s += part[w];
-    *cluster.map_shared_rank(&cluster_part[cluster.block_rank()], tid) = s;
-  }
-  cluster.sync();
   float total = 0.f;
-  for (int r = 0; r < ranks; ++r) total += cluster_part[r];
-  if (rg == 0 && e0 < E) {
+  if (ranks > 1) {
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+    if (tid < ranks) {
+      float s = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) s += part[w];
+      *cluster.map_shared_rank(&cluster_part[cluster.block_rank()], tid) = s;
+    }
+    cluster.sync();
+    for (int r = 0; r < ranks; ++r) total += cluster_part[r];
+  } else {
+#pragma unroll
+    for (int w = 0; w < 8; ++w) total += part[w];
+  }
+  if (rg == 0) {
     const float inv = p.factor / sqrtf(total / static_cast<float>(E) + p.eps);
-    static_cast<T*>(p.out)[b * p.out_ld + static_cast<int64_t>(h) * E + e0] =
-        Num<T>::from_f(o * inv * norm_w * sgate[my]);
+    T* dst = static_cast<T*>(p.out) + b * p.out_ld + static_cast<int64_t>(h) * E + e0;
+#pragma unroll
+    for (int j = 0; j < NC; ++j)
+      if (e0 + j < E) dst[j] = Num<T>::from_f(o[j] * inv * norm_w[j] * sgate[my + j]);
+  }
+
+  // ---- the state, behind the barriers, which would wait for its stores ---------------------------------------------
+#pragma unroll
+  for (int i = 0; i < RV; ++i) {
+    float k4[4];
+    *reinterpret_cast<float4*>(k4) = *reinterpret_cast<const float4*>(&sk[32 * i + 4 * rg]);
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+      if (DELTA)
+#pragma unroll
+        for (int j = 0; j < NC; ++j) st[i][r][j] = fmaf(k4[r], u[j], st[i][r][j]);
+      if ((C == CP || 32 * i + 4 * rg + r < C) && e0 < E) {
+        if constexpr (NC == 4)
+          *reinterpret_cast<float4*>(st_mine + (32 * i + r) * E) = make_float4(st[i][r][0], st[i][r][1], st[i][r][2], st[i][r][3]);
+        else
+          st_mine[(32 * i + r) * E] = st[i][r][0];
+      }
+    }
   }
 }
 
-template <typename T, bool DELTA, int RV>
+template <typename T, bool DELTA, int RV, int NC>
 int launch(const StepParams& p, int B, cudaStream_t st) {
+  constexpr int kCols = 32 * NC;
   const size_t x_bytes = (static_cast<size_t>(p.a_rank) + (DELTA ? p.g_rank : 0)) * 4;
   const size_t w_bytes = (static_cast<size_t>(p.C) * p.a_rank + (DELTA ? static_cast<size_t>(kCols) * p.g_rank : 0)) * sizeof(T);
+  const unsigned cs = (p.E + kCols - 1) / kCols;
   StepParams q = p;
   q.staged = w_bytes <= kStageBytes;
-  auto kern = state_step_kernel<T, DELTA, RV>;
+  auto kern = state_step_kernel<T, DELTA, RV, NC>;
   static std::atomic<unsigned long long> attr_set{0};
   LRI_ONCE_PER_DEVICE(attr_set, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * kStageBytes));
-  const unsigned cs = (p.E + kCols - 1) / kCols;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(cs, p.H, B);
   cfg.blockDim = dim3(kThreads);
@@ -295,12 +347,20 @@ int launch(const StepParams& p, int B, cudaStream_t st) {
   LRI_LAUNCH_CHECK("state_step_kernel");
   return LRI_OK;
 }
+template <typename T, bool DELTA, int RV>
+int by_grid(const StepParams& p, int B, cudaStream_t st) {
+  if constexpr (RV <= 4) {
+    const int64_t ctas = static_cast<int64_t>(B) * p.H * ((p.E + 31) / 32);
+    if (ctas > 2ll * device_sm_count() && p.E % 4 == 0 && p.E > 32) return launch<T, DELTA, RV, 4>(p, B, st);
+  }
+  return launch<T, DELTA, RV, 1>(p, B, st);
+}
 template <typename T, bool DELTA>
 int by_channels(const StepParams& p, int B, cudaStream_t st) {
-  if (p.C <= 32) return launch<T, DELTA, 1>(p, B, st);
-  if (p.C <= 64) return launch<T, DELTA, 2>(p, B, st);
-  if (p.C <= 128) return launch<T, DELTA, 4>(p, B, st);
-  return launch<T, DELTA, 8>(p, B, st);
+  if (p.C <= 32) return by_grid<T, DELTA, 1>(p, B, st);
+  if (p.C <= 64) return by_grid<T, DELTA, 2>(p, B, st);
+  if (p.C <= 128) return by_grid<T, DELTA, 4>(p, B, st);
+  return by_grid<T, DELTA, 8>(p, B, st);
 }
 template <bool DELTA>
 int run(const char* who, int dtype, const StepParams& p, int B, cudaStream_t st) {
@@ -310,7 +370,8 @@ int run(const char* who, int dtype, const StepParams& p, int B, cudaStream_t st)
               B, p.H, p.G);
   LRI_REQUIRE(lri_state_step_supports(p.C, p.E, p.a_rank, p.g_rank), LRI_ERR_UNSUPPORTED, "%s: dim=%d vdim=%d ranks %d, %d", who, p.C, p.E,
               p.a_rank, p.g_rank);
-  LRI_REQUIRE(aligned16(p.a2) && aligned16(p.g2), LRI_ERR_ALIGN, "%s: second projections must be 16-byte aligned", who);
+  LRI_REQUIRE(aligned16(p.a2) && aligned16(p.g2) && aligned16(p.state), LRI_ERR_ALIGN,
+              "%s: second projections and state must be 16-byte aligned", who);
   if (B == 0) return LRI_OK;
   if (dtype == LRI_BF16) return by_channels<__nv_bfloat16, DELTA>(p, B, st);
   if (dtype == LRI_FP16) return by_channels<__half, DELTA>(p, B, st);
@@ -323,7 +384,7 @@ int run(const char* who, int dtype, const StepParams& p, int B, cudaStream_t st)
 using namespace lri;
 
 extern "C" int lri_state_step_supports(int dim, int vdim, int decay_rank, int gate_rank) {
-  return dim >= 1 && dim <= 256 && vdim >= 1 && vdim <= kCols * kMaxCluster && decay_rank >= 8 && decay_rank % 8 == 0 && decay_rank <= 4096 &&
+  return dim >= 1 && dim <= 256 && vdim >= 1 && vdim <= 32 * kMaxCluster && decay_rank >= 8 && decay_rank % 8 == 0 && decay_rank <= 4096 &&
          gate_rank >= 0 && gate_rank % 8 == 0 && gate_rank <= 4096;
 }
 

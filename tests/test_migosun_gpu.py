@@ -277,7 +277,8 @@ class _Delta:
 
 
 DELTA_SIZES = [(1, 41, 2, 1, 12, 20, 4, 5, 9, -1.0), (2, 60, 4, 2, 64, 64, 3, 16, 8, -3.0), (1, 75, 2, 2, 128, 96, 4, 24, 16, 0.0), (1, 33, 3, 3, 48, 128, 1, 8, 8, 3.0),
-               (2, 37, 2, 1, 9, 7, 2, 1, 1, -1.0), (1, 30, 1, 1, 200, 40, 7, 8, 70, -2.0), (1, 24, 1, 1, 32, 32, 4, 8, 8, 60.0)]
+               (2, 37, 2, 1, 9, 7, 2, 1, 1, -1.0), (1, 30, 1, 1, 200, 40, 7, 8, 70, -2.0), (1, 24, 1, 1, 32, 32, 4, 8, 8, 60.0),
+               (1, 14, 2, 1, 256, 250, 4, 8, 8, -1.0), (30, 9, 4, 2, 52, 72, 3, 16, 8, -1.0)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
