@@ -101,7 +101,7 @@ def _stream_list(n_layer, width, streams, left, right, gla, ff, vocab, every=3):
 # Residual streams with dense feed-forwards: width, depth, vocabulary and feed-forward of the Llama shape of the same name.
 STREAM_LISTS = {
     "migosun-tiny": _stream_list(4, 192, 3, (6, 2, 32, 48), (4, 2, 32, 16), (3, 32, 64, 8), 320, 512),
-    "migosun-1b": _stream_list(16, 2048, 4, (32, 8, 64, 2048), (16, 16, 64, 64), (16, 64, 128, 16), 8192, 128256),
+    "migosun-1b": _stream_list(16, 2048, 4, (32, 8, 64, 4096), (16, 16, 64, 64), (16, 64, 128, 16), 8192, 128256),
     "migosun-8b": _stream_list(32, 4096, 4, (32, 8, 128, 8192), (16, 16, 128, 128), (16, 128, 256, 16), 14336, 128256),
 }
 
