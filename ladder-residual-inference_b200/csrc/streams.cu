@@ -32,51 +32,38 @@ struct StreamParams {
   int streams, dim;
 };
 
-template <int VEC>
-__device__ __forceinline__ void load_f(const float* p, float (&f)[VEC]) {
-  if constexpr (VEC == 4) {
-    const float4 v = *reinterpret_cast<const float4*>(p);
-    f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
-  } else {
-    f[0] = p[0];
-  }
+constexpr int kVec = 4;
+__device__ __forceinline__ void load_f(const float* p, float (&f)[kVec]) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
 }
-template <int VEC>
-__device__ __forceinline__ void store_f(float* p, const float (&f)[VEC]) {
-  if constexpr (VEC == 4)
-    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  else
-    p[0] = f[0];
+__device__ __forceinline__ void store_f(float* p, const float (&f)[kVec]) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
 }
-template <typename T, int VEC>
-__device__ __forceinline__ void load_t(const T* p, float (&f)[VEC]) {
+template <typename T>
+__device__ __forceinline__ void load_t(const T* p, float (&f)[kVec]) {
   if constexpr (std::is_same<T, float>::value) {
-    load_f<VEC>(p, f);
-  } else if constexpr (VEC == 4) {
+    load_f(p, f);
+  } else {
     const uint2 v = *reinterpret_cast<const uint2*>(p);
     Num<T>::unpack2(v.x, f[0], f[1]);
     Num<T>::unpack2(v.y, f[2], f[3]);
-  } else {
-    f[0] = Num<T>::to_f(p[0]);
   }
 }
-template <typename T, int VEC>
-__device__ __forceinline__ void store_t(T* p, const float (&f)[VEC]) {
-  if constexpr (std::is_same<T, float>::value) {
-    store_f<VEC>(p, f);
-  } else if constexpr (VEC == 4) {
+template <typename T>
+__device__ __forceinline__ void store_t(T* p, const float (&f)[kVec]) {
+  if constexpr (std::is_same<T, float>::value)
+    store_f(p, f);
+  else
     *reinterpret_cast<uint2*>(p) = make_uint2(pack2<T>(f[0], f[1]), pack2<T>(f[2], f[3]));
-  } else {
-    p[0] = Num<T>::from_f(f[0]);
-  }
 }
 
-// SM: bound of the number of streams.  NV vectors per thread.
-template <typename T, int SM, int VEC, int NV, int THREADS>
+// SM: bound of the number of streams.  NV vectors of four elements per thread.
+template <typename T, int SM, int NV, int THREADS>
 __global__ void __launch_bounds__(THREADS) join_streams_kernel(const StreamParams p) {
   __shared__ float part[33];
   __shared__ float mix[SM][SM], out[SM], in[SM];
-  const int n = p.streams, dim = p.dim, nvec = dim / VEC;
+  const int n = p.streams, dim = p.dim, nvec = dim / kVec;
   const int64_t row = blockIdx.x;
   if (threadIdx.x < SM) {
     const int t = threadIdx.x;
@@ -87,11 +74,11 @@ __global__ void __launch_bounds__(THREADS) join_streams_kernel(const StreamParam
     const int s = i / SM, t = i % SM;
     mix[s][t] = p.mix && s < n && t < n ? Num<T>::to_f(static_cast<const T*>(p.mix)[s * n + t]) : 0.f;
   }
-  float w[NV][VEC];  // constant of the model: fetched while the preceding kernel drains
+  float w[NV][kVec];  // constant of the model: fetched while the preceding kernel drains
   const T* weight = static_cast<const T*>(p.weight);
 #pragma unroll
   for (int i = 0; i < NV; ++i)
-    if (threadIdx.x + i * THREADS < nvec) load_t<T, VEC>(weight + (threadIdx.x + i * THREADS) * VEC, w[i]);
+    if (threadIdx.x + i * THREADS < nvec) load_t<T>(weight + (threadIdx.x + i * THREADS) * kVec, w[i]);
   pdl_launch_dependents();
   pdl_wait();
   __syncthreads();
@@ -102,50 +89,50 @@ __global__ void __launch_bounds__(THREADS) join_streams_kernel(const StreamParam
   }
   const float* x = p.x + row * n * dim;
   float* xo = p.x_out + row * n * dim;
-  float u[NV][VEC], ss = 0.f;
+  float u[NV][kVec], ss = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int v = threadIdx.x + i * THREADS;
     if (v >= nvec) continue;
-    const int64_t e0 = static_cast<int64_t>(v) * VEC;
+    const int64_t e0 = static_cast<int64_t>(v) * kVec;
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) u[i][e] = 0.f;
+    for (int e = 0; e < kVec; ++e) u[i][e] = 0.f;
     if (p.table) {
-      float f[VEC];
-      load_t<T, VEC>(static_cast<const T*>(p.table) + src * dim + e0, f);
+      float f[kVec];
+      load_t<T>(static_cast<const T*>(p.table) + src * dim + e0, f);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) f[e] *= p.scale;
+      for (int e = 0; e < kVec; ++e) f[e] *= p.scale;
 #pragma unroll
       for (int t = 0; t < SM; ++t) {
         if (t >= n) break;
-        if (p.x_out) store_f<VEC>(xo + static_cast<int64_t>(t) * dim + e0, f);
+        if (p.x_out) store_f(xo + static_cast<int64_t>(t) * dim + e0, f);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) u[i][e] = fmaf(in[t], f[e], u[i][e]);
+        for (int e = 0; e < kVec; ++e) u[i][e] = fmaf(in[t], f[e], u[i][e]);
       }
     } else {
-      float y[VEC], old[SM][VEC];
+      float y[kVec], old[SM][kVec];
 #pragma unroll
       for (int s = 0; s < SM; ++s)
-        if (s < n) load_f<VEC>(x + static_cast<int64_t>(s) * dim + e0, old[s]);
-      load_t<T, VEC>(static_cast<const T*>(p.y) + row * dim + e0, y);
+        if (s < n) load_f(x + static_cast<int64_t>(s) * dim + e0, old[s]);
+      load_t<T>(static_cast<const T*>(p.y) + row * dim + e0, y);
 #pragma unroll
       for (int t = 0; t < SM; ++t) {
         if (t >= n) break;
-        float f[VEC];
+        float f[kVec];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) f[e] = out[t] * y[e];
+        for (int e = 0; e < kVec; ++e) f[e] = out[t] * y[e];
 #pragma unroll
         for (int s = 0; s < SM; ++s)
           if (s < n)
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) f[e] = fmaf(mix[s][t], old[s][e], f[e]);
-        if (p.x_out) store_f<VEC>(xo + static_cast<int64_t>(t) * dim + e0, f);
+            for (int e = 0; e < kVec; ++e) f[e] = fmaf(mix[s][t], old[s][e], f[e]);
+        if (p.x_out) store_f(xo + static_cast<int64_t>(t) * dim + e0, f);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) u[i][e] = fmaf(in[t], f[e], u[i][e]);
+        for (int e = 0; e < kVec; ++e) u[i][e] = fmaf(in[t], f[e], u[i][e]);
       }
     }
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) ss += u[i][e] * u[i][e];
+    for (int e = 0; e < kVec; ++e) ss += u[i][e] * u[i][e];
   }
   const float inv = 1.0f / sqrtf(block_sum(ss, part) / static_cast<float>(dim) + p.eps);
   T* dst = static_cast<T*>(p.normed) + row * dim;
@@ -153,16 +140,16 @@ __global__ void __launch_bounds__(THREADS) join_streams_kernel(const StreamParam
   for (int i = 0; i < NV; ++i) {
     const int v = threadIdx.x + i * THREADS;
     if (v >= nvec) continue;
-    float f[VEC];
+    float f[kVec];
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) f[e] = u[i][e] * inv * w[i][e];
-    store_t<T, VEC>(dst + static_cast<int64_t>(v) * VEC, f);
+    for (int e = 0; e < kVec; ++e) f[e] = u[i][e] * inv * w[i][e];
+    store_t<T>(dst + static_cast<int64_t>(v) * kVec, f);
   }
 }
 
-template <typename T, int SM, int VEC, int NV, int THREADS>
+template <typename T, int SM, int NV, int THREADS>
 int launch(const StreamParams& p, int64_t rows, cudaStream_t st) {
-  LRI_CUDA(launch_pdl(join_streams_kernel<T, SM, VEC, NV, THREADS>, dim3(static_cast<unsigned>(rows)), dim3(THREADS), 0, st, p));
+  LRI_CUDA(launch_pdl(join_streams_kernel<T, SM, NV, THREADS>, dim3(static_cast<unsigned>(rows)), dim3(THREADS), 0, st, p));
   LRI_LAUNCH_CHECK("join_streams_kernel");
   return LRI_OK;
 }
@@ -221,11 +208,11 @@ int launch_generic(const StreamParams& p, int64_t rows, cudaStream_t st) {
 template <typename T, int SM>
 int by_size(const StreamParams& p, int64_t rows, cudaStream_t st) {
   const int nvec = p.dim / 4;
-  if (nvec <= 256) return launch<T, SM, 4, 1, 256>(p, rows, st);
-  if (nvec <= 512) return launch<T, SM, 4, 1, 512>(p, rows, st);
-  if (rows <= 16 && nvec <= 1024) return launch<T, SM, 4, 1, 1024>(p, rows, st);  // few rows: one thread's latency chain
-  if (nvec <= 1024) return launch<T, SM, 4, 4, 256>(p, rows, st);
-  return launch<T, SM, 4, 8, 512>(p, rows, st);
+  if (nvec <= 256) return launch<T, SM, 1, 256>(p, rows, st);
+  if (nvec <= 512) return launch<T, SM, 1, 512>(p, rows, st);
+  if (rows <= 16 && nvec <= 1024) return launch<T, SM, 1, 1024>(p, rows, st);  // few rows: one thread's latency chain
+  if (nvec <= 1024) return launch<T, SM, 4, 256>(p, rows, st);
+  return launch<T, SM, 8, 512>(p, rows, st);
 }
 
 template <typename T>
